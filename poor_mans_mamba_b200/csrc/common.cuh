@@ -56,6 +56,20 @@ __device__ __forceinline__ float softplus_f(float v) {
   return log1pf(expf(v));
 }
 
+// Softplus and exponential of the recurrences' walks, in the type the walk computes in (float, or double for the
+// float storage type).
+template <typename ACC>
+__device__ __forceinline__ ACC scan_softplus(ACC v);
+template <>
+__device__ __forceinline__ float scan_softplus<float>(float v) { return softplus_f(v); }
+template <>
+__device__ __forceinline__ double scan_softplus<double>(double v) {
+  if (v > 40.0) return v;
+  return log1p(exp(v));
+}
+__device__ __forceinline__ float scan_exp(float v) { return expf(v); }
+__device__ __forceinline__ double scan_exp(double v) { return exp(v); }
+
 inline int launch_status() { return static_cast<int>(cudaGetLastError()); }
 
 // Programmatic dependent launch.  A kernel started with launch_pdl may begin while the kernel

@@ -254,6 +254,12 @@ __global__ void scale_f32_kernel(float* __restrict__ x, float s, size_t n) {
   if (i < n) x[i] *= s;
 }
 
+// x = cap * tanh(s * x / cap)
+__global__ void softcap_f32_kernel(float* __restrict__ x, float s, float cap, size_t n) {
+  const size_t i = static_cast<size_t>(blockIdx.x) * blockDim.x + threadIdx.x;
+  if (i < n) x[i] = cap * tanhf(s * x[i] / cap);
+}
+
 template <typename S>
 __global__ void cast_scale_kernel(float* __restrict__ out, const S* __restrict__ in, float s, size_t n) {
   const size_t i = static_cast<size_t>(blockIdx.x) * blockDim.x + threadIdx.x;
@@ -326,6 +332,13 @@ PMM_EXPORT int pmm_scale_f32(float* x, float s, long long n, cudaStream_t stream
   if (n <= 0) return 0;
   pmm::scale_f32_kernel<<<static_cast<unsigned>((n + 255) / 256), 256, 0, stream>>>(
       x, s, static_cast<size_t>(n));
+  return pmm::launch_status();
+}
+
+PMM_EXPORT int pmm_softcap_f32(float* x, float s, float cap, long long n, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (!(cap > 0.f)) return PMM_ERR_BAD_ARGUMENT;
+  pmm::softcap_f32_kernel<<<static_cast<unsigned>((n + 255) / 256), 256, 0, stream>>>(x, s, cap, static_cast<size_t>(n));
   return pmm::launch_status();
 }
 

@@ -78,7 +78,8 @@ __global__ void __launch_bounds__(kRouteWarps * 32)
   __syncthreads();
   if (scored) {
     // Scores s = sigmoid(z) (scored == 2: s = softmax(z) over all experts, a group's score is its largest choice
-    // score, and the weights are the chosen s times scale, not divided by their sum).  The choice runs on s + correction, among the experts of the `keep` groups (of `groups`
+    // score, and the weights are the chosen s times scale, not divided by their sum; scored == 3: sigmoids whose
+    // weights are not divided by their sum either).  The choice runs on s + correction, among the experts of the `keep` groups (of `groups`
     // equal groups of neighbours) whose two largest choice scores sum highest; every other expert's choice score is
     // -inf.  The weights are the chosen s over their sum (+ 1e-20), times scale.  The lower index wins a tie.
     float* extra = logits + TOK * E;
@@ -167,7 +168,7 @@ __global__ void __launch_bounds__(kRouteWarps * 32)
         }
         __syncwarp();
       }
-      const float inv = scored == 2 ? scale : scale / (denom + 1e-20f);
+      const float inv = scored >= 2 ? scale : scale / (denom + 1e-20f);
       for (int j = lane; j < top; j += 32) weights[static_cast<size_t>(t0 + r) * top + j] *= inv;
     }
     return;
@@ -340,7 +341,7 @@ __global__ void __launch_bounds__(256)
     moe_gemm_generic_kernel(const S* __restrict__ a, long long ld_a, const S* __restrict__ w,
                             const int* __restrict__ perm, const int* __restrict__ offsets,
                             const int* __restrict__ tile_start, int E, int top, int K, int N, float limit, float alpha,
-                            float shift, int ungated, void* __restrict__ out) {
+                            float shift, int ungated, const float* __restrict__ row_w, void* __restrict__ out) {
   __shared__ float As[kGenRows][kGenK + 1];
   __shared__ float Bs[UP ? 2 : 1][kGenCols][kGenK + 1];
   __shared__ int src_row[kGenRows];
@@ -393,8 +394,9 @@ __global__ void __launch_bounds__(256)
     const int i = row0 + ty * 4 + r;
     if (i >= row1) continue;
     if (UP) {
+      const float rw = row_w ? row_w[perm[i]] : 1.f;
       stf(static_cast<S*>(out) + static_cast<size_t>(i) * N + n0 + tx,
-          clamped_glu(acc[0][r], acc[UP ? 1 : 0][r], limit, alpha, shift));
+          clamped_glu(rw * acc[0][r], rw * acc[UP ? 1 : 0][r], limit, alpha, shift));
     } else {
       // (ungated: the activation's rows stay in the order of the sorted pairs, like the gated form's)
       stf(static_cast<S*>(out) + static_cast<size_t>(ungated ? i : perm[i]) * N + n0 + tx,
@@ -413,7 +415,7 @@ __global__ void __launch_bounds__(128)
     moe_gemm_mma_kernel(const bf16* __restrict__ a, long long ld_a, const bf16* __restrict__ w,
                         const int* __restrict__ perm, const int* __restrict__ offsets,
                         const int* __restrict__ tile_start, int E, int top, int K, int N, float limit, float alpha,
-                        float shift, int ungated, void* __restrict__ out) {
+                        float shift, int ungated, const float* __restrict__ row_w, void* __restrict__ out) {
   constexpr int BROWS = UP ? 2 * kMmaCols : kMmaCols;
   constexpr int LD = kMmaK + kMmaPad;  // 40 elements = 80 bytes: ldmatrix rows fall into different banks
   __shared__ __align__(16) bf16 As[2][kMmaRows][LD];
@@ -493,6 +495,7 @@ __global__ void __launch_bounds__(128)
     const int r = r_lo + half * 8;
     const int i = row0 + r;
     if (i >= row1) continue;
+    const float rw = (UP && row_w) ? row_w[dst_row[r]] : 1.f;
 #pragma unroll
     for (int j = 0; j < kMmaCols / 8; ++j) {
 #pragma unroll
@@ -500,7 +503,7 @@ __global__ void __launch_bounds__(128)
         const int col = n0 + j * 8 + c_in + q;
         if (col >= N) continue;
         if (UP) {
-          const float g = acc[j][half * 2 + q], u = acc[UP ? j + kMmaCols / 8 : j][half * 2 + q];
+          const float g = rw * acc[j][half * 2 + q], u = rw * acc[UP ? j + kMmaCols / 8 : j][half * 2 + q];
           static_cast<bf16*>(out)[static_cast<size_t>(i) * N + col] = __float2bfloat16_rn(clamped_glu(g, u, limit, alpha, shift));
         } else {
           const float val = acc[j][half * 2 + q];
@@ -522,7 +525,7 @@ __global__ void __launch_bounds__(128)
     moe_gemm_few_kernel(const bf16* __restrict__ a, long long ld_a, const bf16* __restrict__ w,
                         const int* __restrict__ perm, const int* __restrict__ offsets,
                         const int* __restrict__ tile_start, int E, int top, int K, int N, float limit, float alpha,
-                        float shift, int ungated, bf16* __restrict__ out) {
+                        float shift, int ungated, const float* __restrict__ row_w, bf16* __restrict__ out) {
   constexpr int BROWS = UP ? 2 * kFewCols : kFewCols;
   constexpr int kStageElems = (kFewRows + BROWS) * kFewLd;
   extern __shared__ __align__(16) unsigned char few_smem[];
@@ -603,6 +606,7 @@ __global__ void __launch_bounds__(128)
     const int r = (lane >> 2) + half * 8;
     const int i = row0 + r;
     if (i >= row1) continue;
+    const float rw = (UP && row_w) ? row_w[dst_row[r]] : 1.f;
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
 #pragma unroll
@@ -611,7 +615,7 @@ __global__ void __launch_bounds__(128)
         if (col >= N) continue;
         if (UP) {
           out[static_cast<size_t>(i) * N + col] =
-              __float2bfloat16_rn(clamped_glu(acc[j][half * 2 + q], acc[UP ? 2 + j : j][half * 2 + q], limit, alpha, shift));
+              __float2bfloat16_rn(clamped_glu(rw * acc[j][half * 2 + q], rw * acc[UP ? 2 + j : j][half * 2 + q], limit, alpha, shift));
         } else {
           const float val = acc[j][half * 2 + q];
           out[static_cast<size_t>(ungated ? i : dst_row[r]) * N + col] = __float2bfloat16_rn(ungated ? relu_squared(val) : val);
@@ -621,7 +625,7 @@ __global__ void __launch_bounds__(128)
   }
 }
 
-// out[t] = sum_j p[t, j] y[t * top + j] (+ shared[t], times shared_gate[t] where there is one); y, shared and out in the storage type, the sum in float.
+// out[t] = sum_j p[t, j] y[t * top + j] (weights null: every p is 1) (+ shared[t], times shared_gate[t] where there is one); y, shared and out in the storage type, the sum in float.
 template <typename S>
 __global__ void __launch_bounds__(256)
     moe_combine_kernel(const S* __restrict__ y, const float* __restrict__ weights, const S* __restrict__ shared,
@@ -632,7 +636,7 @@ __global__ void __launch_bounds__(256)
   for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < D; i += gridDim.y * blockDim.x) {
     float acc = 0.f;
     for (int j = 0; j < top; ++j)
-      acc += weights[static_cast<size_t>(t) * top + j] * ldf(y + (static_cast<size_t>(t) * top + j) * D + i);
+      acc += (weights ? weights[static_cast<size_t>(t) * top + j] : 1.f) * ldf(y + (static_cast<size_t>(t) * top + j) * D + i);
     if (shared) acc += (shared_gate ? shared_gate[t] : 1.f) * ldf(shared + static_cast<size_t>(t) * D + i);
     stf(out + static_cast<size_t>(t) * D + i, acc);
   }
@@ -660,7 +664,7 @@ int launch_route(const void* x, long long ld_x, const float* w, const float* bia
 
 // scored == 0: the `top` largest logits, weights their softmax.  scored != 0: scores sigmoid(z); the choice runs on
 // score + correction (may be null) within the `keep` best of `groups` groups of neighbours; weights are the chosen
-// scores over their sum, times scale.  scored == 2: scores softmax(z) over all experts; groups are ranked by their
+// scores over their sum, times scale (scored == 3: the chosen scores times scale).  scored == 2: scores softmax(z) over all experts; groups are ranked by their
 // largest choice score; weights are the chosen scores times scale.
 PMM_EXPORT int pmm_moe_route(const void* x, long long ld_x, const float* w, const float* bias, int* ids, float* weights,
                              int T, int D, int E, int top, int scored, const float* correction, int groups, int keep,
@@ -708,12 +712,14 @@ PMM_EXPORT int pmm_moe_tile_rows(int tensor_cores) {
 
 // up == 1: a = x [T, K] (ld_a), w [E, 2N, K], out act [A, N] (storage type).  up == 0: a = act [A, K], w [E, N, K],
 // out y [A, N] in the storage type.  up == 2 (ungated experts): a = x [T, K], w [E, N, K], out act [A, N] = max(x W^T, 0)^2
-// in the order of the sorted pairs.  tensor_cores != 0 needs bfloat16, K % 8 == 0, ld_a % 8 == 0 and 16-byte aligned a, w; the
+// in the order of the sorted pairs.  row_w [A] (up == 1, or null): pair i's input is row_w[perm[i]] * x, applied to its
+// gate and up sums before the activation.  tensor_cores != 0 needs bfloat16, K % 8 == 0, ld_a % 8 == 0 and 16-byte aligned a, w; the
 // plan must have been made with pmm_moe_tile_rows(tensor_cores) rows a tile.
 PMM_EXPORT int pmm_moe_gemm(const void* a, long long ld_a, const void* w, const int* perm, const int* offsets,
                             const int* tile_start, int A, int E, int top, int K, int N, int up, float limit, float alpha,
-                            float shift, void* out, int tensor_cores, int dtype, cudaStream_t stream) {
+                            float shift, const float* row_w, void* out, int tensor_cores, int dtype, cudaStream_t stream) {
   if (A <= 0) return 0;
+  if (row_w && up != 1) return PMM_ERR_BAD_ARGUMENT;
   if (E <= 0 || top <= 0 || K <= 0 || N <= 0 || up < 0 || up > 2) return PMM_ERR_BAD_ARGUMENT;
   const int ungated = up == 2 ? 1 : 0;
   if (ungated) up = 0;
@@ -735,34 +741,34 @@ PMM_EXPORT int pmm_moe_gemm(const void* a, long long ld_a, const void* w, const 
         if (err != cudaSuccess) return static_cast<int>(err);
         pmm::launch_pdl(kern, grid, dim3(128), smem, stream, static_cast<const pmm::bf16*>(a), ld_a,
                         static_cast<const pmm::bf16*>(w), perm, offsets, tile_start, E, top, K, N, limit, alpha, shift,
-                        ungated, static_cast<pmm::bf16*>(out));
+                        ungated, row_w, static_cast<pmm::bf16*>(out));
       } else {
         auto kern = pmm::moe_gemm_few_kernel<false>;
         err = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
         if (err != cudaSuccess) return static_cast<int>(err);
         pmm::launch_pdl(kern, grid, dim3(128), smem, stream, static_cast<const pmm::bf16*>(a), ld_a,
                         static_cast<const pmm::bf16*>(w), perm, offsets, tile_start, E, top, K, N, limit, alpha, shift,
-                        ungated, static_cast<pmm::bf16*>(out));
+                        ungated, row_w, static_cast<pmm::bf16*>(out));
       }
       return pmm::launch_status();
     }
     const dim3 grid((N + pmm::kMmaCols - 1) / pmm::kMmaCols, row_tiles);
     if (up)
       pmm::launch_pdl(pmm::moe_gemm_mma_kernel<true>, grid, dim3(128), 0, stream, static_cast<const pmm::bf16*>(a), ld_a,
-                      static_cast<const pmm::bf16*>(w), perm, offsets, tile_start, E, top, K, N, limit, alpha, shift, ungated, out);
+                      static_cast<const pmm::bf16*>(w), perm, offsets, tile_start, E, top, K, N, limit, alpha, shift, ungated, row_w, out);
     else
       pmm::launch_pdl(pmm::moe_gemm_mma_kernel<false>, grid, dim3(128), 0, stream, static_cast<const pmm::bf16*>(a), ld_a,
-                      static_cast<const pmm::bf16*>(w), perm, offsets, tile_start, E, top, K, N, limit, alpha, shift, ungated, out);
+                      static_cast<const pmm::bf16*>(w), perm, offsets, tile_start, E, top, K, N, limit, alpha, shift, ungated, row_w, out);
     return pmm::launch_status();
   }
   const dim3 grid((N + pmm::kGenCols - 1) / pmm::kGenCols, row_tiles);
   PMM_DISPATCH_DTYPE(dtype, S, {
     if (up)
       pmm::launch_pdl(pmm::moe_gemm_generic_kernel<S, true>, grid, dim3(256), 0, stream, static_cast<const S*>(a), ld_a,
-                      static_cast<const S*>(w), perm, offsets, tile_start, E, top, K, N, limit, alpha, shift, ungated, out);
+                      static_cast<const S*>(w), perm, offsets, tile_start, E, top, K, N, limit, alpha, shift, ungated, row_w, out);
     else
       pmm::launch_pdl(pmm::moe_gemm_generic_kernel<S, false>, grid, dim3(256), 0, stream, static_cast<const S*>(a), ld_a,
-                      static_cast<const S*>(w), perm, offsets, tile_start, E, top, K, N, limit, alpha, shift, ungated, out);
+                      static_cast<const S*>(w), perm, offsets, tile_start, E, top, K, N, limit, alpha, shift, ungated, row_w, out);
   });
   return pmm::launch_status();
 }

@@ -49,8 +49,8 @@ template <bool UP>
 __global__ void __launch_bounds__(kGThreads)
     moe_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
                   const int* __restrict__ perm, const int* __restrict__ offsets, const int* __restrict__ tile_start, int E,
-                  int K, int N, float limit, float alpha, float shift, int ungated, void* __restrict__ out,
-                  int* __restrict__ status) {
+                  int K, int N, float limit, float alpha, float shift, int ungated,
+                  const float* __restrict__ row_w, void* __restrict__ out, int* __restrict__ status) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ unsigned char smem_raw[];
@@ -153,6 +153,7 @@ __global__ void __launch_bounds__(kGThreads)
       const unsigned lane_base = tmem_base + (static_cast<unsigned>(quad * 32) << 16);
       if (UP) {
         bf16* dst_row = static_cast<bf16*>(out) + static_cast<size_t>(row_ok ? i : 0) * N;
+        const float rw = (row_w && row_ok) ? row_w[perm[i]] : 1.f;  // the pair's input is rw * x
 #pragma unroll 1
         for (int c = 0; c < kGN / 64; ++c) {
           unsigned g[32], u[32];
@@ -171,8 +172,8 @@ __global__ void __launch_bounds__(kGThreads)
                   float r[2];
 #pragma unroll
                   for (int h = 0; h < 2; ++h) {
-                    const float gv = fminf(__uint_as_float(g[j + 2 * q + h]), limit);
-                    const float uv = fminf(fmaxf(__uint_as_float(u[j + 2 * q + h]), -limit), limit);
+                    const float gv = fminf(rw * __uint_as_float(g[j + 2 * q + h]), limit);
+                    const float uv = fminf(fmaxf(rw * __uint_as_float(u[j + 2 * q + h]), -limit), limit);
                     r[h] = __fdividef(gv, 1.f + __expf(-alpha * gv)) * (uv + shift);
                   }
                   p2[q] = __floats2bfloat162_rn(r[0], r[1]);
@@ -270,11 +271,12 @@ PMM_EXPORT int pmm_moe_gather_rows(const void* x, long long ld_x, const int* per
 
 // a [A, K] bfloat16 rows in the order of the sorted pairs (row stride ld_a); w the experts' stacked matrices
 // [E * (up ? 2N : N), K]; the plan made with rows of pmm_moe_tc_tile_rows().  up: out = act [A, N] bfloat16;
-// else out = y [A, N] bfloat16, row perm[i].  status: one int, stays 0 unless a bounded wait gave up.
+// else out = y [A, N] bfloat16, row perm[i].  row_w [A] (up == 1, or null): pair i's input is row_w[perm[i]] times its row.  status: one int, stays 0 unless a bounded wait gave up.
 PMM_EXPORT int pmm_moe_tc_gemm(const void* a, long long ld_a, const void* w, const int* perm, const int* offsets,
                                const int* tile_start, int A, int E, int K, int N, int up, float limit, float alpha,
-                               float shift, void* out, int* status, cudaStream_t stream) {
+                               float shift, const float* row_w, void* out, int* status, cudaStream_t stream) {
   if (A <= 0) return 0;
+  if (row_w && up != 1) return PMM_ERR_BAD_ARGUMENT;
   if (E <= 0 || !pmm_moe_tc_supported(K, N, ld_a) || !status || up < 0 || up > 2) return PMM_ERR_BAD_ARGUMENT;
   const int ungated = up == 2 ? 1 : 0;  // up == 2: w [E * N, K], out = max(a W^T, 0)^2 in the order of the sorted pairs
   if (ungated) up = 0;
@@ -293,13 +295,13 @@ PMM_EXPORT int pmm_moe_tc_gemm(const void* a, long long ld_a, const void* w, con
     err = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(pmm::kGSmem));
     if (err != cudaSuccess) return static_cast<int>(err);
     pmm::launch_pdl(kern, grid, dim3(pmm::kGThreads), pmm::kGSmem, stream, map_a, map_w, perm, offsets, tile_start, E, K, N,
-                    limit, alpha, shift, ungated, out, status);
+                    limit, alpha, shift, ungated, row_w, out, status);
   } else {
     auto kern = pmm::moe_tc_kernel<false>;
     err = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(pmm::kGSmem));
     if (err != cudaSuccess) return static_cast<int>(err);
     pmm::launch_pdl(kern, grid, dim3(pmm::kGThreads), pmm::kGSmem, stream, map_a, map_w, perm, offsets, tile_start, E, K, N,
-                    limit, alpha, shift, ungated, out, status);
+                    limit, alpha, shift, ungated, row_w, out, status);
   }
   return pmm::launch_status();
 }

@@ -10,12 +10,14 @@
 // [page, plane, page_size, G*Dp]: all heads are laid out Dp = max(d, dv) rounded up wide, padded
 // with zeros, so that one attention kernel of head size Dp serves both sizes (zeros add nothing to
 // a score, and the padded value columns come out zero and are dropped by the output projection's
-// operand view).
+// operand view).  v_norm_eps >= 0: every value head is divided by its own root mean square
+// (v / sqrt(mean(v^2) + eps) over its dv entries, no weight, float) before it is written.
 #include "common.cuh"
 
 namespace pmm {
 
 constexpr int kRopeMaxPairs = 128;  // rot_dims <= 256
+constexpr int kRopeMaxGroups = 256;  // key/value heads whose values are normed
 
 // `sn`, `cs`: the token's sines and cosines per rotated pair (shared memory, made once a token).
 template <typename S>
@@ -42,8 +44,10 @@ __global__ void __launch_bounds__(256)
                             int page_size, S* __restrict__ q_out, int H, int G, int d, int dv, int Dp,
                             int rot_dims, int half_layout, const float* __restrict__ q_bias,
                             const float* __restrict__ k_bias, const float* __restrict__ v_bias,
-                            const float* __restrict__ q_norm_w, const float* __restrict__ k_norm_w, float norm_eps) {
+                            const float* __restrict__ q_norm_w, const float* __restrict__ k_norm_w, float norm_eps,
+                            float v_norm_eps) {
   __shared__ float sn_t[kRopeMaxPairs], cs_t[kRopeMaxPairs];
+  __shared__ float inv_v[kRopeMaxGroups];
   __shared__ float red[32];
   pdl_launch_dependents();
   pdl_wait();
@@ -70,6 +74,18 @@ __global__ void __launch_bounds__(256)
     }
     inv_k = 1.f / sqrtf(block_sum(ss, red) / static_cast<float>(G * d) + norm_eps);
   }
+  if (v_norm_eps >= 0.f) {
+    const int lane = threadIdx.x & 31;
+    for (int g = threadIdx.x >> 5; g < G; g += blockDim.x >> 5) {  // a warp per value head
+      float ss = 0.f;
+      for (int i = lane; i < dv; i += 32) {
+        const float x = ldf(v + static_cast<long long>(t) * ld_v + g * dv + i) + (v_bias ? v_bias[g * dv + i] : 0.f);
+        ss += x * x;
+      }
+      ss = warp_sum(ss);
+      if (lane == 0) inv_v[g] = 1.f / sqrtf(ss / static_cast<float>(dv) + v_norm_eps);
+    }
+  }
   __syncthreads();
   const int n_q = H * Dp, n_kv = G * Dp;
   const int page = block_table[static_cast<size_t>(seq_of[t]) * max_blocks + pos / page_size];
@@ -88,7 +104,9 @@ __global__ void __launch_bounds__(256)
       stf(k_row + c, val);
     } else {
       const int c = e - n_q - n_kv, g = c / Dp, i = c - g * Dp;
-      stf(v_row + c, i < dv ? ldf(v + static_cast<long long>(t) * ld_v + g * dv + i) + (v_bias ? v_bias[g * dv + i] : 0.f) : 0.f);
+      float val = i < dv ? ldf(v + static_cast<long long>(t) * ld_v + g * dv + i) + (v_bias ? v_bias[g * dv + i] : 0.f) : 0.f;
+      if (v_norm_eps >= 0.f) val *= inv_v[g];
+      stf(v_row + c, val);
     }
   }
 }
@@ -98,23 +116,24 @@ __global__ void __launch_bounds__(256)
 // q [T, H*d], k [T, G*d], v [T, G*dv] rows of stride ld; inv_freq [rot_dims/2] floats (may be nullptr when
 // rot_dims is 0); pool [pages, 2, page_size, G*Dp]; q_out [T, H*Dp]; q_bias [H*d], k_bias [G*d], v_bias [G*dv]
 // floats or nullptr; q_norm_w [H*d], k_norm_w [G*d] floats or nullptr: an RMS norm over the token's whole query
-// (key) projection before rotation, eps inside the root.  Values are never normed.
+// (key) projection before rotation, eps inside the root; v_norm_eps >= 0: every value head over its own root mean
+// square (at most kRopeMaxGroups heads).
 PMM_EXPORT int pmm_rope_pairs_store(const void* q, long long ld_q, const void* k, long long ld_k, const void* v,
                                     long long ld_v, const float* inv_freq, const int* positions, const int* seq_of,
                                     const int* block_table, int max_blocks, void* pool, int page_size, void* q_out,
                                     int T, int H, int G, int d, int dv, int Dp, int rot_dims, int half_layout,
                                     const float* q_bias, const float* k_bias, const float* v_bias,
-                                    const float* q_norm_w, const float* k_norm_w, float norm_eps, int dtype,
-                                    cudaStream_t stream) {
+                                    const float* q_norm_w, const float* k_norm_w, float norm_eps, float v_norm_eps,
+                                    int dtype, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (H <= 0 || G <= 0 || d <= 0 || dv <= 0 || Dp < d || Dp < dv || rot_dims < 0 || rot_dims > d || rot_dims % 2 ||
-      rot_dims > 2 * pmm::kRopeMaxPairs || (rot_dims > 0 && !inv_freq) || page_size <= 0)
+      (v_norm_eps >= 0.f && G > pmm::kRopeMaxGroups) || rot_dims > 2 * pmm::kRopeMaxPairs || (rot_dims > 0 && !inv_freq) || page_size <= 0)
     return PMM_ERR_BAD_ARGUMENT;
   PMM_DISPATCH_DTYPE(dtype, S, pmm::launch_pdl(pmm::rope_pairs_store_kernel<S>, dim3(T), dim3(256), 0, stream,
                                                static_cast<const S*>(q), ld_q, static_cast<const S*>(k), ld_k,
                                                static_cast<const S*>(v), ld_v, inv_freq, positions, seq_of,
                                                block_table, max_blocks, static_cast<S*>(pool), page_size,
                                                static_cast<S*>(q_out), H, G, d, dv, Dp, rot_dims, half_layout, q_bias,
-                                               k_bias, v_bias, q_norm_w, k_norm_w, norm_eps));
+                                               k_bias, v_bias, q_norm_w, k_norm_w, norm_eps, v_norm_eps));
   return pmm::launch_status();
 }

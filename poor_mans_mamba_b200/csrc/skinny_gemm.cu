@@ -58,6 +58,7 @@ struct SkinnyArgs {
   float* h_out;        // RESIDUAL target [M, N]
   float* y32;          // STORE_F32: y32[m, n] = y_scale * y
   float y_scale;
+  float y_cap;         // > 0: y32 = y_cap * tanh(y_scale * y / y_cap)
 };
 
 __device__ __forceinline__ void sg_cp16(void* smem, const void* gmem, bool pred) {
@@ -398,7 +399,8 @@ __device__ void SkinnyBlock<MT, MODE>::finish_tile(float (&acc)[MT][4], int n0) 
             const float inv = pr.h_in ? sInv[m] : 1.f;  // the row's norm factor (norm prologue)
             args.y[static_cast<size_t>(m) * args.ldy + n] = __float2bfloat16_rn(acc[nt][e] * inv);
           } else if (MODE == kSgStoreF32) {
-            args.y32[static_cast<size_t>(m) * args.ldy + n] = args.y_scale * acc[nt][e];
+            args.y32[static_cast<size_t>(m) * args.ldy + n] =
+                args.y_cap > 0.f ? args.y_cap * tanhf(args.y_scale * acc[nt][e] / args.y_cap) : args.y_scale * acc[nt][e];
           } else {
             atomicAdd(args.h_out + static_cast<size_t>(m) * args.N + n, pr.scale * acc[nt][e]);
           }
@@ -617,10 +619,10 @@ PMM_EXPORT int pmm_skinny_gemm(int mode, int M, int N, const void* x0, long long
   }
 }
 
-// y32[M, ldy] (float32) = scale * (x[M, K] W[N, K]^T) for up to 64 rows of bfloat16 activations: the
+// y32[M, ldy] (float32) = scale * (x[M, K] W[N, K]^T) (cap > 0: cap * tanh(that / cap)) for up to 64 rows of bfloat16 activations: the
 // output head of steps that ask for few rows of logits.
 PMM_EXPORT int pmm_skinny_gemm_f32out(int M, int N, const void* x, long long ldx, const void* w, int K, float scale,
-                                      float* y32, long long ldy, cudaStream_t stream) {
+                                      float cap, float* y32, long long ldy, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (M > 64 || K <= 0 || K % 8 || !x || !w || !y32) return PMM_ERR_BAD_ARGUMENT;
   pmm::SkinnyArgs a{};
@@ -632,6 +634,7 @@ PMM_EXPORT int pmm_skinny_gemm_f32out(int M, int N, const void* x, long long ldx
   a.ldy = ldy;
   a.y32 = y32;
   a.y_scale = scale;
+  a.y_cap = cap;
   return pmm::dispatch_skinny<pmm::kSgStoreF32>(a, K, stream);
 }
 

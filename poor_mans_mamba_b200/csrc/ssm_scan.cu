@@ -25,18 +25,6 @@ constexpr int kScanTpr = 8;     // threads per state row
 // over the state are double, so that a long portion does not lose the small increments of a slowly
 // decaying state to rounding (measured on a 1,100-token prompt whose gated norm divides by a small
 // root mean square: 5e-5 of the logits' spread with a float walk, 3e-6 with this one).
-template <typename ACC>
-__device__ __forceinline__ ACC scan_softplus(ACC v);
-template <>
-__device__ __forceinline__ float scan_softplus<float>(float v) { return softplus_f(v); }
-template <>
-__device__ __forceinline__ double scan_softplus<double>(double v) {
-  if (v > 40.0) return v;
-  return log1p(exp(v));
-}
-__device__ __forceinline__ float scan_exp(float v) { return expf(v); }
-__device__ __forceinline__ double scan_exp(double v) { return exp(v); }
-
 template <typename S, int NPT, typename ACC>
 __global__ void __launch_bounds__(kScanRows* kScanTpr)
     ssm_scan_seq_kernel(const S* __restrict__ xbc, int ld_xbc, const S* __restrict__ dt_raw,

@@ -4,7 +4,7 @@ order in which the layers run, final norm and output head.
 The forward pass is the same for every architecture:
   h = multiplier * E[tokens]                       (float32 residual stream; then the embedding's norm, if any)
   for (layer, cache_of) in order: layers[layer](h, cache of cache_of)
-  logits = (norm(h)[wanted rows] @ W_head^T) * head_multiplier       (float32)
+  logits = (norm(h)[wanted rows] @ W_head^T) * head_multiplier       (float32; then the softcap, if any)
 (reference src/runtime/runner/falconh1_runner.cpp:129-228, which keeps the last row only).
 """
 from __future__ import annotations
@@ -57,6 +57,7 @@ class Model:
         self.head: Optional[Tensor] = None
         self.dtype: Optional[torch.dtype] = None
         self.device: Optional[torch.device] = None
+        self._second_stream_buffer = any(getattr(l, "folds_across_rows", lambda: False)() for l in self.layers)
         self._branch_buffers = max(l.branch_buffers_needed() for l in self.layers) if self.layers else 1
 
     # ------------------------------------------------------------------ tensors
@@ -145,8 +146,9 @@ class Model:
             K.embed(h, self.embedding, ctx.tokens, self.spec.embedding_multiplier, norm_w, norm_eps)
         else:
             K.embed(h, self.embedding, ctx.tokens, self.spec.embedding_multiplier)
-        stream = ResidualStream(h, ctx, self._branch_buffers, lanes=self.spec.residual_lanes)
-        if self.reentry is not None:
+        stream = ResidualStream(h, ctx, self._branch_buffers, lanes=self.spec.residual_lanes,
+                                second_buffer=self._second_stream_buffer)
+        if self.reentry is not None and self.reentry.reads_embedding:
             stream.reentry = ws.alloc((T, 2 * D), ctx.dtype)
             K.cast_rows(h, [], stream.reentry[:, D:])
         order = self.spec.order
@@ -163,7 +165,7 @@ class Model:
                 self._join(ctx, h.device)
             if call.enters:
                 self._join(ctx, h.device)
-                self.reentry.forward(stream, ctx)
+                self.reentry.enter(stream, ctx, call.pass_index)
             layer.forward(stream, ctx, caches[call.cache_of])
         ctx.fetch_ahead = None
         self._join(ctx, h.device)
@@ -225,18 +227,22 @@ class Model:
         n_rows, V = normed.shape[0], self.vocab_size
         ws = ctx.workspace
         logits = ws.alloc((n_rows, V), torch.float32)
-        mult = self.spec.head_multiplier
+        mult, cap = self.spec.head_multiplier, self.spec.logit_softcap
         if normed.dtype == torch.float32:
             K.linear(normed, self.head, logits)
-            if mult != 1.0:
+            if cap > 0.0:
+                K.softcap_f32_(logits, mult, cap)
+            elif mult != 1.0:
                 K.scale_f32_(logits, mult)
         elif _SKINNY_HEAD and self._head_row_group(n_rows) > 0:
             # the table is read at memory speed by this repository's weight-streaming product
-            # (float32 out, multiplier in the epilogue), once per group of rows that fits its shared memory
+            # (float32 out, multiplier and softcap in the epilogue), once per group of rows that fits its shared memory
             group = self._head_row_group(n_rows)
             for r0 in range(0, n_rows, group):
-                K.skinny_linear_f32(normed[r0:r0 + group], self.head, logits[r0:r0 + group], mult)
+                K.skinny_linear_f32(normed[r0:r0 + group], self.head, logits[r0:r0 + group], mult, cap)
         else:
             low = None if K.mm_has_f32_out() else ws.alloc((n_rows, V), normed.dtype)
-            K.linear_f32_out(normed, self.head, logits, low, mult)
+            K.linear_f32_out(normed, self.head, logits, low, mult if cap <= 0.0 else 1.0)
+            if cap > 0.0:
+                K.softcap_f32_(logits, mult, cap)
         return logits

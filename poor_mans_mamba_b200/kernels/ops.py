@@ -33,6 +33,16 @@ _SIGNATURES = {
                                  c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
     "pmm_add_rmsnorm": [c_void_p, c_void_p, c_float, c_void_p, c_float, c_void_p, c_float, c_void_p,
                         c_void_p, c_int, c_int, c_int, c_void_p],
+    "pmm_fold_norm": [c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_float, c_void_p, c_void_p, c_float, c_int, c_void_p,
+                      c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int,
+                      c_void_p],
+    "pmm_softcap_f32": [c_void_p, c_float, c_float, c_longlong, c_void_p],
+    "pmm_selective_scan_channels": [c_int],
+    "pmm_selective_scan": [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_int, c_void_p, c_longlong,
+                           c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+                           c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
+    "pmm_selective_step": [c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p, c_longlong,
+                           c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
     "pmm_scale_f32": [c_void_p, c_float, c_longlong, c_void_p],
     "pmm_cast_scale": [c_void_p, c_void_p, c_float, c_longlong, c_int, c_void_p],
     "pmm_conv1d_fwd": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
@@ -71,7 +81,8 @@ _SIGNATURES = {
                        c_void_p],
     "pmm_rope_pairs_store": [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_void_p,
                              c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                             c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_int, c_void_p],
+                             c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_float, c_int,
+                             c_void_p],
     "pmm_delta_scan": [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong,
                        c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
                        c_int, c_int, c_int, c_float, c_float, c_int, c_void_p],
@@ -105,7 +116,7 @@ _SIGNATURES = {
     "pmm_skinny_gemm": [c_int, c_int, c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_float, c_void_p, c_int,
                         c_float, c_void_p, c_longlong, c_void_p, c_int, c_float, c_void_p, c_longlong, c_void_p,
                         c_int, c_void_p],
-    "pmm_skinny_gemm_f32out": [c_int, c_int, c_void_p, c_longlong, c_void_p, c_int, c_float, c_void_p, c_longlong,
+    "pmm_skinny_gemm_f32out": [c_int, c_int, c_void_p, c_longlong, c_void_p, c_int, c_float, c_float, c_void_p, c_longlong,
                                c_void_p],
     "pmm_skinny_tc_supported": [c_int, c_int, c_int, c_int, c_int, c_longlong, c_longlong, c_longlong],
     "pmm_skinny_tc": [c_int, c_int, c_int, c_void_p, c_longlong, c_void_p, c_int, c_float, c_void_p, c_longlong,
@@ -128,13 +139,13 @@ _SIGNATURES = {
     "pmm_moe_plan": [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p],
     "pmm_moe_tile_rows": [c_int],
     "pmm_moe_gemm": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                     c_int, c_float, c_float, c_float, c_void_p, c_int, c_int, c_void_p],
+                     c_int, c_float, c_float, c_float, c_void_p, c_void_p, c_int, c_int, c_void_p],
     "pmm_moe_combine": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
     "pmm_moe_tc_tile_rows": [],
     "pmm_moe_tc_supported": [c_int, c_int, c_longlong],
     "pmm_moe_gather_rows": [c_void_p, c_longlong, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p],
     "pmm_moe_tc_gemm": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                        c_float, c_float, c_float, c_void_p, c_void_p, c_void_p],
+                        c_float, c_float, c_float, c_void_p, c_void_p, c_void_p, c_void_p],
     "pmm_latent_norm_store": [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_void_p, c_float, c_void_p, c_void_p,
                               c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
                               c_int, c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_void_p],
@@ -544,6 +555,72 @@ def scale_f32_(x: Tensor, s: float) -> None:
     _call("pmm_scale_f32", x.data_ptr(), float(s), x.numel(), _stream())
 
 
+def softcap_f32_(x: Tensor, s: float, cap: float) -> None:
+    """x <- cap * tanh(s * x / cap)."""
+    _cuda(x)
+    if not (x.dtype == torch.float32 and x.is_contiguous() and cap > 0.0):
+        raise KernelError("softcap_f32_: contiguous float32 and a positive cap")
+    _call("pmm_softcap_f32", x.data_ptr(), float(s), float(cap), x.numel(), _stream())
+
+
+def fold_norm(h: Tensor, h_out: Optional[Tensor], branches: Sequence[Tuple[Tensor, float]], vector: Optional[Tensor],
+              weight: Optional[Tensor], eps: float, groups: int, out: Optional[Tensor], rows: Optional[Tensor] = None,
+              conv: Optional[Tensor] = None, window: Optional[Tensor] = None, cu: Optional[Tensor] = None,
+              slots: Optional[Tensor] = None, seq_of: Optional[Tensor] = None, n_seq: int = 0,
+              one_token: bool = False) -> None:
+    """v = h + s0*b0 + s1*b1 + vector (float32 [D], every row);  h_out = v (rows is None);  out = v over the root mean
+    square of each of ``groups`` equal parts of the row, times ``weight`` (None: fold only).  With ``conv`` (tap-major
+    float32 [taps, D]) out is that norm n plus its causal convolution, n_t + sum_j conv[j] n_(t - taps + 1 + j), from and
+    into the requests' windows (float32 [slots, taps - 1, D], the last taps - 1 normed rows); h_out must then be another
+    buffer than h unless nothing waits or every sequence brings one token (``one_token``).  With ``rows`` h is left as
+    it is and out[r] comes from row rows[r]."""
+    items = list(branches)
+    _cuda(h, h_out, vector, weight, out, rows, conv, window, cu, slots, seq_of, *[b for b, _ in items])
+    T, D = h.shape
+    if len(items) > 2:
+        raise KernelError("fold_norm: at most two branches")
+    if not (h.dtype == torch.float32 and h.is_contiguous()):
+        raise KernelError("fold_norm: the residual stream must be contiguous float32 [T, D]")
+    if h_out is not None and not (h_out.dtype == torch.float32 and h_out.is_contiguous() and h_out.shape == h.shape):
+        raise KernelError("fold_norm: h_out must match h")
+    dtype = None if out is None else _dt(out)
+    for b, _ in items:
+        if not (b.shape == h.shape and b.is_contiguous() and dtype in (None, _dt(b))):
+            raise KernelError("fold_norm: branches must be contiguous [T, D] of out's type")
+        dtype = _dt(b)
+    if not (groups >= 1 and D % groups == 0):
+        raise KernelError("fold_norm: the groups must divide the width")
+    _f32vec(vector, D, "fold_norm: vector")
+    _f32vec(weight, D, "fold_norm: weight")
+    R = T
+    if rows is not None:
+        _i32(rows, "fold_norm: rows")
+        R = rows.numel()
+    if (weight is None) != (out is None) or (out is not None and not (out.shape == (R, D) and out.is_contiguous())):
+        raise KernelError("fold_norm: a norm needs its weight and a contiguous out [rows, D]")
+    if out is None and not items and vector is None:
+        return
+    taps = 0
+    if conv is not None:
+        taps = conv.shape[0]
+        if not (rows is None and conv.dtype == torch.float32 and conv.is_contiguous() and conv.shape == (taps, D)):
+            raise KernelError("fold_norm: conv must be contiguous float32 [taps, D], for all rows of the step")
+        if taps > 1:
+            if not (window is not None and window.dtype == torch.float32 and window.is_contiguous() and window.dim() == 3
+                    and tuple(window.shape[1:]) == (taps - 1, D)):
+                raise KernelError("fold_norm: window must be float32 [slots, taps - 1, D]")
+            for t, what in ((cu, "cu"), (slots, "slots"), (seq_of, "seq_of")):
+                if t is None:
+                    raise KernelError(f"fold_norm: a convolution needs {what}")
+                _i32(t, f"fold_norm: {what}")
+            if not (cu.numel() == n_seq + 1 and slots.numel() == n_seq and seq_of.numel() == T and (not one_token or n_seq == T)):
+                raise KernelError("fold_norm: cu [n_seq + 1], slots [n_seq], seq_of [T]")
+    (a, sa), (b, sb) = (items + [(None, 0.0), (None, 0.0)])[:2]
+    _call("pmm_fold_norm", h.data_ptr(), _ptr(h_out), _ptr(a), float(sa), _ptr(b), float(sb), _ptr(vector), _ptr(weight),
+          float(eps), int(groups), _ptr(conv), taps, _ptr(window), _ptr(cu), _ptr(slots), _ptr(seq_of), int(n_seq),
+          int(bool(one_token)), _ptr(rows), _ptr(out), R, D, 0 if dtype is None else dtype, _stream())
+
+
 def cast_scale(out: Tensor, src: Tensor, s: float) -> None:
     _cuda(out, src)
     if not (out.dtype == torch.float32 and out.is_contiguous() and src.is_contiguous()
@@ -789,6 +866,98 @@ def ssm_scan_tc(xbc: Tensor, dt_raw: Tensor, dt_scale: float, dt_shift: Tensor, 
           chunk_state, chunk_decay, chunk_dt, start_state, len(new_lens), n_chunks, H, P, N, n_groups, zp, ld_z, zs, zb,
           int(bool(skip_single)), n_multi if skip_single else 0,
           _tc_status(xbc.device).data_ptr(), _stream())
+
+
+# ----------------------------------------------------------------------------- selective scan
+SELECTIVE_MAX_STATE = 256
+_SELECTIVE_FULL_WARPS = 1200  # warps of one walk (4 a block) from which the GPU is busy without chunks
+_SELECTIVE_MIN_CHUNK = 64
+
+
+def selective_scan_plan(new_lens: Sequence[int], inner: int, d_state: int, dtype: torch.dtype) -> Tuple[int, int]:
+    """(tokens per chunk, upper bound of chunks) for a step's portions.  One walk per channel where the channels and
+    sequences fill the GPU, or where two chunks would (a chunked walk makes every exponential twice); else as many
+    chunks as fill it.  Float32 walks are never cut."""
+    longest = max(new_lens)
+    chunk = longest
+    if dtype == torch.bfloat16 and longest > _SELECTIVE_MIN_CHUNK:
+        warps = 4 * -(-inner // selective_scan_channels(d_state)) * sum(1 for n in new_lens if n > longest // 2)
+        want = _SELECTIVE_FULL_WARPS // warps
+        if want >= 3:
+            chunk = max(_SELECTIVE_MIN_CHUNK, (-(-longest // want) + 15) // 16 * 16)
+    return chunk, sum(-(-n // chunk) for n in new_lens)
+
+
+def selective_scan_channels(d_state: int) -> int:
+    """Channels of one block of the walk."""
+    n = int(_fn("pmm_selective_scan_channels")(int(d_state)))
+    if n <= 0:
+        raise KernelError(f"selective scan: state sizes 1..{SELECTIVE_MAX_STATE}, got {d_state}")
+    return n
+
+
+def _selective_common(x: Tensor, low: Tensor, z: Tensor, bias: Tensor, a_log: Tensor, d_skip: Tensor, state: Tensor,
+                      slots: Tensor, off_b: int, off_c: int, out: Tensor, what: str) -> Tuple[int, int]:
+    T, I = x.shape
+    if not (state.dtype == torch.float32 and state.dim() == 3 and state.is_contiguous() and state.shape[1] == I):
+        raise KernelError(f"{what}: state must be contiguous float32 [slots, I, N]")
+    N = state.shape[2]
+    if not (1 <= N <= SELECTIVE_MAX_STATE):
+        raise KernelError(f"{what}: state sizes 1..{SELECTIVE_MAX_STATE}, got {N}")
+    if not (z.shape == (T, I) and out.shape == (T, I) and out.is_contiguous() and x.dtype == z.dtype == low.dtype == out.dtype
+            and low.shape[0] == T and 0 <= off_b and off_b + N <= low.shape[1] and 0 <= off_c and off_c + N <= low.shape[1]):
+        raise KernelError(f"{what}: x, z and out [T, I], low [T, ...] with B and C inside its columns, of one type")
+    _f32vec(bias, I, f"{what}: bias")
+    _f32vec(d_skip, I, f"{what}: D")
+    _f32vec(a_log, I * N, f"{what}: A_log")
+    _i32(slots, f"{what}: slots")
+    return I, N
+
+
+def selective_scan(x: Tensor, raw: Tensor, low: Tensor, off_b: int, off_c: int, z: Tensor, bias: Tensor, a_log: Tensor,
+                   d_skip: Tensor, state: Tensor, cu: Tensor, slots: Tensor, n_seq: int, plan: Tuple[int, int],
+                   scratch: Optional[Tensor], out: Tensor) -> None:
+    """The selective scan with a decay per channel and state entry over the step's portions, from and into state
+    [slots, I, N]:  dt = softplus(raw + bias);  S <- exp(-dt exp(A_log)) S + dt x B;  out = (S . C + D x) * silu(z).
+    ``low``: B in the N columns from off_b, C from off_c.  ``plan``: selective_scan_plan; where it has more chunks than
+    sequences, ``scratch`` holds float32 [chunks * I * (N + 1)]."""
+    _cuda(x, raw, low, z, bias, a_log, d_skip, state, cu, slots, out, scratch)
+    I, N = _selective_common(x, low, z, bias, a_log, d_skip, state, slots, off_b, off_c, out, "selective_scan")
+    if not (raw.shape == x.shape and raw.dtype == x.dtype):
+        raise KernelError("selective_scan: raw step sizes [T, I] of x's type")
+    _i32(cu, "selective_scan: cu")
+    chunk, n_chunks = plan
+    multi = n_chunks > n_seq
+    cs = cd = None
+    if multi:
+        if not (scratch is not None and scratch.dtype == torch.float32 and scratch.is_contiguous()
+                and scratch.numel() >= n_chunks * I * (N + 1)):
+            raise KernelError("selective_scan: scratch of chunks * I * (N + 1) floats")
+        cs = scratch.data_ptr()
+        cd = cs + 4 * n_chunks * I * N
+    _call("pmm_selective_scan", x.data_ptr(), _rows_view(x, "selective_scan: x"), raw.data_ptr(), _rows_view(raw, "selective_scan: raw"),
+          low.data_ptr(), _rows_view(low, "selective_scan: low"), int(off_b), int(off_c), z.data_ptr(),
+          _rows_view(z, "selective_scan: z"), bias.data_ptr(), a_log.data_ptr(), d_skip.data_ptr(), state.data_ptr(), cs, cd,
+          cu.data_ptr(), slots.data_ptr(), out.data_ptr(), int(n_seq), int(n_chunks), int(chunk), int(multi), I, N, _dt(x),
+          _stream())
+    if multi:
+        global launch_count
+        launch_count += 2  # chunk states, their pass, the walk
+
+
+def selective_step(x: Tensor, low: Tensor, rank: int, off_b: int, off_c: int, w_dt: Tensor, z: Tensor, bias: Tensor,
+                   a_log: Tensor, d_skip: Tensor, state: Tensor, slots: Tensor, out: Tensor) -> None:
+    """selective_scan for one token per sequence, with the raw step sizes made in the same launch: raw = low[:, :rank] @
+    w_dt^T, w_dt [I, rank]."""
+    _cuda(x, low, w_dt, z, bias, a_log, d_skip, state, slots, out)
+    I, N = _selective_common(x, low, z, bias, a_log, d_skip, state, slots, off_b, off_c, out, "selective_step")
+    if not (w_dt.shape == (I, rank) and w_dt.is_contiguous() and w_dt.dtype == x.dtype and rank <= low.shape[1]
+            and slots.numel() == x.shape[0]):
+        raise KernelError("selective_step: w_dt contiguous [I, rank] of x's type, one slot per token")
+    _call("pmm_selective_step", x.data_ptr(), _rows_view(x, "selective_step: x"), low.data_ptr(), _rows_view(low, "selective_step: low"),
+          int(rank), int(off_b), int(off_c), w_dt.data_ptr(), z.data_ptr(), _rows_view(z, "selective_step: z"), bias.data_ptr(),
+          a_log.data_ptr(), d_skip.data_ptr(), state.data_ptr(), slots.data_ptr(), out.data_ptr(), x.shape[0], I, N, _dt(x),
+          _stream())
 
 
 def gated_norm(y: Tensor, z_raw: Tensor, z_scale: float, z_bias: Optional[Tensor],
@@ -1174,9 +1343,10 @@ def skinny_linear(x: Tensor, weight: Tensor, out: Tensor) -> None:
           1.0, None, 0, None, 0, 0.0, out.data_ptr(), out.stride(0), None, 1, _stream())
 
 
-def skinny_linear_f32(x: Tensor, weight: Tensor, out: Tensor, scale: float) -> None:
+def skinny_linear_f32(x: Tensor, weight: Tensor, out: Tensor, scale: float, cap: float = 0.0) -> None:
     """out[M, N] (float32) = scale * (x @ weight^T) for M <= 64 rows of bfloat16 activations: the
-    output head of a step that asks for few rows of logits (the table is streamed once)."""
+    output head of a step that asks for few rows of logits (the table is streamed once).  ``cap`` > 0:
+    out = cap * tanh(that / cap)."""
     _cuda(x, weight, out)
     M, K = x.shape
     _skinny_check(M, weight, K, "skinny_linear_f32")
@@ -1186,7 +1356,7 @@ def skinny_linear_f32(x: Tensor, weight: Tensor, out: Tensor, scale: float) -> N
     N = weight.shape[0]
     if not (out.dtype == torch.float32 and out.shape == (M, N) and out.stride(1) == 1):
         raise KernelError("skinny_linear_f32: out [M, N] float32")
-    _call("pmm_skinny_gemm_f32out", M, N, x.data_ptr(), x.stride(0), weight.data_ptr(), K, float(scale),
+    _call("pmm_skinny_gemm_f32out", M, N, x.data_ptr(), x.stride(0), weight.data_ptr(), K, float(scale), float(cap),
           out.data_ptr(), out.stride(0), _stream())
 
 
@@ -1769,7 +1939,8 @@ def moe_route(x: Tensor, router_w: Tensor, router_b: Optional[Tensor], top: int,
     ``scored``: s = sigmoid(z); the ``top`` largest of s + correction among the experts of the ``keep`` groups (of
     ``groups`` equal groups of neighbours) whose two largest s + correction sum highest; weights the chosen s over
     their sum, times ``scale``.  ``scored`` "softmax": s = softmax(z) over all experts, a group counts by its largest
-    s + correction, and the weights are the chosen s times ``scale`` (not divided by their sum).  ``gate_w`` [D] float32: gate_out[t] = sigmoid(x[t] . gate_w) as well."""
+    s + correction, and the weights are the chosen s times ``scale`` (not divided by their sum).  ``scored`` "sigmoid": as
+    plain ``scored``, with the chosen s times ``scale`` as they are for weights.  ``gate_w`` [D] float32: gate_out[t] = sigmoid(x[t] . gate_w) as well."""
     _cuda(x, router_w, router_b, ids, weights, correction, gate_w, gate_out)
     T, D = x.shape
     E = router_w.shape[0]
@@ -1788,10 +1959,11 @@ def moe_route(x: Tensor, router_w: Tensor, router_b: Optional[Tensor], top: int,
         if not (gate_out is not None and gate_out.dtype == torch.float32 and gate_out.is_contiguous() and gate_out.numel() == T):
             raise KernelError("moe_route: gate_out must be contiguous float32 [T]")
     _call("pmm_moe_route", x.data_ptr(), _rows_view(x, "moe_route"), router_w.data_ptr(), _ptr(router_b), ids.data_ptr(),
-          weights.data_ptr(), T, D, E, int(top), 2 if scored == "softmax" else int(bool(scored)), _ptr(correction), int(groups), int(keep), float(scale),
+          weights.data_ptr(), T, D, E, int(top), _ROUTE_MODES[scored], _ptr(correction), int(groups), int(keep), float(scale),
           _ptr(gate_w), _ptr(gate_out) if gate_w is not None else None, _dt(x), _stream())
 
 
+_ROUTE_MODES = {False: 0, True: 1, "softmax": 2, "sigmoid": 3}
 _MOE_FORMS = {"float": 0, "mma": 1, "mma_few": 2}
 
 
@@ -1836,14 +2008,23 @@ def moe_gather_rows(x: Tensor, perm: Tensor, top: int, out: Tensor) -> None:
           out.data_ptr(), Kd, _stream())
 
 
+def _row_weights(w: Optional[Tensor], A: int, gated: bool) -> None:
+    if w is not None and not (gated and w.dtype == torch.float32 and w.is_contiguous() and w.numel() == A):
+        raise KernelError("grouped product: row weights are float32, one per pair, of a gated up product")
+
+
 def moe_tc_gemm(a: Tensor, w: Tensor, perm: Tensor, offsets: Tensor, tile_start: Tensor, up: bool, out: Tensor,
-                limit: float = 0.0, alpha: float = 0.0, shift: float = 0.0, ungated: bool = False) -> None:
+                limit: float = 0.0, alpha: float = 0.0, shift: float = 0.0, ungated: bool = False,
+                row_weights: Optional[Tensor] = None) -> None:
     """The grouped product on the fifth-generation tensor cores.  a [pairs, K]: rows in the order of the sorted
     pairs (the gathered token rows, or the activation); w [E, N (2N), K]; the plan made for "tcgen05" row tiles.
     ``up``: out = act [pairs, N] with the clamped gated activation; else out = y [pairs, N] in the order of the
-    pairs (both bfloat16).  ``up`` and ``ungated``: w [E, N, K], out = act [pairs, N] = max(a W^T, 0)^2."""
-    _cuda(a, w, perm, offsets, tile_start, out)
+    pairs (both bfloat16).  ``up`` and ``ungated``: w [E, N, K], out = act [pairs, N] = max(a W^T, 0)^2.
+    ``row_weights`` (gated ``up`` only; float32, one per pair in the order of the pairs): the pair's input is its weight times
+    its row."""
+    _cuda(a, w, perm, offsets, tile_start, out, row_weights)
     A, Kd = a.shape
+    _row_weights(row_weights, A, up and not ungated)
     E, N = w.shape[0], out.shape[1]
     if ungated and not up:
         raise KernelError("moe_tc_gemm: only an up product is gated or ungated")
@@ -1853,7 +2034,7 @@ def moe_tc_gemm(a: Tensor, w: Tensor, perm: Tensor, offsets: Tensor, tile_start:
         raise KernelError("moe_tc_gemm: operands outside what the kernel takes")
     _call("pmm_moe_tc_gemm", a.data_ptr(), a.stride(0), w.data_ptr(), perm.data_ptr(), offsets.data_ptr(),
           tile_start.data_ptr(), A, E, Kd, N, (2 if ungated else 1) if up else 0, float(limit), float(alpha), float(shift),
-          out.data_ptr(), _tc_status(a.device).data_ptr(), _stream())
+          _ptr(row_weights), out.data_ptr(), _tc_status(a.device).data_ptr(), _stream())
 
 
 def moe_gemm_tc_ok(a: Tensor, w: Tensor) -> bool:
@@ -1863,13 +2044,15 @@ def moe_gemm_tc_ok(a: Tensor, w: Tensor) -> bool:
 
 
 def moe_gemm(a: Tensor, w: Tensor, perm: Tensor, offsets: Tensor, tile_start: Tensor, top: int, up: bool, out: Tensor,
-             form: str, limit: float = 0.0, alpha: float = 0.0, shift: float = 0.0, ungated: bool = False) -> None:
+             form: str, limit: float = 0.0, alpha: float = 0.0, shift: float = 0.0, ungated: bool = False,
+             row_weights: Optional[Tensor] = None) -> None:
     """Grouped product over the rows of a plan.  ``up``: a = x [T, K], w [E, 2N, K] ([gate | up] rows of
     every expert), out = act [T*top, N] in the storage type, with the clamped gated activation.  Else:
     a = act [T*top, K], w [E, N, K], out = y [T*top, N] in the order of the pairs.  ``up`` and ``ungated``: w [E, N, K],
-    out = act [T*top, N] = max(x W^T, 0)^2."""
-    _cuda(a, w, perm, offsets, tile_start, out)
+    out = act [T*top, N] = max(x W^T, 0)^2.  ``row_weights``: as in moe_tc_gemm."""
+    _cuda(a, w, perm, offsets, tile_start, out, row_weights)
     A = perm.numel()
+    _row_weights(row_weights, A, up and not ungated)
     E = w.shape[0]
     K = a.shape[1]
     N = out.shape[1]
@@ -1886,24 +2069,26 @@ def moe_gemm(a: Tensor, w: Tensor, perm: Tensor, offsets: Tensor, tile_start: Te
         raise KernelError("moe_gemm: the tensor-core forms need bfloat16, K a multiple of 8 and 16-byte aligned rows")
     _call("pmm_moe_gemm", a.data_ptr(), _rows_view(a, "moe_gemm"), w.data_ptr(), perm.data_ptr(), offsets.data_ptr(),
           tile_start.data_ptr(), A, E, int(top), K, N, (2 if ungated else 1) if up else 0, float(limit), float(alpha),
-          float(shift), out.data_ptr(), tensor_cores, _dt(a), _stream())
+          float(shift), _ptr(row_weights), out.data_ptr(), tensor_cores, _dt(a), _stream())
 
 
-def moe_combine(y: Tensor, weights: Tensor, shared: Optional[Tensor], out: Tensor,
+def moe_combine(y: Tensor, weights: Optional[Tensor], shared: Optional[Tensor], out: Tensor,
                 shared_gate: Optional[Tensor] = None) -> None:
-    """out[t] = sum_j weights[t, j] * y[t*top + j] (+ shared[t], times shared_gate[t] where given)."""
+    """out[t] = sum_j weights[t, j] * y[t*top + j] (+ shared[t], times shared_gate[t] where given).  ``weights`` None:
+    every weight is 1."""
     _cuda(y, weights, shared, out, shared_gate)
-    T, top = weights.shape
-    D = out.shape[1]
+    T, D = out.shape
+    top = y.shape[0] // T if weights is None else weights.shape[1]
     if not (y.shape == (T * top, D) and y.dtype == out.dtype and y.is_contiguous() and out.shape == (T, D)
-            and out.is_contiguous() and weights.dtype == torch.float32 and weights.is_contiguous()):
+            and out.is_contiguous() and (weights is None or (weights.dtype == torch.float32 and weights.is_contiguous()
+                                                             and weights.shape == (T, top)))):
         raise KernelError("moe_combine: y [T*top, D] of out's type, weights [T, top] float32, out contiguous [T, D]")
     if shared is not None and not (shared.shape == (T, D) and shared.is_contiguous() and shared.dtype == out.dtype):
         raise KernelError("moe_combine: shared must be contiguous [T, D] of out's type")
     if shared_gate is not None and not (shared is not None and shared_gate.dtype == torch.float32
                                         and shared_gate.is_contiguous() and shared_gate.numel() == T):
         raise KernelError("moe_combine: shared_gate must be contiguous float32 [T] beside a shared output")
-    _call("pmm_moe_combine", y.data_ptr(), weights.data_ptr(), _ptr(shared), _ptr(shared_gate), out.data_ptr(), T, D, top,
+    _call("pmm_moe_combine", y.data_ptr(), _ptr(weights), _ptr(shared), _ptr(shared_gate), out.data_ptr(), T, D, top,
           _dt(out), _stream())
 
 
@@ -2062,13 +2247,14 @@ def rope_pairs_store(q: Tensor, k: Tensor, v: Tensor, inv_freq: Optional[Tensor]
                      seq_of: Tensor, block_table: Tensor, pool: Tensor, q_out: Tensor, n_heads: int,
                      n_kv_heads: int, dim: int, vdim: int, padded_dim: int, half_layout: bool = False,
                      biases: Optional[Tuple[Tensor, Tensor, Tensor]] = None,
-                     qk_norm: Optional[Tuple[Tensor, Tensor, float]] = None) -> None:
+                     qk_norm: Optional[Tuple[Tensor, Tensor, float]] = None, v_norm_eps: Optional[float] = None) -> None:
     """Rotates pairs among the first ``rot_dims`` entries of every query and key head (neighbours
     (2i, 2i+1), or with ``half_layout`` entries (i, i + rot_dims/2)), writes queries to q_out [T, H*Dp]
     and keys and values into their pages [pages, 2, page, G*Dp], every head padded with zeros to Dp =
     ``padded_dim`` entries.  ``biases``: float vectors added to q, k and v as they are read.  ``qk_norm`` (weight
     [H*d], weight [G*d], eps): before rotation the token's whole query projection, and its whole key projection, is
-    divided by its root mean square and multiplied by the weight (float); values are left as they are."""
+    divided by its root mean square and multiplied by the weight (float); values are left as they are.  ``v_norm_eps``:
+    every value head is divided by its own root mean square over its vdim entries (eps inside the root, float)."""
     _cuda(q, k, v, inv_freq, positions, seq_of, block_table, pool, q_out)
     qn = kn = None
     norm_eps = 0.0
@@ -2099,7 +2285,8 @@ def rope_pairs_store(q: Tensor, k: Tensor, v: Tensor, inv_freq: Optional[Tensor]
     _call("pmm_rope_pairs_store", q.data_ptr(), ld_q, k.data_ptr(), ld_k, v.data_ptr(), ld_v, _ptr(inv_freq),
           positions.data_ptr(), seq_of.data_ptr(), block_table.data_ptr(), block_table.shape[1], pool.data_ptr(),
           pool.shape[2], q_out.data_ptr(), T, n_heads, n_kv_heads, dim, vdim, padded_dim, int(rot_dims),
-          int(bool(half_layout)), _ptr(qb), _ptr(kb), _ptr(vb), _ptr(qn), _ptr(kn), float(norm_eps), _dt(q), _stream())
+          int(bool(half_layout)), _ptr(qb), _ptr(kb), _ptr(vb), _ptr(qn), _ptr(kn), float(norm_eps),
+          -1.0 if v_norm_eps is None else float(v_norm_eps), _dt(q), _stream())
 
 
 # ----------------------------------------------------------------------------- matrix-state recurrences

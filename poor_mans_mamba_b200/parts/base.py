@@ -144,6 +144,12 @@ class Norm(Part):
         other norm (it is then launched on its own through `forward`)."""
         return None
 
+    def group_prologue(self) -> Optional[Tuple[Tensor, float, int]]:
+        """(weight [D] float32, eps, groups) if this norm divides each of ``groups`` equal neighbouring parts of the
+        row by its own root mean square and multiplies by the weight (1: the plain RMS norm): the launch that folds
+        the stream can then also run the convolution of the sublayer's input.  None for any other norm."""
+        return None
+
 
 class PositionEncoding(Part):
     """Applied by a mixer to its queries and keys at absolute positions."""
@@ -236,13 +242,35 @@ class FeedForward(Part):
         return []
 
 
+class InputMap(Part):
+    """Stands between a sublayer's norm and the sublayer and may look at earlier tokens through state of its own:
+    forward(x, ctx, cache, out), x [T, D] the normed rows, out [T, D] (another buffer) what the sublayer reads."""
+
+    def state_specs(self) -> List[StateSpec]:
+        return []
+
+    def fused_conv(self, cache: "LayerCache") -> Optional[Tuple[Tensor, Optional[Tensor]]]:
+        """(taps [taps, D] tap-major float32, window [slots, taps - 1, D] or None) if this map is
+        x_t + sum_j taps[j] x_(t - taps + 1 + j): the launch that folds the stream and norms it can then run it too."""
+        return None
+
+    def forward(self, x: Tensor, ctx, cache: "LayerCache", out: Tensor) -> None:
+        raise NotImplementedError
+
+
 class StreamUpdate(Part):
     """Changes the residual stream in place at the end of a layer, reading nothing but the stream and the
     step's tokens (a per-token input, for instance): forward(stream, ctx), with ``stream`` the
-    ResidualStream, whose waiting branches the part folds in first."""
+    ResidualStream, whose waiting branches the part folds in first.  As a model's ``reentry`` part it runs
+    before a pass over a span of layers: `enter` with the pass's number."""
+    # Whether, as a reentry part, it reads the embedding's output of the step (see ModelSpec.reentry).
+    reads_embedding: bool = False
 
     def forward(self, stream, ctx) -> None:
         raise NotImplementedError
+
+    def enter(self, stream, ctx, pass_index: int) -> None:
+        self.forward(stream, ctx)
 
 
 # ----------------------------------------------------------------------------- specs (data)
@@ -273,10 +301,11 @@ class LayerSpec:
 class LayerCall:
     """One entry of the execution order: run ``layer`` on the cache of ``cache_of``
     (its own unless it reads another layer's).  ``enters``: the model's ``reentry`` part
-    changes the stream right before this call."""
+    changes the stream right before this call, which begins pass ``pass_index``."""
     layer: int
     cache_of: int
     enters: bool = False
+    pass_index: int = 0
 
 
 @dataclass(frozen=True)
@@ -293,12 +322,14 @@ class ModelSpec:
     eos_token_id: int = -1
     bos_token_id: int = 0
     # A stream update (`register_stream_update`) that runs before every call of the order with ``enters``.
-    # With one, the embedding's output is kept for the whole step (in the storage type, as the right half
+    # With one that ``reads_embedding``, the embedding's output is kept for the whole step (in the storage type, as the right half
     # of ``ResidualStream.reentry`` [T, 2D]; the left half is the part's scratch).
     reentry: Optional[PartSpec] = None
     # A norm applied to the embedding's output before the first layer (in float, inside the embedding launch;
     # an RMS norm: one whose `rms_prologue` answers).
     embedding_norm: Optional[PartSpec] = None
+    # > 0: logits <- logit_softcap * tanh(logits / logit_softcap), after the head's multiplier.
+    logit_softcap: float = 0.0
     # None: one residual stream [T, D].  n >= 1: the residual state is n lanes [n, T, D], all equal to
     # the embedding's output at the start and summed before the final norm (arrangements that mix
     # lanes, such as ``hyper_prenorm``, read and write them through the ResidualStream)
@@ -308,6 +339,7 @@ class ModelSpec:
 # ----------------------------------------------------------------------------- registries
 _REGISTRIES: Dict[str, Dict[str, Callable[..., Part]]] = {
     "mixer": {}, "feed_forward": {}, "norm": {}, "position_encoding": {}, "arrangement": {}, "stream_update": {},
+    "input_map": {},
 }
 
 
@@ -340,6 +372,10 @@ def register_arrangement(kind: str, factory: Callable[..., Any]) -> None:
 
 def register_stream_update(kind: str, factory: Callable[..., "StreamUpdate"]) -> None:
     _register("stream_update", kind, factory)
+
+
+def register_input_map(kind: str, factory: Callable[..., "InputMap"]) -> None:
+    _register("input_map", kind, factory)
 
 
 def build_part(family: str, spec: PartSpec, **extra: Any) -> Any:

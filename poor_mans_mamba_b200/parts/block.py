@@ -19,7 +19,7 @@ import torch
 
 from ..kernels import ops as K
 from . import branches, streaming
-from .base import (FeedForward, LayerCache, LayerSpec, Mixer, Norm, Part, PartSpec, StateSpec,
+from .base import (FeedForward, InputMap, LayerCache, LayerSpec, Mixer, Norm, Part, PartSpec, StateSpec,
                    build_part, register_arrangement)
 from .norm import fold_branches
 
@@ -36,15 +36,21 @@ _JOINED_OUTPUTS = os.environ.get("PMM_JOINED_OUTPUTS", "1") == "1"
 
 def prenorm_layer(prefix: str, mixer_norm: PartSpec, mixers, ffn_norm: Optional[PartSpec] = None,
                   ffn: Optional[PartSpec] = None, mixer_post_norm: Optional[PartSpec] = None,
-                  ffn_post_norm: Optional[PartSpec] = None) -> LayerSpec:
+                  ffn_post_norm: Optional[PartSpec] = None, mixer_input: Optional[PartSpec] = None,
+                  ffn_input: Optional[PartSpec] = None) -> LayerSpec:
     """The LayerSpec of a ``parallel_prenorm`` layer: norm -> parallel mixers -> norm -> feed-forward.
     With post norms each sublayer's result is normed once more before it joins the stream:
-    x <- x + post(sum of the scaled mixers' outputs), x <- x + post(feed-forward)."""
+    x <- x + post(sum of the scaled mixers' outputs), x <- x + post(feed-forward).  With input maps what a
+    sublayer reads passes one more part behind its norm (`register_input_map`): mixer(map(norm(x)))."""
     parts = {"mixer_norm": mixer_norm, "mixers": tuple(mixers), "ffn_norm": ffn_norm, "ffn": ffn}
     if mixer_post_norm is not None:
         parts["mixer_post_norm"] = mixer_post_norm
     if ffn_post_norm is not None:
         parts["ffn_post_norm"] = ffn_post_norm
+    if mixer_input is not None:
+        parts["mixer_input"] = mixer_input
+    if ffn_input is not None:
+        parts["ffn_input"] = ffn_input
     return LayerSpec("parallel_prenorm", prefix, parts)
 
 
@@ -61,10 +67,16 @@ def _lane_ones(n: int, device) -> Tensor:
 class ResidualStream:
     """The float32 hidden state [T, D] of a step plus the branches waiting to be added."""
 
-    def __init__(self, h: Tensor, ctx, n_branch_buffers: int, lanes: Optional[int] = None):
+    def __init__(self, h: Tensor, ctx, n_branch_buffers: int, lanes: Optional[int] = None, second_buffer: bool = False):
+        """``second_buffer``: the model has launches that fold the stream while several blocks read the same rows of
+        it (`normed_mapped`): they write the folded stream to another buffer and the two change places."""
         self.h = h
         self.ctx = ctx
+        self._other: Optional[Tensor] = None
+        if second_buffer and not ctx.decode_only:
+            self._other = ctx.workspace.alloc(tuple(h.shape), torch.float32)
         self.pending: List[Tuple[Tensor, float]] = []
+        self.pending_vector: Optional[Tensor] = None  # [D] float32, waits to join every row of the stream
         self.pending_post: Optional[Norm] = None  # normed once more before the pending branches join (see Norm.folds_post)
         self._buffers = [ctx.workspace.alloc(tuple(h.shape), ctx.dtype) for _ in range(n_branch_buffers)]
         self._taken = 0
@@ -89,6 +101,22 @@ class ResidualStream:
         self._taken += 1
         return buf
 
+    def add_vector(self, vector: Tensor) -> None:
+        """A vector [D] (float32) waits to join every row of the stream, with the branches that wait already."""
+        if self.lanes is not None:
+            raise RuntimeError("a residual state in lanes has no single stream for a vector to join")
+        if self.pending_post is not None or self.pending_vector is not None:
+            self.flush()
+        self.pending_vector = vector
+
+    def _settle_vector(self) -> None:
+        """Fold the waiting vector (and two waiting branches with it) into the stream by a launch of its own."""
+        vec, self.pending_vector = self.pending_vector, None
+        if vec is not None:
+            self._settle_post()
+            K.fold_norm(self.h, self.h, self.pending[:2], vec, None, 0.0, 1, None)
+            self.pending = self.pending[2:]
+
     def add(self, branch: Tensor, scale: float) -> None:
         if self.pending_post is not None:
             self._settle_post()  # what waits with a post norm is one sublayer's result: settle it first
@@ -96,7 +124,7 @@ class ResidualStream:
 
     def add_normed(self, branches: Sequence[Tuple[Tensor, float]], post: Norm) -> None:
         """A sublayer's result sum(scale_i * branch_i) waits to join the stream as post(that sum)."""
-        if self.pending:
+        if self.pending or self.pending_vector is not None:
             self.flush()
         self.pending = [(b, float(s)) for b, s in branches]
         self.pending_post = post
@@ -142,6 +170,13 @@ class ResidualStream:
             return self.lanes_normed(self._ones, norm, rows)
         n_rows = self.h.shape[0] if rows is None else rows.numel()
         out = self.ctx.workspace.alloc((n_rows, self.h.shape[1]), self.ctx.dtype)
+        if self.pending_vector is not None:
+            pro = norm.group_prologue()
+            if pro is not None and rows is None and self.pending_post is None and len(self.pending) <= 2:
+                K.fold_norm(self.h, self.h, self.pending, self.pending_vector, *pro, out)
+                self.pending, self.pending_vector, self._taken = [], None, 0
+                return out
+            self._settle_vector()
         if self.pending_post is not None and self.pending and norm.folds_post(self.pending_post):
             norm.forward(self.h, self.pending, out, rows, self.ctx, post=self.pending_post)
         else:
@@ -153,12 +188,41 @@ class ResidualStream:
             self._taken = 0
         return out
 
+    def normed_mapped(self, norm: Norm, input_map: Optional[InputMap], cache: LayerCache) -> Tensor:
+        """What a sublayer reads: map(norm(stream)), with the pending branches folded in.  One launch where the map is
+        a convolution over time and the norm offers its parameters; the plain norm without a map."""
+        if input_map is None:
+            return self.normed(norm)
+        pro, conv = norm.group_prologue(), input_map.fused_conv(cache)
+        if pro is None or conv is None or self.lanes is not None:
+            n = self.normed(norm)
+            out = self.ctx.workspace.alloc(tuple(n.shape), n.dtype)
+            input_map.forward(n, self.ctx, cache, out)
+            return out
+        self._settle_post()
+        while len(self.pending) > 2:
+            fold_branches(self.h, self.pending[:2])
+            self.pending = self.pending[2:]
+        ctx = self.ctx
+        out = ctx.workspace.alloc(tuple(self.h.shape), ctx.dtype)
+        in_place = ctx.decode_only or (not self.pending and self.pending_vector is None)
+        if not in_place and self._other is None:
+            raise RuntimeError("the stream has no second buffer (an arrangement with input maps says folds_across_rows)")
+        dst = self.h if in_place else self._other
+        K.fold_norm(self.h, dst, self.pending, self.pending_vector, *pro, out, conv=conv[0], window=conv[1],
+                    cu=ctx.cu_seqlens, slots=ctx.slots, seq_of=ctx.seq_of, n_seq=ctx.n_seq, one_token=ctx.decode_only)
+        if dst is not self.h:
+            self.h, self._other = dst, self.h
+        self.pending, self.pending_vector, self._taken = [], None, 0
+        return out
+
     def take_pending(self, at_most: int = 2) -> List[Tuple[Tensor, float]]:
         """Hands the waiting branches (at most ``at_most``; the surplus and a waiting post norm are settled
         first) to a launch that folds them into the stream itself; the stream then holds none."""
         if self.lanes is not None:
             raise RuntimeError("a residual state in lanes has no single stream to fold branches into")
         self._settle_post()
+        self._settle_vector()
         while len(self.pending) > at_most:
             fold_branches(self.h, self.pending[:2])
             self.pending = self.pending[2:]
@@ -169,6 +233,7 @@ class ResidualStream:
     def flush(self) -> Tensor:
         if self.lanes is not None:
             raise RuntimeError("a residual state in lanes has no single stream to flush into")
+        self._settle_vector()
         if self.pending_post is not None and self.pending:
             self.pending_post.fold(self.h, self.pending, self.ctx)
         else:
@@ -183,10 +248,12 @@ class ParallelPreNormBlock(Part):
     def __init__(self, spec: LayerSpec, hidden_size: int):
         self.prefix = spec.prefix
         self.hidden_size = hidden_size
-        unknown = set(spec.parts) - {"mixer_norm", "mixers", "ffn_norm", "ffn", "mixer_post_norm", "ffn_post_norm"}
+        unknown = set(spec.parts) - {"mixer_norm", "mixers", "ffn_norm", "ffn", "mixer_post_norm", "ffn_post_norm",
+                                     "mixer_input", "ffn_input"}
         if unknown or spec.part("mixer_norm") is None or not spec.part("mixers"):
             raise ValueError("parallel_prenorm takes the parts mixer_norm, mixers (at least one), ffn_norm, ffn, "
-                             "mixer_post_norm and ffn_post_norm" + (f"; got also {sorted(unknown)}" if unknown else ""))
+                             "mixer_post_norm, ffn_post_norm, mixer_input and ffn_input"
+                             + (f"; got also {sorted(unknown)}" if unknown else ""))
         self.mixer_norm: Norm = build_part("norm", spec.part("mixer_norm"), width=hidden_size)
         self.mixers: List[Mixer] = [build_part("mixer", m, hidden_size=hidden_size) for m in spec.part("mixers")]
         self.mixer_post_norm: Optional[Norm] = None
@@ -195,9 +262,15 @@ class ParallelPreNormBlock(Part):
         self.ffn_norm: Optional[Norm] = None
         self.ffn: Optional[FeedForward] = None
         self.ffn_post_norm: Optional[Norm] = None
+        self.mixer_input: Optional[InputMap] = None
+        self.ffn_input: Optional[InputMap] = None
+        if spec.part("mixer_input") is not None:
+            self.mixer_input = build_part("input_map", spec.part("mixer_input"), hidden_size=hidden_size)
         if spec.part("ffn") is not None:
             if spec.part("ffn_norm") is None:
                 raise ValueError("a feed-forward needs its norm")
+            if spec.part("ffn_input") is not None:
+                self.ffn_input = build_part("input_map", spec.part("ffn_input"), hidden_size=hidden_size)
             self.ffn_norm = build_part("norm", spec.part("ffn_norm"), width=hidden_size)
             self.ffn = build_part("feed_forward", spec.part("ffn"), hidden_size=hidden_size)
             if spec.part("ffn_post_norm") is not None:
@@ -211,11 +284,19 @@ class ParallelPreNormBlock(Part):
         out: List[Part] = [self.mixer_norm, *self.mixers]
         if self.mixer_post_norm is not None:
             out.append(self.mixer_post_norm)
+        out += self._input_maps()
         if self.ffn is not None:
             out += [self.ffn_norm, self.ffn]
             if self.ffn_post_norm is not None:
                 out.append(self.ffn_post_norm)
         return out
+
+    def _input_maps(self) -> List[InputMap]:
+        return [m for m in (self.mixer_input, self.ffn_input) if m is not None]
+
+    def folds_across_rows(self) -> bool:
+        """Whether this layer folds the stream in launches whose blocks read one another's rows (see ResidualStream)."""
+        return bool(self._input_maps())
 
     def branch_buffers_needed(self) -> int:
         # with post norms a sublayer's result may still wait while the next one takes its buffer
@@ -223,8 +304,8 @@ class ParallelPreNormBlock(Part):
         return max(len(self.mixers), 1) + extra
 
     def state_specs(self) -> List[Tuple[str, StateSpec]]:
-        """(qualified name, spec) for every state of every mixer of this layer."""
-        return [(f"{m.name}.{s.name}", s) for m in self.mixers for s in m.state_specs()]
+        """(qualified name, spec) for every state of every mixer and input map of this layer."""
+        return [(f"{m.name}.{s.name}", s) for m in [*self.mixers, *self._input_maps()] for s in m.state_specs()]
 
     def finalize(self, dtype: torch.dtype, device: torch.device) -> None:
         for p in self.parts():
@@ -261,6 +342,8 @@ class ParallelPreNormBlock(Part):
             return False
         if self.mixer_post_norm is not None or self.ffn_post_norm is not None:
             return False  # the products of that path add straight into the stream
+        if self._input_maps():
+            return False  # ... and norm it in their prologues
         if any(m.output_weight() is None or m.output_bias() is not None for m in self.mixers):
             return False
         return len(self.mixers) <= 2
@@ -326,7 +409,7 @@ class ParallelPreNormBlock(Part):
 
     def accepts_length_bounds(self, dtype: torch.dtype, page_size: int) -> bool:
         """See Mixer.accepts_length_bounds: norms and feed-forwards go row by row, the mixers decide."""
-        return all(m.accepts_length_bounds(dtype, page_size) for m in self.mixers)
+        return not self._input_maps() and all(m.accepts_length_bounds(dtype, page_size) for m in self.mixers)
 
     def joins_side_stream(self, ctx) -> bool:
         """Whether this layer may start while ``ctx.unjoined_stream`` still works (a weight fetch that
@@ -339,7 +422,7 @@ class ParallelPreNormBlock(Part):
             return
         ws = ctx.workspace
         mark = ws.mark()
-        n = stream.normed(self.mixer_norm)
+        n = stream.normed_mapped(self.mixer_norm, self.mixer_input, cache)
         if self._fused_in is not None:
             proj = ws.alloc((n.shape[0], self._fused_in.shape[0]), n.dtype)
             if self.mixer_post_norm is not None:
@@ -389,7 +472,7 @@ class ParallelPreNormBlock(Part):
             for out, scale in results:
                 stream.add(out, scale)
         if self.ffn is not None:
-            f = stream.normed(self.ffn_norm)
+            f = stream.normed_mapped(self.ffn_norm, self.ffn_input, cache)
             out = stream.take_branch()
             self.ffn.forward(f, ctx, out)
             if self.ffn_post_norm is not None:

@@ -9,7 +9,8 @@ latent is kept per token.
     entries i and i + rot_dims/2) turn together by the angle p * rot_base^(-2i / rot_dims);
     score = (q_h . k_h) * scale;  token i sees every j <= i (``window`` > 0: only 0 <= i - j < window);
     softmax, with ``sink`` also exp(sink_h) in its denominator (a score without key or value);
-    with ``gate`` head h's result is multiplied by sigmoid(Wg x)_h;  out = Wo [heads].
+    with ``gate`` "head" (or True) head h's result is multiplied by sigmoid(Wg x)_h, with "channel" every channel of
+    the concatenated heads by its own sigmoid(Wg x);  out = Wo [heads].
 
 The per-head matrices move from the cached side to the query and the result, so that a token's cache
 row serves every head:
@@ -47,7 +48,7 @@ class LatentAttention(PagedSoftmaxAttention):
 
     def __init__(self, hidden_size: int, heads: int, dim: int, vdim: int, q_rank: int, kv_rank: int, scale: float,
                  norm_eps: float, rot_dim: int = 0, rot_dims: int = 0, rot_base: float = 10000.0, sink: bool = False,
-                 gate: bool = False, out_multiplier: float = 1.0, rot_layout: str = "pairs", window: int = 0,
+                 gate=False, out_multiplier: float = 1.0, rot_layout: str = "pairs", window: int = 0,
                  shared_kv: bool = False, cache_window: Optional[int] = None):
         if rot_dims % 2 or not 0 <= rot_dims <= rot_dim:
             raise ValueError("rot_dims must be even and at most rot_dim")
@@ -70,7 +71,9 @@ class LatentAttention(PagedSoftmaxAttention):
         self.q_rank, self.kv_rank = int(q_rank), int(kv_rank)
         self.rot_dim, self.rot_dims, self.rot_base = int(rot_dim), int(rot_dims), float(rot_base)
         self.scale, self.norm_eps = float(scale), float(norm_eps)
-        self.has_sink, self.has_gate = bool(sink), bool(gate)
+        if gate not in (False, True, "head", "channel"):
+            raise ValueError("gate is False, 'head' (True) or 'channel'")
+        self.has_sink, self.has_gate, self.channel_gate = bool(sink), bool(gate), gate == "channel"
         self.out_scale = float(out_multiplier)
         self.padded_dim = K.latent_padded_dim(self.kv_rank, self.rot_dim)
         K.check_head_dim(self.padded_dim, K.FLOAT_ATTENTION_MAX_HEAD)
@@ -96,7 +99,7 @@ class LatentAttention(PagedSoftmaxAttention):
         if self.has_sink:
             specs.append(ParamSpec("sink", (H,), kind="vector", init=("normal", 1.0)))
         if self.has_gate:
-            specs.append(ParamSpec("g", (H, D)))
+            specs.append(ParamSpec("g", (self.o_dim if self.channel_gate else H, D)))
         specs.append(ParamSpec("o", (D, self.o_dim)))
         return specs
 
@@ -169,7 +172,10 @@ class LatentAttention(PagedSoftmaxAttention):
         if not self.has_gate:
             return heads
         gated = ws.alloc((T, self.o_dim), proj.dtype)
-        K.head_gate(heads, proj[:, c_g:c_g + H], 1.0, gated, H, self.vdim)
+        if self.channel_gate:
+            K.sigmoid_gate(heads, proj[:, c_g:c_g + self.o_dim], 1.0, gated, H, self.vdim, self.vdim)
+        else:
+            K.head_gate(heads, proj[:, c_g:c_g + H], 1.0, gated, H, self.vdim)
         return gated
 
 

@@ -4,9 +4,10 @@
     weights p the softmax over the chosen z only (``router`` "softmax_all": scores s = softmax(z) over ALL
     experts; only experts of the ``keep`` best of ``groups`` equal groups of neighbours can be chosen, a group
     counting by its largest score; the ``top`` largest s are chosen and the weights are those s themselves,
-    not divided by their sum);
+    not divided by their sum; ``router`` "sigmoid": s = sigmoid(z), the ``top`` largest, weights s as they are);
     expert e:  g = min(Wg_e x, limit), u = clamp(Wu_e x, -limit, limit),
                y_e = Wd_e [ g * sigmoid(act_alpha * g) * (u + act_shift) ];
+    (``weigh`` "input": the weight multiplies the expert's input instead, y_e = expert_e(p_e x), and the sum is plain);
     out = sum over the chosen e of p_e y_e  (+ the shared expert's output, same form with its own
     width and limit, for every token).
 
@@ -45,18 +46,23 @@ class RoutedGLU(FeedForward):
     def __init__(self, hidden_size: int, experts: int, top: int, expert_ff: int, expert_limit: float,
                  shared_ff: int = 0, shared_limit: float = 0.0, act_alpha: float = 1.702, act_shift: float = 1.0,
                  router_bias: bool = True, out_multiplier: float = 1.0, router: str = "top_softmax", groups: int = 1,
-                 keep: int = 1):
+                 keep: int = 1, weigh: str = "output"):
         if not 1 <= top <= experts:
             raise ValueError("top must be between 1 and the number of experts")
         if expert_ff <= 0 or shared_ff < 0:
             raise ValueError("expert widths must be positive")
-        if router not in ("top_softmax", "softmax_all"):
-            raise ValueError("router is 'top_softmax' or 'softmax_all'")
+        if router not in ("top_softmax", "softmax_all", "sigmoid"):
+            raise ValueError("router is 'top_softmax', 'softmax_all' or 'sigmoid'")
+        if weigh not in ("output", "input"):
+            raise ValueError("weigh is 'output' or 'input'")
         if groups < 1 or experts % groups or not 1 <= keep <= groups or top > keep * (experts // groups):
             raise ValueError("groups must divide the experts, keep <= groups, top <= keep * experts / groups")
-        if router == "top_softmax" and groups != 1:
+        if router != "softmax_all" and groups != 1:
             raise ValueError("groups of experts need the 'softmax_all' router")
-        self.softmax_all, self.groups, self.keep = router == "softmax_all", int(groups), int(keep)
+        # the router kernel's mode (see kernels.ops.moe_route)
+        self.scored = {"top_softmax": False, "softmax_all": "softmax", "sigmoid": "sigmoid"}[router]
+        self.groups, self.keep = int(groups), int(keep)
+        self.weigh_input = weigh == "input"
         self.hidden_size = int(hidden_size)
         self.experts, self.top, self.expert_ff = int(experts), int(top), int(expert_ff)
         self.expert_limit, self.shared_ff, self.shared_limit = float(expert_limit), int(shared_ff), float(shared_limit)
@@ -112,11 +118,9 @@ class RoutedGLU(FeedForward):
         A = T * top
         ids = ws.alloc((T, top), torch.int32)
         weights = ws.alloc((T, top), torch.float32)
-        if self.softmax_all:
-            K.moe_route(x, self.router_w, self.router_b, top, ids, weights, scored="softmax", groups=self.groups,
-                        keep=self.keep)
-        else:
-            K.moe_route(x, self.router_w, self.router_b, top, ids, weights)
+        K.moe_route(x, self.router_w, self.router_b, top, ids, weights, scored=self.scored, groups=self.groups, keep=self.keep)
+        # the experts have no biases, so a weight on their input is a weight on their gate and up sums
+        in_w, out_w = (weights, None) if self.weigh_input else (None, weights)
         offsets = ws.alloc((E + 1,), torch.int32)
         tile_start = ws.alloc((E + 1,), torch.int32)
         perm = ws.alloc((A,), torch.int32)
@@ -144,7 +148,7 @@ class RoutedGLU(FeedForward):
             xs = ws.alloc((A, D), x.dtype)
             K.moe_gather_rows(x, perm, top, xs)
             K.moe_tc_gemm(xs, self.gate_up, perm, offsets, tile_start, True, act, limit=self.expert_limit,
-                          alpha=self.act_alpha, shift=self.act_shift)
+                          alpha=self.act_alpha, shift=self.act_shift, row_weights=in_w)
             K.moe_tc_gemm(act, self.down, perm, offsets, tile_start, False, y)
         else:
             form = "float"
@@ -152,11 +156,11 @@ class RoutedGLU(FeedForward):
                 form = "mma_few" if A <= _FEW_PAIRS else "mma"
             K.moe_plan(ids, E, form, offsets, tile_start, perm)
             K.moe_gemm(x, self.gate_up, perm, offsets, tile_start, top, True, act, form, limit=self.expert_limit,
-                       alpha=self.act_alpha, shift=self.act_shift)
+                       alpha=self.act_alpha, shift=self.act_shift, row_weights=in_w)
             K.moe_gemm(act, self.down, perm, offsets, tile_start, top, False, y, form)
         if side is not None:
             main.wait_stream(side)
-        K.moe_combine(y, weights, shared, out)
+        K.moe_combine(y, out_w, shared, out)
 
     def streamed_weights(self) -> List[Tensor]:
         return [w for w in (self.shared_gate_up, self.shared_down) if w is not None]

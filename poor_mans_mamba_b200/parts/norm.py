@@ -1,5 +1,9 @@
 """Norms with the residual additions folded in: RMSNorm and the statistic-free tanh norm.
 
+The RMS norm may take its root mean square over ``groups`` equal neighbouring parts of the row instead of
+the whole row (`Norm.group_prologue`; the fold, a vector that waits on the stream and the convolution of a
+sublayer's input then share its launch, csrc/fold_norm.cu).
+
 y = x * (1/sqrt(mean(x^2) + eps)) * w; eps inside the root, the weight multiplies after
 normalisation (reference src/ops/cpu/rms_norm.cpp:11-16).  Statistics are float32.  A weight
 stored around zero (y = ... * (1 + w)) is the same norm with ``offset`` 1.  The RMS norm also serves as
@@ -29,9 +33,13 @@ def fold_branches(h: Tensor, pending) -> None:
 class RMSNorm(Norm):
     """``offset``: the stored weight is kept around zero and the norm multiplies by offset + w (the sum
     is made once, in float32, when the tensors are bound).  ``tensor``: the weight's name within the
-    part ("" where the part's own name is the tensor's)."""
+    part ("" where the part's own name is the tensor's).  ``groups``: the row is cut into that many equal
+    neighbouring parts and each is divided by its own root mean square."""
 
-    def __init__(self, width: int, eps: float, offset: float = 0.0, tensor: str = "weight"):
+    def __init__(self, width: int, eps: float, offset: float = 0.0, tensor: str = "weight", groups: int = 1):
+        if groups < 1 or width % groups:
+            raise ValueError("the norm's groups must divide the width")
+        self.groups = int(groups)
         self.width = int(width)
         self.eps = float(eps)
         self.offset = float(offset)
@@ -47,16 +55,19 @@ class RMSNorm(Norm):
         self.weight = w if self.offset == 0.0 else (w + self.offset).contiguous()
 
     def rms_prologue(self):
-        return self.weight, self.eps
+        return (self.weight, self.eps) if self.groups == 1 else None
+
+    def group_prologue(self):
+        return self.weight, self.eps, self.groups
 
     def folds_post(self, post: Norm) -> bool:
-        return isinstance(post, RMSNorm)
+        return isinstance(post, RMSNorm) and self.groups == 1 and post.groups == 1
 
     def forward(self, h: Tensor, pending, out: Tensor, rows: Optional[Tensor], ctx, post: Optional[Norm] = None) -> None:
         items = list(pending)
         if post is not None and items:
             # a sublayer's result, normed once more before it joins: x <- x + post(sum), out = norm(x), one launch
-            if not isinstance(post, RMSNorm) or len(items) > 2:
+            if not self.folds_post(post) or len(items) > 2:
                 raise ValueError("the RMS norm folds a post norm of its own kind over at most two branches")
             K.add_postnorm_rmsnorm(h, items, post.weight, post.eps, self.weight, self.eps, out, rows)
             return
@@ -65,12 +76,21 @@ class RMSNorm(Norm):
                 raise ValueError("row-selected norm takes at most two pending branches")
             K.add_rmsnorm(h, items[:2], None, 0.0, None)
             items = items[2:]
-        K.add_rmsnorm(h, items, self.weight, self.eps, out, rows)
+        if self.groups > 1:
+            K.fold_norm(h, h, items, None, self.weight, self.eps, self.groups, out, rows)
+        else:
+            K.add_rmsnorm(h, items, self.weight, self.eps, out, rows)
+
+    def _whole_row(self) -> None:
+        if self.groups > 1:
+            raise NotImplementedError("an RMS norm over groups of channels cannot norm a sublayer's result")
 
     def apply(self, pending, out: Tensor, ctx) -> None:
+        self._whole_row()
         K.add_postnorm_rmsnorm(None, list(pending), self.weight, self.eps, None, 0.0, out)
 
     def fold(self, h: Tensor, pending, ctx) -> None:
+        self._whole_row()
         K.add_postnorm_rmsnorm(h, list(pending), self.weight, self.eps, None, 0.0, None)
 
 

@@ -7,13 +7,30 @@ The whole head is rotated; there is no scaling of positions.
 """
 from __future__ import annotations
 
-from typing import Optional
+import math
+from typing import Optional, Sequence
 
 import torch
 
 from .base import PositionEncoding, register_position_encoding
 
 Tensor = torch.Tensor
+
+
+def rotary_frequencies(dims: int, base: float, factor: float = 1.0,
+                       scaling: Optional[Sequence[float]] = None) -> Tensor:
+    """base^(-2i/dims) / factor for i < dims/2, made in float64 and rounded to float32 once.  ``scaling`` = (factor, low,
+    high, original): by how often a frequency's wavelength fits into ``original`` positions, n = original * f / (2 pi),
+    it is divided by the factor (n < low), kept (n > high) or blended, (1 - s) f / factor + s f with
+    s = (n - low) / (high - low)."""
+    i = torch.arange(dims // 2, dtype=torch.float64)
+    f = torch.pow(torch.tensor(float(base), dtype=torch.float64), -2.0 * i / float(max(dims, 1))) / float(factor)
+    if scaling is not None:
+        by, low, high, original = (float(v) for v in scaling)
+        n = original * f / (2.0 * math.pi)
+        s = (n - low) / (high - low) if high != low else torch.zeros_like(n)
+        f = torch.where(n > high, f, torch.where(n < low, f / by, (1.0 - s) * f / by + s * f))
+    return f.to(torch.float32)
 
 
 class RotaryEncoding(PositionEncoding):

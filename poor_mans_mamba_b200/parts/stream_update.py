@@ -16,6 +16,9 @@ read, the two small products, the activation, the root mean square and the sum a
 
 (the model keeps x0 for the step as the right half of ``ResidualStream.reentry``).  The result is written
 into the float32 stream directly.
+
+``pass_step``: a learned vector of the pass's number joins the stream, x <- x + step[pass]; it waits on the stream
+and is folded in by the launch that norms it next.
 """
 from __future__ import annotations
 
@@ -60,7 +63,26 @@ class TokenGatedUpdate(StreamUpdate):
                              self.w_proj_t, self.norm_w, self.eps, w_proj_rows=self.w_proj)
 
 
+class PassStep(StreamUpdate):
+    def __init__(self, hidden_size: int, passes: int, tensor: str = "step"):
+        if passes < 1:
+            raise ValueError("at least one pass")
+        self.hidden_size, self.passes, self.tensor = int(hidden_size), int(passes), str(tensor)
+
+    def param_specs(self) -> List[ParamSpec]:
+        return [ParamSpec(self.tensor, (self.passes, self.hidden_size), kind="vector", init=("normal", 0.5))]
+
+    def bind(self, params: Dict[str, Tensor]) -> None:
+        # a tensor per pass: every row starts on a boundary of its own
+        self.steps = [row.clone() for row in params[self.tensor]]
+
+    def enter(self, stream, ctx, pass_index: int) -> None:
+        stream.add_vector(self.steps[pass_index])
+
+
 class EmbeddingReentry(StreamUpdate):
+    reads_embedding = True
+
     def __init__(self, hidden_size: int, tensor: str = "in"):
         self.hidden_size = int(hidden_size)
         self.tensor = str(tensor)
@@ -87,3 +109,4 @@ class EmbeddingReentry(StreamUpdate):
 
 register_stream_update("token_gated_update", TokenGatedUpdate)
 register_stream_update("embedding_reentry", EmbeddingReentry)
+register_stream_update("pass_step", PassStep)
