@@ -23,7 +23,8 @@ L2 flush is needed between timed iterations.
 `--workload compare` is a measurement beside the benchmark (its own JSON line): a Boketar model (or, with
 `--design tafesun`, a Tafesun model) and a Falcon-H1 model of equal width, feed-forward size, layer count and
 vocabulary, one prompt step and decode steps of each with the L2 flushed before every timed step, and every
-kernel's device time.  `--design sorovik` measures a Sorovik model beside the Tafesun and the Gikovik models.
+kernel's device time.  `--design sorovik` measures a Sorovik model beside the Tafesun and the Gikovik models,
+`--design piladra` a Piladra model beside the Sorovik and the Falcon-H1 models.
 `--design gikovik` measures a Gikovik model beside the Tafesun model (the closest one:
 paged softmax attention and routed experts) in the same way.
 """
@@ -577,6 +578,31 @@ def sorovik_config(falcon, mixer_sizes, ff_sizes, layers, dense_ff):
             "layers": out}
 
 
+# `--workload compare --design piladra`: a Piladra model beside the Sorovik model and the Falcon-H1 model above (equal
+# width, layers and vocabulary; Sorovik's experts, experts a token and expert widths).  Of every four layers the first
+# and the last are attention layers with Falcon-H1's head counts and head size behind a window of 1,024 tokens, the second
+# is a latent layer with Sorovik's sizes (a cache row of 128), the third a Mamba-1 layer twice the width wide with 16
+# state entries per channel.  The first and third feed-forwards are dense (`dense_ff` wide), the others routed.  All
+# layers are one loop that runs once, so that the pass's vector is part of the step.
+def piladra_config(falcon, mixer_sizes, ff_sizes, layers, dense_ff):
+    experts, top, expert_ff, shared_ff = ff_sizes
+    heads, dim, vdim, _ = mixer_sizes
+    hd, width = falcon["head_dim"], falcon["hidden_size"]
+    att = {"heads": falcon["num_attention_heads"], "kv_heads": falcon["num_key_value_heads"], "dim": hd, "vdim": hd,
+           "scale": hd ** -0.5, "mask": {"size": 1024},
+           "rot": {"dims": hd, "base": 5e5, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+    lat = {"heads": heads, "dim": dim, "rot_dim": 32, "vdim": vdim, "kv_rank": 96, "scale": (dim + 32) ** -0.5,
+           "rot": {"dims": 32, "base": 1e6}}
+    scan = {"inner": 2 * width, "state": 16, "dt_rank": width // 16, "conv": 4}
+    dense = {"kind": "dense", "ff": dense_ff}
+    moe = {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": expert_ff}, "shared": {"ff": shared_ff}}
+    kinds = [("attention", att, dense), ("latent_attention", lat, moe), ("mamba1", scan, dense), ("attention", att, moe)]
+    out = [dict(zip(("type", "mixer", "mlp"), kinds[i % 4])) for i in range(layers)]
+    return {"architecture": "Piladra", "vocab": falcon["vocab_size"], "width": width, "norm": {"eps": 1e-6, "groups": 4},
+            "canon": {"taps": 3}, "residual_mult": 0.5, "logit_softcap": 30.0,
+            "loop": {"start": 0, "stop": layers, "times": 1}, "layers": out}
+
+
 def compare_workload(args, peaks) -> int:
     import torch
 
@@ -591,7 +617,13 @@ def compare_workload(args, peaks) -> int:
     falcon.update(falcon_keys)
     falcon["num_hidden_layers"] = layers
     vocab = falcon["vocab_size"]
-    if args.design == "sorovik":
+    if args.design == "piladra":
+        sizes = (falcon, GIKOVIK_MIXER[args.sizes], TAFESUN_FF[args.sizes], layers, ff)
+        configs = {"piladra": piladra_config(*sizes), "sorovik": sorovik_config(*sizes), "falcon_h1": falcon}
+        design_sizes = {"routed_ff": dict(zip(("experts", "top", "expert_ff", "shared_ff"), TAFESUN_FF[args.sizes])),
+                        "latent_mixer": dict(zip(("heads", "dim", "vdim", "q_rank"), GIKOVIK_MIXER[args.sizes])),
+                        "scan_mixer": configs["piladra"]["layers"][2]["mixer"] if layers > 2 else None}
+    elif args.design == "sorovik":
         configs = {"sorovik": sorovik_config(falcon, GIKOVIK_MIXER[args.sizes], TAFESUN_FF[args.sizes], layers, ff),
                    "tafesun": tafesun_config(falcon, TAFESUN_FF[args.sizes], layers),
                    "gikovik": gikovik_config(falcon, GIKOVIK_MIXER[args.sizes], TAFESUN_FF[args.sizes], layers)}
@@ -726,9 +758,9 @@ def main() -> int:
                          "count (--layers, default 4) and vocabulary at --sizes 0.5b or 7b: one prompt step of "
                          "--prompt-tokens and decode steps of --batch requests at --context, device-timed with the "
                          "L2 flushed, and the device time of every kernel of one step of each")
-    ap.add_argument("--design", default="boketar", choices=["boketar", "tafesun", "gikovik", "sorovik"],
+    ap.add_argument("--design", default="boketar", choices=["boketar", "tafesun", "gikovik", "sorovik", "piladra"],
                     help="--workload compare: the model that is measured beside Falcon-H1 (gikovik: beside Tafesun; "
-                         "sorovik: beside Tafesun and Gikovik)")
+                         "sorovik: beside Tafesun and Gikovik; piladra: beside Sorovik and Falcon-H1)")
     ap.add_argument("--no-check", dest="check", action="store_false",
                     help="skip the comparison with the plain implementation that runs before the timing: the first "
                          "two layers of the run's model, in the run's dtype, on the benchmark's schedule (a "
