@@ -7,13 +7,14 @@
 // so there is no matrix form: the work is one exponential and four multiply-adds per (token, channel, entry), and
 // the exponential unit (16 lanes a clock and SM) is the bound of prompt steps.
 //
-// LN neighbouring lanes share a channel and keep NPT entries each in registers for the whole walk (LN * NPT >= N;
-// entries beyond N have B = C = 0).  A block of 128 threads owns CH = 128 / LN channels of one chunk.  Tokens come
-// through shared memory in tiles of kTile: every thread makes the softplus and dt * x of its share of the tile
-// once, B and C are widened once, and the outputs of a tile are gated and written together.  The next tile's rows
-// are requested before a tile is walked.
+// A block owns 128 / LN channels of one chunk and has two halves of four warps.  In the walking half LN neighbouring lanes
+// share a channel and keep NPT state entries each in registers for the whole walk (LN * NPT >= N; entries beyond N have
+// B = C = 0): a token costs a lane two shared-memory reads and five instructions an entry, and nothing but the
+// state's own multiply-add waits for the token before.  The other half runs beside it, one tile of tokens ahead and one
+// behind: it widens the next tile's B and C, makes its step sizes and dt * x, requests the tile after that, and gates
+// and writes the outputs of the tile before.  One barrier a tile; the tiles' shared memory has two places.
 //
-// Prompt portions are cut into chunks only where one walk per channel would leave the GPU empty:
+// Portions are cut into chunks only where one walk per channel would leave most of the GPU empty:
 //   chunk_state   every chunk but a sequence's last, from a zero state: its end state and the sum of its dt
 //   chunk_pass    per state entry, over the chunks of a sequence: the chunks' start states
 //   walk          every chunk from its start state, with the outputs
@@ -26,7 +27,7 @@
 namespace pmm {
 
 constexpr int kSelThreads = 128;
-constexpr int kSelTile = 16;  // tokens per shared-memory tile
+constexpr int kSelWalkThreads = 2 * kSelThreads;  // the walking half and the half that makes its inputs
 
 // Base-2 exponential: the walk multiplies A by log2(e) once.  Approximate to 2 ulp in float.
 __device__ __forceinline__ float sel_exp2(float v) {
@@ -62,21 +63,6 @@ __device__ __forceinline__ void sel_st_state(float* row, int n0, int N, bool vec
   for (int i = 0; i < NPT; ++i)
     if (n0 + i < N) row[n0 + i] = o[i];
 }
-// NPT neighbouring floats of shared memory (16-byte aligned where NPT is a multiple of 4).
-template <int NPT>
-__device__ __forceinline__ void sel_ld_shared(const float* p, float* o) {
-  if (NPT % 4 == 0) {
-#pragma unroll
-    for (int i = 0; i < NPT; i += 4) {
-      const float4 v = *reinterpret_cast<const float4*>(p + i);
-      o[i] = v.x; o[i + 1] = v.y; o[i + 2] = v.z; o[i + 3] = v.w;
-    }
-    return;
-  }
-#pragma unroll
-  for (int i = 0; i < NPT; ++i) o[i] = p[i];
-}
-
 struct SelArgs {
   const void* x;        // [T, I] after convolution and activation, rows of ld_x
   const void* raw;      // [T, I] step sizes before bias and softplus
@@ -96,6 +82,8 @@ struct SelArgs {
   int n_seq, I, N, chunk_len;
   const void* w_dt;     // decode: [I, R]
   int R;
+  int pairs;            // rows of x, raw, z and y may be read two channels at a time
+  int bc_pairs;         // B and C two entries at a time
 };
 
 // The sequence and the chunk within it of global chunk `idx`; false when there is no such chunk.  Called by whole warps.
@@ -127,145 +115,279 @@ __device__ __forceinline__ bool sel_find_chunk(const int* __restrict__ cu, int n
   return false;
 }
 
-// OUT: the walk with outputs.  Otherwise chunk_state.
-template <typename S, typename ACC, int LN, int NPT, bool OUT>
-__global__ void __launch_bounds__(kSelThreads) selective_walk_kernel(const SelArgs p) {
-  constexpr int CH = kSelThreads / LN;
-  constexpr int NS = NPT + (NPT % 4 == 0 ? 4 : 0);  // a lane's entries of B or C (padded against bank conflicts)
-  __shared__ ACC s_dt[kSelTile][CH], s_u[kSelTile][CH];
-  __shared__ __align__(16) float s_b[kSelTile][LN * NS];
-  __shared__ __align__(16) float s_c[OUT ? kSelTile : 1][LN * NS];
-  __shared__ ACC s_y[OUT ? kSelTile : 1][CH + 1];
-  pdl_launch_dependents();
-  const int ch = threadIdx.x / LN, q = threadIdx.x % LN;
-  const int c0 = blockIdx.x * CH, c = c0 + ch;
-  const int N = p.N, I = p.I;
-  const bool ch_ok = c < I;
-  // constants of the channel: weights, read before the wait
-  ACC a2[NPT];
-#pragma unroll
-  for (int i = 0; i < NPT; ++i) {
-    const int n = q * NPT + i;
-    a2[i] = (ch_ok && n < N) ? static_cast<ACC>(-1.4426950408889634) * scan_exp(static_cast<ACC>(p.a_log[static_cast<size_t>(c) * N + n])) : static_cast<ACC>(0);
+// A thread's two neighbouring channels of one token as they lie in memory.
+template <typename S>
+struct SelPair;
+template <>
+struct SelPair<__nv_bfloat16> {
+  __nv_bfloat162 v;
+  __device__ __forceinline__ float2 get() const { return __bfloat1622float2(v); }
+};
+template <>
+struct SelPair<float> {
+  float2 v;
+  __device__ __forceinline__ float2 get() const { return v; }
+};
+__device__ __forceinline__ void sel_ld_pair(const __nv_bfloat16* p, bool whole, bool second, SelPair<__nv_bfloat16>& o) {
+  if (whole) {
+    o.v = *reinterpret_cast<const __nv_bfloat162*>(p);
+  } else {
+    o.v.x = p[0];
+    o.v.y = second ? p[1] : __float2bfloat16_rn(0.f);
   }
+}
+__device__ __forceinline__ void sel_ld_pair(const float* p, bool, bool second, SelPair<float>& o) {
+  o.v.x = p[0];
+  o.v.y = second ? p[1] : 0.f;
+}
+__device__ __forceinline__ void sel_zero(SelPair<__nv_bfloat16>& o) { o.v = __floats2bfloat162_rn(0.f, 0.f); }
+__device__ __forceinline__ void sel_zero(SelPair<float>& o) { o.v = make_float2(0.f, 0.f); }
+
+// softplus(v) = max(v, 0) + log(1 + e), e = exp(-|v|).  Float: base-2 approximations; where e is small, 1 + e would round
+// it away, so the series of log(1 + e) takes over (below 1/16 its fifth term is under 2e-7 of the sum).
+__device__ __forceinline__ float sel_softplus(float v) {
+  const float e = sel_exp2(-1.4426950408889634f * fabsf(v));
+  float lg;
+  asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(lg) : "f"(1.f + e));
+  const float series = e * (1.f - e * (0.5f - e * (1.f / 3.f - e * (0.25f - e * 0.2f))));
+  return fmaxf(v, 0.f) + (e < 0.0625f ? series : 0.6931471805599453f * lg);
+}
+__device__ __forceinline__ double sel_softplus(double v) { return scan_softplus<double>(v); }
+
+template <typename ACC>
+struct SelDu {
+  ACC dt, u;
+};
+
+__device__ __forceinline__ void sel_barrier() { asm volatile("bar.sync 1, %0;" ::"n"(kSelWalkThreads) : "memory"); }
+
+// Tokens per tile for NB state entries of a channel (padded).
+template <typename ACC, int NB>
+struct SelTile {
+  static constexpr int kFloat = NB <= 32 ? 32 : NB <= 128 ? 16 : 8;
+  static constexpr int kTokens = sizeof(ACC) == 8 && kFloat > 16 ? 16 : kFloat;
+};
+
+// OUT: the walk with outputs.  Otherwise chunk_state.  A lane's entries are pairs: entry (i * LN + q) * 2 + j.
+template <typename S, typename ACC, int LN, int NPT, bool OUT>
+__global__ void __launch_bounds__(kSelWalkThreads, sizeof(ACC) == 4 ? 3 : 2) selective_walk_kernel(const SelArgs p) {
+  constexpr int CH = kSelThreads / LN, NB = LN * NPT, NP = NPT / 2;
+  constexpr int TT = SelTile<ACC, NB>::kTokens;
+  constexpr int G = LN < 8 ? LN : 8;   // tokens whose sums over the lanes are made together
+  __shared__ __align__(16) SelDu<ACC> s_du[2][TT][CH];
+  __shared__ __align__(16) float2 s_bc[2][TT][NB];  // (B, C) of an entry
+  __shared__ ACC s_y[2][OUT ? TT : 1][CH];
+  pdl_launch_dependents();
+  const bool walker = threadIdx.x < kSelThreads;
+  const int tid = threadIdx.x % kSelThreads;
+  const int c0 = blockIdx.x * CH;
+  const int N = p.N, I = p.I;
   pdl_wait();
   int seq, k, n_chunks;
   if (!sel_find_chunk(p.cu, p.n_seq, p.chunk_len, blockIdx.y, &seq, &k, &n_chunks)) return;
   if (!OUT && k == n_chunks - 1) return;  // nobody starts from a sequence's last chunk
   const int t_end = p.cu[seq + 1];
   const int t0 = p.cu[seq] + k * p.chunk_len, t1 = min(t_end, t0 + p.chunk_len);
-  float* slot_state = p.state + (static_cast<size_t>(p.slots[seq]) * I + (ch_ok ? c : 0)) * N;
-  float* mine = n_chunks > 1 ? p.chunk_state + (static_cast<size_t>(blockIdx.y) * I + (ch_ok ? c : 0)) * N : slot_state;
-  const bool svec = N % 4 == 0;
-  ACC st[NPT];
-  {
-    float f[NPT];
-    if (OUT) sel_ld_state<NPT>(mine, q * NPT, N, svec, f);
-#pragma unroll
-    for (int i = 0; i < NPT; ++i) st[i] = OUT ? static_cast<ACC>(f[i]) : static_cast<ACC>(0);
-  }
-  ACC dt_sum = 0;
+  const int n_tiles = (t1 - t0 + TT - 1) / TT;
 
-  // A tile's raw values wait in registers while the tile before it is walked.
-  constexpr int PX = kSelTile * CH / kSelThreads;                     // (token, channel) pairs per thread
-  constexpr int PB = (kSelTile * LN * NPT + kSelThreads - 1) / kSelThreads;  // (token, entry) pairs per thread
-  float rx[PX], rd[PX], rz[OUT ? PX : 1], rb[PB], rc[OUT ? PB : 1];
-  const S* xs = static_cast<const S*>(p.x);
-  const S* ds = static_cast<const S*>(p.raw);
-  const S* zs = static_cast<const S*>(p.z);
-  const S* ls = static_cast<const S*>(p.low);
-  auto request = [&](int base) {
+  if (walker) {
+    const int ch = tid / LN, q = tid % LN, c = c0 + ch;
+    const bool ok = c < I;
+    const bool even = N % 2 == 0;
+    float* slot_state = p.state + (static_cast<size_t>(p.slots[seq]) * I + (ok ? c : 0)) * N;
+    float* mine = n_chunks > 1 ? p.chunk_state + (static_cast<size_t>(blockIdx.y) * I + (ok ? c : 0)) * N : slot_state;
+    const float* al = p.a_log + static_cast<size_t>(ok ? c : 0) * N;
+    ACC a2[NPT], st[NPT];
 #pragma unroll
-    for (int r = 0; r < PX; ++r) {
-      const int e = r * kSelThreads + threadIdx.x, tt = e / CH, cc = c0 + e % CH;
-      const long long t = base + tt;
-      const bool ok = t < t1 && cc < I;
-      rx[r] = ok ? ldf(xs + t * p.ld_x + cc) : 0.f;
-      rd[r] = ok ? ldf(ds + t * p.ld_raw + cc) : 0.f;
-      if (OUT) rz[OUT ? r : 0] = ok ? ldf(zs + t * p.ld_z + cc) : 0.f;
-    }
-#pragma unroll
-    for (int r = 0; r < PB; ++r) {
-      const int e = r * kSelThreads + threadIdx.x, tt = e / (LN * NPT), n = e % (LN * NPT);
-      const long long t = base + tt;
-      const bool ok = tt < kSelTile && t < t1 && n < N;
-      rb[r] = ok ? ldf(ls + t * p.ld_low + p.off_b + n) : 0.f;
-      if (OUT) rc[OUT ? r : 0] = ok ? ldf(ls + t * p.ld_low + p.off_c + n) : 0.f;
-    }
-  };
-  float bias[PX];
-#pragma unroll
-  for (int r = 0; r < PX; ++r) {
-    const int cc = c0 + (r * kSelThreads + threadIdx.x) % CH;
-    bias[r] = cc < I ? p.bias[cc] : 0.f;
-  }
-  request(t0);
-  for (int base = t0; base < t1; base += kSelTile) {
-    float zg[OUT ? PX : 1], xg[OUT ? PX : 1];
-#pragma unroll
-    for (int r = 0; r < PX; ++r) {
-      const int e = r * kSelThreads + threadIdx.x, tt = e / CH, cc = e % CH;
-      // (tokens past the chunk's end: dt = 0 leaves the state as it is)
-      const ACC dt = base + tt < t1 ? scan_softplus<ACC>(static_cast<ACC>(rd[r]) + static_cast<ACC>(bias[r])) : static_cast<ACC>(0);
-      s_dt[tt][cc] = dt;
-      s_u[tt][cc] = dt * static_cast<ACC>(rx[r]);
-      if (OUT) {
-        xg[OUT ? r : 0] = rx[r];
-        zg[OUT ? r : 0] = rz[OUT ? r : 0];
+    for (int i = 0; i < NP; ++i) {
+      const int n = (i * LN + q) * 2;
+      float2 av = make_float2(0.f, 0.f), sv = make_float2(0.f, 0.f);
+      if (n < N && even) {
+        av = *reinterpret_cast<const float2*>(al + n);
+        if (OUT) sv = *reinterpret_cast<const float2*>(mine + n);
+      } else if (n < N) {
+        av = make_float2(al[n], n + 1 < N ? al[n + 1] : 0.f);
+        if (OUT) sv = make_float2(mine[n], n + 1 < N ? mine[n + 1] : 0.f);
       }
+      a2[2 * i] = static_cast<ACC>(-1.4426950408889634) * scan_exp(static_cast<ACC>(av.x));
+      a2[2 * i + 1] = static_cast<ACC>(-1.4426950408889634) * scan_exp(static_cast<ACC>(av.y));
+      st[2 * i] = sv.x;
+      st[2 * i + 1] = sv.y;
     }
+    ACC dt_sum = 0;
+    sel_barrier();
+    for (int tile = 0; tile < n_tiles; ++tile) {
+      const int buf = tile & 1;
 #pragma unroll
-    for (int r = 0; r < PB; ++r) {
-      const int e = r * kSelThreads + threadIdx.x, tt = e / (LN * NPT), n = e % (LN * NPT);
-      if (tt < kSelTile) {
-        s_b[tt][(n / NPT) * NS + n % NPT] = rb[r];
-        if (OUT) s_c[OUT ? tt : 0][(n / NPT) * NS + n % NPT] = rc[OUT ? r : 0];
+      for (int g = 0; g < TT; g += G) {
+        ACC acc[G];
+#pragma unroll
+        for (int j = 0; j < G; ++j) {
+          const SelDu<ACC> du = s_du[buf][g + j][ch];
+          ACC sum = 0;
+#pragma unroll
+          for (int i = 0; i < NP; ++i) {
+            const float4 bc = *reinterpret_cast<const float4*>(&s_bc[buf][g + j][(i * LN + q) * 2]);
+            st[2 * i] = sel_exp2(du.dt * a2[2 * i]) * st[2 * i] + du.u * static_cast<ACC>(bc.x);
+            st[2 * i + 1] = sel_exp2(du.dt * a2[2 * i + 1]) * st[2 * i + 1] + du.u * static_cast<ACC>(bc.z);
+            if (OUT) {
+              sum += st[2 * i] * static_cast<ACC>(bc.y);
+              sum += st[2 * i + 1] * static_cast<ACC>(bc.w);
+            }
+          }
+          acc[j] = sum;
+          if (!OUT) dt_sum += du.dt;
+        }
+        if (OUT) {
+          // the lanes' sums of G tokens: at every level a lane hands half of its tokens to its partner and keeps the
+          // other half, so that lane q ends with the whole sum of token q
+#pragma unroll
+          for (int o = G / 2; o > 0; o >>= 1) {
+            const bool up = (q & o) != 0;
+#pragma unroll
+            for (int j = 0; j < o; ++j) {
+              const ACC send = up ? acc[j] : acc[j + o];
+              const ACC keep = up ? acc[j + o] : acc[j];
+              acc[j] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+            }
+          }
+#pragma unroll
+          for (int o = G; o < LN; o <<= 1) acc[0] += __shfl_xor_sync(0xffffffffu, acc[0], o);
+          if (q < G) s_y[buf][OUT ? g + q : 0][ch] = acc[0];
+        }
       }
+      sel_barrier();
     }
-    __syncthreads();
-    if (base + kSelTile < t1) request(base + kSelTile);
-#pragma unroll 4
-    for (int tt = 0; tt < kSelTile; ++tt) {
-      const ACC dt = s_dt[tt][ch], u = s_u[tt][ch];
-      ACC acc = 0;
-      float bv[NPT], cv[NPT];
-      sel_ld_shared<NPT>(&s_b[tt][q * NS], bv);
-      if (OUT) sel_ld_shared<NPT>(&s_c[OUT ? tt : 0][q * NS], cv);
+    if (!ok) return;
+    float* dst = OUT ? slot_state : mine;
+    if (!OUT || k == n_chunks - 1) {
 #pragma unroll
-      for (int i = 0; i < NPT; ++i) {
-        st[i] = sel_exp2(dt * a2[i]) * st[i] + u * static_cast<ACC>(bv[i]);
-        if (OUT) acc += st[i] * static_cast<ACC>(cv[i]);
-      }
-      if (OUT) {
-#pragma unroll
-        for (int o = LN / 2; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
-        if (q == 0) s_y[OUT ? tt : 0][ch] = acc;
-      } else if (q == 0) {
-        dt_sum += dt;
-      }
-    }
-    __syncthreads();
-    if (OUT) {
-#pragma unroll
-      for (int r = 0; r < PX; ++r) {
-        const int e = r * kSelThreads + threadIdx.x, tt = e / CH, cc = c0 + e % CH;
-        if (base + tt < t1 && cc < I) {
-          const ACC y = s_y[tt][e % CH] + static_cast<ACC>(p.d[cc]) * static_cast<ACC>(xg[OUT ? r : 0]);
-          const float g = sizeof(S) == 2 ? silu_fast(zg[OUT ? r : 0]) : silu_f(zg[OUT ? r : 0]);
-          stf(static_cast<S*>(p.y) + static_cast<size_t>(base + tt) * I + cc, static_cast<float>(y) * g);
+      for (int i = 0; i < NP; ++i) {
+        const int n = (i * LN + q) * 2;
+        if (n < N && even) {
+          *reinterpret_cast<float2*>(dst + n) = make_float2(static_cast<float>(st[2 * i]), static_cast<float>(st[2 * i + 1]));
+        } else if (n < N) {
+          dst[n] = static_cast<float>(st[2 * i]);
+          if (n + 1 < N) dst[n + 1] = static_cast<float>(st[2 * i + 1]);
         }
       }
     }
+    if (!OUT && q == 0) p.chunk_dt[static_cast<size_t>(blockIdx.y) * I + c] = static_cast<float>(dt_sum);
+    return;
   }
-  if (!ch_ok) return;
-  float* dst = OUT ? slot_state : mine;
-  if (!OUT || k == n_chunks - 1) {
-    float f[NPT];
+
+  // ------------------------------------------------------------------ the other half: thread -> (token of the tile, pair of channels)
+  constexpr int HC = CH / 2;
+  constexpr int PX = (TT * HC + kSelThreads - 1) / kSelThreads;
+  constexpr int TSTEP = kSelThreads / HC;                          // tokens between a thread's pairs
+  constexpr int HB = NB / 2;
+  constexpr int PB = (TT * HB + kSelThreads - 1) / kSelThreads;    // (token, pair of entries) per thread
+  const int tt0 = tid / HC, cp = (tid % HC) * 2, cc = c0 + cp;
+  const bool in0 = cc < I && tt0 < TT, in1 = cc + 1 < I;
+  const float bias0 = in0 ? p.bias[cc] : 0.f, bias1 = in0 && in1 ? p.bias[cc + 1] : 0.f;
+  const float d0 = (OUT && in0) ? p.d[cc] : 0.f, d1 = (OUT && in0 && in1) ? p.d[cc + 1] : 0.f;
+  SelPair<S> rx[PX], rd[PX], rz[OUT ? PX : 1];      // the next tile as it lies in memory
+  SelPair<S> rb[PB], rc[PB];
+  SelPair<S> xw[OUT ? PX : 1], zw[OUT ? PX : 1];    // x and z of the tile that is walked
+  SelPair<S> xg[OUT ? PX : 1], zg[OUT ? PX : 1];    // ... and of the one before it
+  const bool whole = in1 && p.pairs, bwhole = p.bc_pairs != 0;
+  const S* xs = static_cast<const S*>(p.x) + static_cast<long long>(t0 + tt0) * p.ld_x + (in0 ? cc : 0);
+  const S* ds = static_cast<const S*>(p.raw) + static_cast<long long>(t0 + tt0) * p.ld_raw + (in0 ? cc : 0);
+  const S* zs = OUT ? static_cast<const S*>(p.z) + static_cast<long long>(t0 + tt0) * p.ld_z + (in0 ? cc : 0) : nullptr;
+  const S* ls = static_cast<const S*>(p.low) + static_cast<long long>(t0) * p.ld_low;
+  auto request = [&](int tile) {
+    const int left = t1 - t0 - tile * TT;  // the chunk's tokens from the tile's first on
 #pragma unroll
-    for (int i = 0; i < NPT; ++i) f[i] = static_cast<float>(st[i]);
-    sel_st_state<NPT>(dst, q * NPT, N, svec, f);
+    for (int r = 0; r < PX; ++r) {
+      if (in0 && tt0 + r * TSTEP < left) {
+        sel_ld_pair(xs + r * TSTEP * p.ld_x, whole, in1, rx[r]);
+        sel_ld_pair(ds + r * TSTEP * p.ld_raw, whole, in1, rd[r]);
+        if (OUT) sel_ld_pair(zs + r * TSTEP * p.ld_z, whole, in1, rz[OUT ? r : 0]);
+      } else {
+        sel_zero(rx[r]);
+        sel_zero(rd[r]);
+        if (OUT) sel_zero(rz[OUT ? r : 0]);
+      }
+    }
+#pragma unroll
+    for (int r = 0; r < PB; ++r) {
+      const int e = r * kSelThreads + tid, tt = e / HB, n = (e % HB) * 2;
+      if (tt < TT && tt < left && n < N) {
+        const S* row = ls + tt * p.ld_low + n;
+        sel_ld_pair(row + p.off_b, bwhole, n + 1 < N, rb[r]);
+        if (OUT) sel_ld_pair(row + p.off_c, bwhole, n + 1 < N, rc[r]);
+      } else {
+        sel_zero(rb[r]);
+        if (OUT) sel_zero(rc[r]);
+      }
+      if (!OUT) sel_zero(rc[r]);
+    }
+    xs += TT * p.ld_x;
+    ds += TT * p.ld_raw;
+    if (OUT) zs += TT * p.ld_z;
+    ls += TT * p.ld_low;
+  };
+  auto stage = [&](int tile) {
+    const int buf = tile & 1, left = t1 - t0 - tile * TT;
+#pragma unroll
+    for (int r = 0; r < PX; ++r) {
+      const int tt = tt0 + r * TSTEP;
+      if (OUT) {
+        xg[OUT ? r : 0] = xw[OUT ? r : 0];
+        zg[OUT ? r : 0] = zw[OUT ? r : 0];
+        xw[OUT ? r : 0] = rx[r];
+        zw[OUT ? r : 0] = rz[OUT ? r : 0];
+      }
+      if (TT * HC < kSelThreads && tt >= TT) continue;
+      const float2 x = rx[r].get(), raw = rd[r].get();
+      // (tokens past the chunk's end: dt = 0 leaves the state as it is)
+      const ACC dt0 = tt < left ? sel_softplus(static_cast<ACC>(raw.x) + static_cast<ACC>(bias0)) : static_cast<ACC>(0);
+      const ACC dt1 = tt < left ? sel_softplus(static_cast<ACC>(raw.y) + static_cast<ACC>(bias1)) : static_cast<ACC>(0);
+      s_du[buf][tt][cp] = {dt0, dt0 * static_cast<ACC>(x.x)};
+      s_du[buf][tt][cp + 1] = {dt1, dt1 * static_cast<ACC>(x.y)};
+    }
+#pragma unroll
+    for (int r = 0; r < PB; ++r) {
+      const int e = r * kSelThreads + tid, tt = e / HB, n = (e % HB) * 2;
+      if (tt < TT) {
+        const float2 b = rb[r].get(), c = rc[r].get();
+        *reinterpret_cast<float4*>(&s_bc[buf][tt][n]) = make_float4(b.x, c.x, b.y, c.y);
+      }
+    }
+  };
+  auto finish = [&](int tile, const SelPair<S>* xr, const SelPair<S>* zr) {  // the tile's outputs
+    const int buf = tile & 1, base = t0 + tile * TT;
+#pragma unroll
+    for (int r = 0; r < PX; ++r) {
+      const int tt = tt0 + r * TSTEP;
+      if (!in0 || base + tt >= t1 || tt >= TT) continue;
+      const float2 x = xr[r].get(), z = zr[r].get();
+      const ACC y0 = static_cast<ACC>(d0) * static_cast<ACC>(x.x) + s_y[buf][OUT ? tt : 0][cp];
+      const ACC y1 = static_cast<ACC>(d1) * static_cast<ACC>(x.y) + s_y[buf][OUT ? tt : 0][cp + 1];
+      const float o0 = static_cast<float>(y0) * (sizeof(S) == 2 ? silu_fast(z.x) : silu_f(z.x));
+      const float o1 = static_cast<float>(y1) * (sizeof(S) == 2 ? silu_fast(z.y) : silu_f(z.y));
+      S* dst = static_cast<S*>(p.y) + static_cast<size_t>(base + tt) * I + cc;
+      if (sizeof(S) == 2 && whole) {
+        *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(o0, o1);
+      } else {
+        stf(dst, o0);
+        if (in1) stf(dst + 1, o1);
+      }
+    }
+  };
+  request(0);
+  stage(0);
+  request(1);
+  sel_barrier();
+  for (int tile = 0; tile < n_tiles; ++tile) {
+    if (OUT && tile > 0) finish(tile - 1, xg, zg);
+    if (tile + 1 < n_tiles) {
+      stage(tile + 1);  // (what is walked now becomes xg, zg)
+      request(tile + 2);
+    }
+    sel_barrier();
   }
-  if (!OUT && q == 0) p.chunk_dt[static_cast<size_t>(blockIdx.y) * I + c] = static_cast<float>(dt_sum);
+  if (OUT) finish(n_tiles - 1, xw, zw);
 }
 
 // A thread per state entry of a sequence of several chunks: chunk_state becomes the chunks' start states.
@@ -372,33 +494,40 @@ __global__ void __launch_bounds__(kSelThreads) selective_step_kernel(const SelAr
   }
 }
 
-// Lanes per channel and entries per lane for N state entries.
+// Lanes per channel of the walk for N state entries.
+inline int sel_walk_lanes(int N) { return N <= 8 ? 4 : N <= 32 ? 8 : 16; }
+
+template <typename S, bool OUT>
+int launch_selective_walk(const SelArgs& p, int n_chunks, cudaStream_t stream) {
+  using ACC = typename std::conditional<sizeof(S) == 4, double, float>::type;
+  const int ch = kSelThreads / sel_walk_lanes(p.N);
+  dim3 grid((p.I + ch - 1) / ch, n_chunks);
+  // (no programmatic launch: blocks that start while the kernel before still holds part of the GPU pile up on the SMs it
+  // has left, and this kernel lives from one long walk per SM)
+#define PMM_SEL_WALK(LN, NPT) selective_walk_kernel<S, ACC, LN, NPT, OUT><<<grid, kSelWalkThreads, 0, stream>>>(p)
+  if (p.N <= 8) PMM_SEL_WALK(4, 2);
+  else if (p.N <= 16) PMM_SEL_WALK(8, 2);
+  else if (p.N <= 32) PMM_SEL_WALK(8, 4);
+  else if (p.N <= 64) PMM_SEL_WALK(16, 4);
+  else if (p.N <= 128) PMM_SEL_WALK(16, 8);
+  else PMM_SEL_WALK(16, 16);
+#undef PMM_SEL_WALK
+  return launch_status();
+}
+
+// Lanes per channel and entries per lane of the single step.
 #define PMM_SEL_DISPATCH(N, CALL)      \
   do {                                 \
     if ((N) <= 4) { CALL(4, 1); }      \
     else if ((N) <= 8) { CALL(4, 2); } \
-    else if ((N) <= 12) { CALL(4, 3); } \
     else if ((N) <= 16) { CALL(4, 4); } \
-    else if ((N) <= 24) { CALL(8, 3); } \
     else if ((N) <= 32) { CALL(8, 4); } \
-    else if ((N) <= 48) { CALL(16, 3); } \
     else if ((N) <= 64) { CALL(16, 4); } \
     else if ((N) <= 128) { CALL(16, 8); } \
     else { CALL(16, 16); }             \
   } while (0)
 
 inline int sel_lanes(int N) { return N <= 16 ? 4 : N <= 32 ? 8 : 16; }
-
-template <typename S, bool OUT>
-int launch_selective_walk(const SelArgs& p, int n_chunks, cudaStream_t stream) {
-  using ACC = typename std::conditional<sizeof(S) == 4, double, float>::type;
-  const int ch = kSelThreads / sel_lanes(p.N);
-  dim3 grid((p.I + ch - 1) / ch, n_chunks);
-#define PMM_SEL_WALK(LN, NPT) launch_pdl(selective_walk_kernel<S, ACC, LN, NPT, OUT>, grid, dim3(kSelThreads), 0, stream, p)
-  PMM_SEL_DISPATCH(p.N, PMM_SEL_WALK);
-#undef PMM_SEL_WALK
-  return launch_status();
-}
 
 template <typename S>
 int launch_selective_step(const SelArgs& p, int vec, cudaStream_t stream) {
@@ -414,7 +543,7 @@ int launch_selective_step(const SelArgs& p, int vec, cudaStream_t stream) {
 }  // namespace pmm
 
 // Channels of one block of the walk (for the host's choice of chunks).
-PMM_EXPORT int pmm_selective_scan_channels(int N) { return N <= 0 || N > 256 ? 0 : pmm::kSelThreads / pmm::sel_lanes(N); }
+PMM_EXPORT int pmm_selective_scan_channels(int N) { return N <= 0 || N > 256 ? 0 : pmm::kSelThreads / pmm::sel_walk_lanes(N); }
 
 // x, raw, z [T, I] and low (B at off_b, C at off_c) in the storage type, unit column stride; y [T, I] contiguous.  n_chunks: at least
 // sum over the sequences of ceil(tokens / chunk_len).  multi: some sequence may have more than one chunk (then chunk_state
@@ -428,7 +557,10 @@ PMM_EXPORT int pmm_selective_scan(const void* x, long long ld_x, const void* raw
   if (I <= 0 || N <= 0 || N > 256 || chunk_len <= 0 || n_chunks > 65535 || n_seq > 65535) return PMM_ERR_BAD_ARGUMENT;
   if (multi && (!chunk_state || !chunk_dt || dtype != PMM_DTYPE_BF16)) return PMM_ERR_BAD_ARGUMENT;
   pmm::SelArgs p{x, raw, low, z, ld_x, ld_raw, ld_low, ld_z, off_b, off_c, bias, a_log, d, state, chunk_state, chunk_dt, cu,
-                 slots, y, n_seq, I, N, chunk_len, nullptr, 0};
+                 slots, y, n_seq, I, N, chunk_len, nullptr, 0, 0, 0};
+  auto even = [&](const void* q, long long ld) { return reinterpret_cast<uintptr_t>(q) % 4 == 0 && ld % 2 == 0; };
+  p.pairs = even(x, ld_x) && even(raw, ld_raw) && even(z, ld_z) && even(y, I);
+  p.bc_pairs = even(low, ld_low) && off_b % 2 == 0 && off_c % 2 == 0 && N % 2 == 0;
   if (multi) {
     int rc = pmm::launch_selective_walk<__nv_bfloat16, false>(p, n_chunks, stream);
     if (rc != 0) return rc;
@@ -449,7 +581,7 @@ PMM_EXPORT int pmm_selective_step(const void* x, long long ld_x, const void* low
   if (n_seq <= 0) return 0;
   if (I <= 0 || N <= 0 || N > 256 || R <= 0 || n_seq > 65535) return PMM_ERR_BAD_ARGUMENT;
   pmm::SelArgs p{x, nullptr, low, z, ld_x, 0, ld_low, ld_z, off_b, off_c, bias, a_log, d, state, nullptr, nullptr, nullptr,
-                 slots, y, n_seq, I, N, 0, w_dt, R};
+                 slots, y, n_seq, I, N, 0, w_dt, R, 0, 0};
   const int vec = R % 8 == 0 && ld_low % 8 == 0 && reinterpret_cast<uintptr_t>(low) % 16 == 0 && reinterpret_cast<uintptr_t>(w_dt) % 16 == 0;
   PMM_DISPATCH_DTYPE(dtype, S, return pmm::launch_selective_step<S>(p, vec, stream));
   return 0;

@@ -870,20 +870,19 @@ def ssm_scan_tc(xbc: Tensor, dt_raw: Tensor, dt_scale: float, dt_shift: Tensor, 
 
 # ----------------------------------------------------------------------------- selective scan
 SELECTIVE_MAX_STATE = 256
-_SELECTIVE_FULL_WARPS = 1200  # warps of one walk (4 a block) from which the GPU is busy without chunks
 _SELECTIVE_MIN_CHUNK = 64
 
 
 def selective_scan_plan(new_lens: Sequence[int], inner: int, d_state: int, dtype: torch.dtype) -> Tuple[int, int]:
     """(tokens per chunk, upper bound of chunks) for a step's portions.  One walk per channel where the channels and
-    sequences fill the GPU, or where two chunks would (a chunked walk makes every exponential twice); else as many
-    chunks as fill it.  Float32 walks are never cut."""
+    sequences give a block to at least a quarter of the SMs or so (a chunked walk makes every exponential twice); else as
+    many chunks as give every SM two.  Float32 walks are never cut."""
     longest = max(new_lens)
     chunk = longest
     if dtype == torch.bfloat16 and longest > _SELECTIVE_MIN_CHUNK:
-        warps = 4 * -(-inner // selective_scan_channels(d_state)) * sum(1 for n in new_lens if n > longest // 2)
-        want = _SELECTIVE_FULL_WARPS // warps
-        if want >= 3:
+        blocks = -(-inner // selective_scan_channels(d_state)) * sum(1 for n in new_lens if n > longest // 2)
+        want = 296 // blocks
+        if want >= 6:
             chunk = max(_SELECTIVE_MIN_CHUNK, (-(-longest // want) + 15) // 16 * 16)
     return chunk, sum(-(-n // chunk) for n in new_lens)
 
