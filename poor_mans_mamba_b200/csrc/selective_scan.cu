@@ -20,7 +20,7 @@
 //   walk          every chunk from its start state, with the outputs
 // (two exponentials per entry instead of one); else the walk starts from the request's state.  The float storage
 // type walks in double, unchunked.  One token per sequence (decode): selective_step, which also makes the channel's
-// raw step size from the low-rank row, raw_c = W_dt[c] . low[:R].
+// raw step size from the low-rank row, raw_c = W_dt[c] . low[:R], unless it is given.
 #include "common.cuh"
 #include <type_traits>
 
@@ -427,71 +427,96 @@ __device__ __forceinline__ void sel_ld8(const __nv_bfloat16* p, float* o) {
     o[2 * i + 1] = f.y;
   }
 }
+// NPT neighbouring entries of B or C of a token (0 beyond N); vec: N a multiple of 4, pieces of 4 aligned.
+template <int NPT>
+__device__ __forceinline__ void sel_ld_row(const __nv_bfloat16* row, int n0, int N, bool vec, float* o) {
+  if (NPT % 4 == 0 && vec) {
+#pragma unroll
+    for (int i = 0; i < NPT; i += 4) {
+      uint2 raw = make_uint2(0u, 0u);
+      if (n0 + i < N) raw = *reinterpret_cast<const uint2*>(row + n0 + i);
+      const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+      const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+      o[i] = a.x; o[i + 1] = a.y; o[i + 2] = b.x; o[i + 3] = b.y;
+    }
+    return;
+  }
+#pragma unroll
+  for (int i = 0; i < NPT; ++i) o[i] = n0 + i < N ? __bfloat162float(row[n0 + i]) : 0.f;
+}
+template <int NPT>
+__device__ __forceinline__ void sel_ld_row(const float* row, int n0, int N, bool, float* o) {
+#pragma unroll
+  for (int i = 0; i < NPT; ++i) o[i] = n0 + i < N ? row[n0 + i] : 0.f;
+}
 __device__ __forceinline__ void sel_ld8(const float* p, float* o) {
 #pragma unroll
   for (int i = 0; i < 8; ++i) o[i] = p[i];
 }
 
-// One token per sequence: token s of sequence s.  vec: rows of low and W_dt in whole pieces of 8 elements.
+// One token per sequence: token s of sequence s.  vec: rows of low and W_dt in whole pieces of 8 elements.  (A block for
+// several sequences, which would read the channel's constants once for all of them, was slower: 20 us for two and 27
+// for four against 17, at 64 sequences of 6,144 channels.)
 template <typename S, typename ACC, int LN, int NPT>
 __global__ void __launch_bounds__(kSelThreads) selective_step_kernel(const SelArgs p, int vec) {
   constexpr int CH = kSelThreads / LN;
   pdl_launch_dependents();
   const int ch = threadIdx.x / LN, q = threadIdx.x % LN;
-  const int c = blockIdx.x * CH + ch;
-  const int s = blockIdx.y;
+  const int c = blockIdx.x * CH + ch, s = blockIdx.y;
   const int N = p.N, I = p.I;
-  const bool ok = c < I;
-  const int cs = ok ? c : 0;
+  const bool ok = c < I, svec = N % 4 == 0;
+  const int cs = ok ? c : 0, n0 = q * NPT;
   ACC a2[NPT];
+  {
+    float al[NPT];
+    sel_ld_state<NPT>(p.a_log + static_cast<size_t>(cs) * N, n0, N, svec, al);
 #pragma unroll
-  for (int i = 0; i < NPT; ++i) {
-    const int n = q * NPT + i;
-    a2[i] = (ok && n < N) ? static_cast<ACC>(-1.4426950408889634) * scan_exp(static_cast<ACC>(p.a_log[static_cast<size_t>(cs) * N + n])) : static_cast<ACC>(0);
+    for (int i = 0; i < NPT; ++i) a2[i] = static_cast<ACC>(-1.4426950408889634) * scan_exp(static_cast<ACC>(al[i]));
   }
   const ACC bias = p.bias[cs], dskip = p.d[cs];
-  const int slot = p.slots[s];
+  float* srow = p.state + (static_cast<size_t>(p.slots[s]) * I + cs) * N;
   pdl_wait();
-  float* srow = p.state + (static_cast<size_t>(slot) * I + cs) * N;
-  const bool svec = N % 4 == 0;
-  float st[NPT];
-  sel_ld_state<NPT>(srow, q * NPT, N, svec, st);
+  float st[NPT], bv[NPT], cv[NPT];
+  sel_ld_state<NPT>(srow, n0, N, svec, st);
   const S* low = static_cast<const S*>(p.low) + static_cast<long long>(s) * p.ld_low;
-  const S* w = static_cast<const S*>(p.w_dt) + static_cast<size_t>(cs) * p.R;
-  ACC raw = 0;
-  if (vec) {
-    for (int r = q * 8; r < p.R; r += LN * 8) {
-      float lv[8], wv[8];
-      sel_ld8(low + r, lv);
-      sel_ld8(w + r, wv);
-#pragma unroll
-      for (int i = 0; i < 8; ++i) raw += static_cast<ACC>(lv[i]) * static_cast<ACC>(wv[i]);
-    }
-  } else {
-    for (int r = q; r < p.R; r += LN) raw += static_cast<ACC>(ldf(low + r)) * static_cast<ACC>(ldf(w + r));
-  }
-#pragma unroll
-  for (int o = LN / 2; o > 0; o >>= 1) raw += __shfl_xor_sync(0xffffffffu, raw, o);
-  const ACC dt = scan_softplus<ACC>(raw + bias);
+  const bool bvec = svec && vec && p.off_b % 4 == 0 && p.off_c % 4 == 0;
+  sel_ld_row<NPT>(low + p.off_b, n0, N, bvec, bv);
+  sel_ld_row<NPT>(low + p.off_c, n0, N, bvec, cv);
   const ACC xv = ldf(static_cast<const S*>(p.x) + static_cast<long long>(s) * p.ld_x + cs);
+  const float zv = ldf(static_cast<const S*>(p.z) + static_cast<long long>(s) * p.ld_z + cs);
+  ACC raw = 0;
+  if (p.raw) {
+    raw = ldf(static_cast<const S*>(p.raw) + static_cast<long long>(s) * p.ld_raw + cs);
+  } else {
+    const S* w = static_cast<const S*>(p.w_dt) + static_cast<size_t>(cs) * p.R;
+    if (vec) {
+      for (int r = q * 8; r < p.R; r += LN * 8) {
+        float wv[8], lv[8];
+        sel_ld8(w + r, wv);
+        sel_ld8(low + r, lv);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) raw += static_cast<ACC>(lv[i]) * static_cast<ACC>(wv[i]);
+      }
+    } else {
+      for (int r = q; r < p.R; r += LN) raw += static_cast<ACC>(ldf(low + r)) * static_cast<ACC>(ldf(w + r));
+    }
+#pragma unroll
+    for (int o = LN / 2; o > 0; o >>= 1) raw += __shfl_xor_sync(0xffffffffu, raw, o);
+  }
+  const ACC dt = sel_softplus(raw + bias);
   const ACC u = dt * xv;
   ACC acc = 0;
 #pragma unroll
   for (int i = 0; i < NPT; ++i) {
-    const int n = q * NPT + i;
-    if (ok && n < N) {
-      const ACC v = sel_exp2(dt * a2[i]) * static_cast<ACC>(st[i]) + u * static_cast<ACC>(ldf(low + p.off_b + n));
-      acc += v * static_cast<ACC>(ldf(low + p.off_c + n));
-      st[i] = static_cast<float>(v);
-    }
+    const ACC v = sel_exp2(dt * a2[i]) * static_cast<ACC>(st[i]) + u * static_cast<ACC>(bv[i]);
+    acc += v * static_cast<ACC>(cv[i]);
+    st[i] = static_cast<float>(v);
   }
-  if (ok) sel_st_state<NPT>(srow, q * NPT, N, svec, st);
 #pragma unroll
   for (int o = LN / 2; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
-  if (ok && q == 0) {
-    const float zv = ldf(static_cast<const S*>(p.z) + static_cast<long long>(s) * p.ld_z + c);
-    stf(static_cast<S*>(p.y) + static_cast<size_t>(s) * I + c, static_cast<float>(acc + dskip * xv) * silu_f(zv));
-  }
+  if (!ok) return;
+  sel_st_state<NPT>(srow, n0, N, svec, st);
+  if (q == 0) stf(static_cast<S*>(p.y) + static_cast<size_t>(s) * I + c, static_cast<float>(acc + dskip * xv) * silu_f(zv));
 }
 
 // Lanes per channel of the walk for N state entries.
@@ -573,14 +598,14 @@ PMM_EXPORT int pmm_selective_scan(const void* x, long long ld_x, const void* raw
 }
 
 // One token per sequence.  low [n_seq, ...]: the low-rank row of the step sizes in columns 0 .. R - 1, B at off_b, C at off_c;
-// w_dt [I, R] contiguous.
-PMM_EXPORT int pmm_selective_step(const void* x, long long ld_x, const void* low, long long ld_low, int R, int off_b, int off_c,
+// w_dt [I, R] contiguous.  raw [n_seq, I]: the raw step sizes, made already (w_dt and R are then not used); or nullptr.
+PMM_EXPORT int pmm_selective_step(const void* x, long long ld_x, const void* raw, long long ld_raw, const void* low, long long ld_low, int R, int off_b, int off_c,
                                   const void* w_dt, const void* z, long long ld_z, const float* bias, const float* a_log,
                                   const float* d, float* state, const int* slots, void* y, int n_seq, int I, int N, int dtype,
                                   cudaStream_t stream) {
   if (n_seq <= 0) return 0;
-  if (I <= 0 || N <= 0 || N > 256 || R <= 0 || n_seq > 65535) return PMM_ERR_BAD_ARGUMENT;
-  pmm::SelArgs p{x, nullptr, low, z, ld_x, 0, ld_low, ld_z, off_b, off_c, bias, a_log, d, state, nullptr, nullptr, nullptr,
+  if (I <= 0 || N <= 0 || N > 256 || (!raw && (R <= 0 || !w_dt)) || n_seq > 65535) return PMM_ERR_BAD_ARGUMENT;
+  pmm::SelArgs p{x, raw, low, z, ld_x, ld_raw, ld_low, ld_z, off_b, off_c, bias, a_log, d, state, nullptr, nullptr, nullptr,
                  slots, y, n_seq, I, N, 0, w_dt, R, 0, 0};
   const int vec = R % 8 == 0 && ld_low % 8 == 0 && reinterpret_cast<uintptr_t>(low) % 16 == 0 && reinterpret_cast<uintptr_t>(w_dt) % 16 == 0;
   PMM_DISPATCH_DTYPE(dtype, S, return pmm::launch_selective_step<S>(p, vec, stream));

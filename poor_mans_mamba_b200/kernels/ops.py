@@ -41,7 +41,7 @@ _SIGNATURES = {
     "pmm_selective_scan": [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_int, c_void_p, c_longlong,
                            c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                            c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
-    "pmm_selective_step": [c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p, c_longlong,
+    "pmm_selective_step": [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p, c_longlong,
                            c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
     "pmm_scale_f32": [c_void_p, c_float, c_longlong, c_void_p],
     "pmm_cast_scale": [c_void_p, c_void_p, c_float, c_longlong, c_int, c_void_p],
@@ -945,15 +945,19 @@ def selective_scan(x: Tensor, raw: Tensor, low: Tensor, off_b: int, off_c: int, 
 
 
 def selective_step(x: Tensor, low: Tensor, rank: int, off_b: int, off_c: int, w_dt: Tensor, z: Tensor, bias: Tensor,
-                   a_log: Tensor, d_skip: Tensor, state: Tensor, slots: Tensor, out: Tensor) -> None:
+                   a_log: Tensor, d_skip: Tensor, state: Tensor, slots: Tensor, out: Tensor,
+                   raw: Optional[Tensor] = None) -> None:
     """selective_scan for one token per sequence, with the raw step sizes made in the same launch: raw = low[:, :rank] @
-    w_dt^T, w_dt [I, rank]."""
-    _cuda(x, low, w_dt, z, bias, a_log, d_skip, state, slots, out)
+    w_dt^T, w_dt [I, rank]; or given as ``raw`` [T, I]."""
+    _cuda(x, low, w_dt, z, bias, a_log, d_skip, state, slots, out, raw)
+    if raw is not None and not (raw.shape == x.shape and raw.dtype == x.dtype):
+        raise KernelError("selective_step: raw step sizes [T, I] of x's type")
     I, N = _selective_common(x, low, z, bias, a_log, d_skip, state, slots, off_b, off_c, out, "selective_step")
     if not (w_dt.shape == (I, rank) and w_dt.is_contiguous() and w_dt.dtype == x.dtype and rank <= low.shape[1]
             and slots.numel() == x.shape[0]):
         raise KernelError("selective_step: w_dt contiguous [I, rank] of x's type, one slot per token")
-    _call("pmm_selective_step", x.data_ptr(), _rows_view(x, "selective_step: x"), low.data_ptr(), _rows_view(low, "selective_step: low"),
+    _call("pmm_selective_step", x.data_ptr(), _rows_view(x, "selective_step: x"), _ptr(raw),
+          0 if raw is None else _rows_view(raw, "selective_step: raw"), low.data_ptr(), _rows_view(low, "selective_step: low"),
           int(rank), int(off_b), int(off_c), w_dt.data_ptr(), z.data_ptr(), _rows_view(z, "selective_step: z"), bias.data_ptr(),
           a_log.data_ptr(), d_skip.data_ptr(), state.data_ptr(), slots.data_ptr(), out.data_ptr(), x.shape[0], I, N, _dt(x),
           _stream())

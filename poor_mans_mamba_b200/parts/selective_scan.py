@@ -10,7 +10,7 @@ State per request (float32, in a slot, zero for a new request): S [inner, state]
 the convolution.  The step sizes, decays, the state and its read-out are float arithmetic in both storage
 types; the projections, the convolution and the gate have the storage type.  W_x is stored with zero rows
 behind the step sizes' rows and at its end, so that t, B and C start on 16-byte boundaries, and W_dt with zero
-columns to match.  A decode step makes W_dt t inside the scan's launch.
+columns to match.  A decode step of few requests makes W_dt t inside the scan's launch.
 """
 from __future__ import annotations
 
@@ -24,6 +24,13 @@ from .base import ParamSpec, StateSpec, register_mixer
 from .recurrent import _StackedInput
 
 Tensor = torch.Tensor
+
+
+# From this many (request, rank) products on, a decode step makes its step sizes by a product of their own: every
+# request of the scan's launch would read W_dt again.  Measured (us, in the launch / product and launch): 16 requests of
+# 6,144 channels and rank 192 9.9 / 8.0, 8 of them 6.4 / 6.0; 32 requests of 2,048 channels and rank 64 5.4 / 6.2, 64 of
+# them 9.0 / 9.0.
+_OWN_PRODUCT_FROM = 2560
 
 
 def _up8(n: int) -> int:
@@ -94,8 +101,12 @@ class SelectiveScanMixer(_StackedInput):
         if ctx.decode_only:
             K.conv1d_decode(raw_x, self.conv_ones, None, self.conv_w, self.conv_b, window, ctx.slots, x)
             streaming.linear(x, self.w_x, low, ctx)
+            raw_dt = None
+            if T * self.dt_rank >= _OWN_PRODUCT_FROM:
+                raw_dt = ws.alloc((T, I), proj.dtype)
+                streaming.linear(low[:, :self.rank_padded], self.w_dt, raw_dt, ctx)
             K.selective_step(x, low, self.rank_padded, self.off_b, self.off_c, self.w_dt, z, self.dt_bias, self.a_log,
-                             self.d_skip, state, ctx.slots, y)
+                             self.d_skip, state, ctx.slots, y, raw=raw_dt)
             return y
         K.conv1d_fwd(raw_x, self.conv_ones, None, self.conv_w, self.conv_b, window, ctx.seq_of, ctx.cu_seqlens, ctx.slots, x,
                      weight_t=self.conv_w_t)

@@ -276,24 +276,34 @@ def test_scan_plan_cuts_only_where_the_gpu_would_stay_empty():
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("n", [3, 18])
 @pytest.mark.parametrize("I,N,R", [(40, 12, 5), (96, 16, 8), (33, 1, 3), (64, 40, 24), (24, 128, 64), (10, 256, 1)])
-def test_selective_step_makes_its_step_sizes(dtype, I, N, R):
-    n, slots = 3, [2, 0, 3]
+def test_selective_step_makes_its_step_sizes(dtype, I, N, R, n):
+    slots = [(5 * s + 2) % (n + 1) for s in range(n)] if n == 18 else [2, 0, 3]
     x, z, _, B, Cm, a_log, bias, d = (t.to(dtype).float() if i < 5 else t for i, t in enumerate(scan_inputs(n, I, N, R)))
     t_low, w_dt = rnd(n, R, seed=60), rnd(I, R, seed=61, scale=R ** -0.5)
     off_b, off_c = (R + 7) // 8 * 8, (R + 7) // 8 * 8 + (N + 7) // 8 * 8
     low = torch.zeros(n, off_c + (N + 7) // 8 * 8)
     low[:, :R], low[:, off_b:off_b + N], low[:, off_c:off_c + N] = t_low, B, Cm
-    state0 = rnd(4, I, N, seed=50)
+    state0 = rnd(n + 1, I, N, seed=50)
     state, y = state0.to(DEV).clone(), torch.empty(n, I, dtype=dtype, device=DEV)
     K.selective_step(x.to(DEV, dtype), low.to(DEV, dtype), R, off_b, off_c, w_dt.to(DEV, dtype), z.to(DEV, dtype), bias.to(DEV),
                      a_log.to(DEV), d.to(DEV), state, i32(slots), y)
     raw = t_low.double() @ w_dt.double().t()
+    given = raw.to(dtype)      # the same with the step sizes made before
+    state2, y2 = state0.to(DEV).clone(), torch.empty(n, I, dtype=dtype, device=DEV)
+    K.selective_step(x.to(DEV, dtype), low.to(DEV, dtype), R, off_b, off_c, w_dt.to(DEV, dtype), z.to(DEV, dtype), bias.to(DEV),
+                     a_log.to(DEV), d.to(DEV), state2, i32(slots), y2, raw=given.to(DEV))
+    for s in range(n):
+        want, S = plain_scan(x[s:s + 1], z[s:s + 1], given.double()[s:s + 1], B[s:s + 1], Cm[s:s + 1], a_log, bias, d, state0[slots[s]])
+        close(y2[s:s + 1], want, dtype, "step, sizes given", bf16=1e-2)
+        close(state2[slots[s]], S, torch.float32, "state, sizes given")
     for s in range(n):
         want, S = plain_scan(x[s:s + 1], z[s:s + 1], raw[s:s + 1], B[s:s + 1], Cm[s:s + 1], a_log, bias, d, state0[slots[s]])
         close(y[s:s + 1], want, dtype, "step", bf16=1e-2)
         close(state[slots[s]], S, torch.float32, "state")
-    assert torch.equal(state[1].cpu(), state0[1])
+    left = (set(range(n + 1)) - set(slots)).pop()
+    assert torch.equal(state[left].cpu(), state0[left])
 
 
 # ----------------------------------------------------------------------------- attention
