@@ -2,11 +2,12 @@
 sequence, slots for per-request state of fixed size.
 
 Layers declare what they keep (StateSpec).  Paged states with the same row layout and
-window form a *group*: the group has pages of its own ([member, page, plane, page_size,
+window (or chunk) form a *group*: the group has pages of its own ([member, page, plane, page_size,
 width] on the device, one member per layer state) and one block table per request, shared
 by the group's layers.  A group that only ever reads a window of the sequence gives pages
 back as soon as the window has passed them (all but the pages that hold the first tokens, where
-the group's layers keep those visible).  Fixed states live in slots ([slot, *shape]
+the group's layers keep those visible); one that only reads the chunk of the sequence a token lies in gives the
+pages before a chunk back when the sequence enters it.  Fixed states live in slots ([slot, *shape]
 per layer state; the states of one shape and dtype are slices of one tensor, so that admitting a
 request zeroes its slot in all layers with one fill per kind: 72 fills of the 36-layer model cost
 the host 0.5 ms per admitted request).  Everything a request holds is given back when it
@@ -37,6 +38,8 @@ def _dtype_of(spec_dtype: str, compute: torch.dtype) -> torch.dtype:
         return compute
     if spec_dtype == "float32":
         return torch.float32
+    if spec_dtype == "int32":
+        return torch.int32
     raise ValueError(f"unknown state dtype {spec_dtype!r}")
 
 
@@ -50,8 +53,11 @@ class PagedGroup:
     """Pages and block tables of the layer states that share one row layout and window."""
 
     def __init__(self, key: Tuple, planes: int, width: int, window: int, page_size: int, num_pages: int,
-                 keep_first: int = 0):
+                 keep_first: int = 0, chunk: int = 0):
+        if window > 0 and chunk > 0:
+            raise ValueError("a state has a window or chunks, not both")
         self.key = key
+        self.chunk = chunk
         self.planes, self.width, self.window = planes, width, window
         self.keep_first = keep_first if window > 0 else 0
         self.page_size, self.num_pages = page_size, num_pages
@@ -65,9 +71,16 @@ class PagedGroup:
 
     def first_needed_block(self, next_pos: int) -> int:
         """The first logical block that a token at position >= next_pos can still read."""
+        if self.chunk > 0:
+            return next_pos // self.chunk * self.chunk // self.page_size
         if self.window <= 0:
             return 0
         return max(0, next_pos - self.window + 1) // self.page_size
+
+    @property
+    def bounded(self) -> bool:
+        """Whether pages are given back while a request lives (its tokens stop being read)."""
+        return self.window > 0 or self.chunk > 0
 
     def kept_blocks(self) -> int:
         """The logical blocks at the start of a request that are never given back."""
@@ -94,10 +107,12 @@ class CacheManager:
                     key = (spec.planes, spec.width, spec.window)
                     if spec.window > 0 and spec.keep_first > 0:
                         key += (spec.keep_first,)
+                    if spec.chunk > 0:
+                        key += ("chunk", spec.chunk)
                     if key not in self.groups:
                         n = (pages_per_group or {}).get(key, num_pages)
                         self.groups[key] = PagedGroup(key, spec.planes, spec.width, spec.window,
-                                                      self.page_size, int(n), spec.keep_first)
+                                                      self.page_size, int(n), spec.keep_first, spec.chunk)
                     g = self.groups[key]
                     self._paged_of[(layer, name)] = (g, len(g.members))
                     g.members.append(_Member(layer, name))
@@ -173,7 +188,7 @@ class CacheManager:
         """Give back the pages that no later token of ``req`` (position >= cur_len) can read."""
         n = 0
         for g in self.groups.values():
-            if g.window <= 0:
+            if not g.bounded:
                 continue
             table = g.tables[req]
             for b in range(g.kept_blocks(), min(g.first_needed_block(cur_len), len(table))):

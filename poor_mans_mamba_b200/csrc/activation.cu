@@ -200,3 +200,57 @@ PMM_EXPORT int pmm_clamped_glu(const void* gu, long long ld, float limit, float 
                                                static_cast<S*>(out), F));
   return pmm::launch_status();
 }
+
+namespace pmm {
+enum { kUnaryGelu = 0, kUnaryTanh = 1 };
+
+template <int OP>
+__device__ __forceinline__ float unary_f(float z) { return OP == kUnaryGelu ? gelu_erf_f(z) : tanhf(z); }
+
+// x = f(x) in place on rows of stride ld
+template <typename S, int OP>
+__global__ void unary_kernel(S* __restrict__ x, long long ld, int F) {
+  pdl_launch_dependents();
+  pdl_wait();
+  S* row = x + static_cast<long long>(blockIdx.x) * ld;
+  for (int f = blockIdx.y * blockDim.x + threadIdx.x; f < F; f += gridDim.y * blockDim.x) stf(row + f, unary_f<OP>(ldf(row + f)));
+}
+
+// bfloat16, F and ld multiples of 8, 16-byte aligned rows: eight elements per thread
+template <int OP>
+__global__ void unary_bf16x8_kernel(__nv_bfloat16* __restrict__ x, long long ld, int F) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __nv_bfloat16* row = x + static_cast<long long>(blockIdx.x) * ld;
+  for (int f = (blockIdx.y * blockDim.x + threadIdx.x) * 8; f < F; f += gridDim.y * blockDim.x * 8) {
+    uint4 v = *reinterpret_cast<const uint4*>(row + f);
+    __nv_bfloat162* v2 = reinterpret_cast<__nv_bfloat162*>(&v);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float2 z = __bfloat1622float2(v2[i]);
+      v2[i] = __floats2bfloat162_rn(unary_f<OP>(z.x), unary_f<OP>(z.y));
+    }
+    *reinterpret_cast<uint4*>(row + f) = v;
+  }
+}
+
+template <int OP>
+int launch_unary(void* x, long long ld, int T, int F, int dtype, cudaStream_t stream) {
+  if (dtype == PMM_DTYPE_BF16 && F % 8 == 0 && ld % 8 == 0 && reinterpret_cast<uintptr_t>(x) % 16 == 0) {
+    const int yt = min((F / 8 + 255) / 256, 64);
+    launch_pdl(unary_bf16x8_kernel<OP>, dim3(T, yt), dim3(256), 0, stream, static_cast<__nv_bfloat16*>(x), ld, F);
+    return launch_status();
+  }
+  const int yt = min((F + 1023) / 1024, 64);
+  PMM_DISPATCH_DTYPE(dtype, S, launch_pdl(unary_kernel<S, OP>, dim3(T, yt), dim3(256), 0, stream, static_cast<S*>(x), ld, F));
+  return launch_status();
+}
+}  // namespace pmm
+
+// op 0: the exact form of GELU; op 1: tanh.  x [T, F] rows of stride ld, in place.
+PMM_EXPORT int pmm_unary(int op, void* x, long long ld, int T, int F, int dtype, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (F <= 0 || op < 0 || op > 1) return PMM_ERR_BAD_ARGUMENT;
+  return op == pmm::kUnaryGelu ? pmm::launch_unary<pmm::kUnaryGelu>(x, ld, T, F, dtype, stream)
+                               : pmm::launch_unary<pmm::kUnaryTanh>(x, ld, T, F, dtype, stream);
+}

@@ -68,7 +68,7 @@ __global__ void __launch_bounds__(kAttnWarps * 32)
   const int hk = hq / (Hq / Hkv);
   const int pos = positions[t];
   const int* bt = block_table + static_cast<size_t>(seq_of[t]) * max_blocks;
-  int lo = window > 0 ? max(0, pos - window + 1) : 0;
+  int lo = first_visible(pos, window);
   if (lo <= keep_first) lo = 0;  // the kept first keys and the window are one range
   const int k_end = min(pos + 1, (z + 1) * split_len);
   // two key ranges within this split: the kept first keys (empty unless the window has left them), then the window

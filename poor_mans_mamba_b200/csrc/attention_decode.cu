@@ -139,7 +139,7 @@ __global__ void __launch_bounds__(kDaThreads)
   const int kv_dim = a.Hkv * DH;
   const int page_size = a.page_size;
   const int pos = a.positions[seq];
-  const int lo_all = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+  const int lo_all = first_visible(pos, a.window);
   const int k_begin = max(lo_all, z * a.split_len);
   const int k_end = min(pos + 1, (z + 1) * a.split_len);
   const int first_tile = (k_begin / KT) * KT;

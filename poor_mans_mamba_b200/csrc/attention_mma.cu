@@ -113,7 +113,7 @@ __global__ void __launch_bounds__(128)
 
   if (tid < M) s_pos[tid] = (tid < n_rows) ? positions[tok0 + tid / G] : -1;
   const int pos_min = positions[tok0], pos_max = positions[tok0 + n_tok - 1];
-  const int lo_all = window > 0 ? max(0, pos_min - window + 1) : 0;
+  const int lo_all = first_visible(pos_min, window);
   const int k_begin = max(lo_all, z * split_len);
   const int k_end = min(pos_max + 1, (z + 1) * split_len);
 
@@ -335,19 +335,20 @@ __global__ void __launch_bounds__(128)
     // per score).  A tile that every row of the block may read in full (inside the split, before
     // the first row's position, inside the last row's window) needs no mask.
     const bool full = base >= k_begin && base + KT <= k_end && base + KT - 1 <= pos_min &&
-                      (window <= 0 || base >= pos_max - window + 1);  // rows beyond the tile are never written out
+                      base >= first_visible(pos_max, window);  // rows beyond the tile are never written out
     unsigned pa[MT][KT / 16][4];  // P as bfloat16 A fragments
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt) {
       if (!full) {
         const int pos_lo = s_pos[row_base + mt * 16 + r_lo], pos_hi = s_pos[row_base + mt * 16 + r_hi];
+        const int lo_lo = max(first_visible(pos_lo, window), k_begin), lo_hi = max(first_visible(pos_hi, window), k_begin);
 #pragma unroll
         for (int nt = 0; nt < NT_S; ++nt) {
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
             const int key = base + nt * 8 + (lane & 3) * 2 + (e & 1);
             const int pos = (e < 2) ? pos_lo : pos_hi;
-            const int lo = window > 0 ? max(pos - window + 1, k_begin) : k_begin;
+            const int lo = (e < 2) ? lo_lo : lo_hi;
             const bool ok = pos >= 0 && key <= pos && key >= lo && key < k_end;
             if (!ok) s[mt][nt][e] = -CUDART_INF_F;
           }

@@ -116,7 +116,7 @@ __global__ void __launch_bounds__(kAtThreads, DH == 64 ? 2 : 1)
   const int n_rows = n_tok * G;
   const int* bt = block_table + static_cast<size_t>(seq) * max_blocks;
   const int pos_min = positions[tok0], pos_max = positions[tok0 + n_tok - 1];
-  const int lo_all = window > 0 ? max(0, pos_min - window + 1) : 0;
+  const int lo_all = first_visible(pos_min, window);
   const int k_begin = max(lo_all, z * split_len);
   const int k_end = min(pos_max + 1, (z + 1) * split_len);
   const int first = (k_begin / kAtBox) * kAtBox;  // boxes start on multiples of 64 keys: inside one page
@@ -255,7 +255,7 @@ __global__ void __launch_bounds__(kAtThreads, DH == 64 ? 2 : 1)
     const unsigned lane_base = tmem_base + (static_cast<unsigned>((warp & 3) * 32) << 16);
     const bool row_ok = row < n_rows;
     const int my_pos = row_ok ? positions[tok0 + row / G] : -1;
-    const int my_lo = window > 0 ? max(my_pos - window + 1, k_begin) : k_begin;
+    const int my_lo = max(first_visible(my_pos, window), k_begin);
     float m_run = -CUDART_INF_F, l_run = 0.f;  // the maximum in use (exponent's unit) and the sum against it
     bool alive = true;
     if (n_tiles > 0) {
@@ -288,7 +288,7 @@ __global__ void __launch_bounds__(kAtThreads, DH == 64 ? 2 : 1)
       mbar_arrive(&bar_sfree);
       // a tile that every row of the block may read in full needs no mask
       const bool full = base >= k_begin && base + kAtKeys <= k_end && base + kAtKeys - 1 <= pos_min &&
-                        (window <= 0 || base >= pos_max - window + 1);
+                        base >= first_visible(pos_max, window);
       if (!full) {
 #pragma unroll
         for (int e = 0; e < kAtKeys; ++e) {

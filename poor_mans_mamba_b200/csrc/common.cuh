@@ -49,11 +49,21 @@ __device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); 
 // of special-function work instead of a full-precision exponential and division.
 __device__ __forceinline__ float silu_fast(float x) { return __fdividef(x, 1.f + __expf(-x)); }
 
+// The exact (erf) form of GELU: z/2 (1 + erf(z / sqrt 2)).
+__device__ __forceinline__ float gelu_erf_f(float z) { return 0.5f * z * (1.f + erff(z * 0.70710678118654752f)); }
+
 // v if v>20; exp(v) if v<-20; log1p(exp(v)) otherwise.
 __device__ __forceinline__ float softplus_f(float v) {
   if (v > 20.f) return v;
   if (v < -20.f) return expf(v);
   return log1pf(expf(v));
+}
+
+// The first key that the token at `pos` may see: window > 0 the last `window` keys, window < 0 the keys of its own
+// chunk of -window positions (counted from position 0), window == 0 every key.  Does not fall as pos grows.
+__device__ __forceinline__ int first_visible(int pos, int window) {
+  if (window > 0) return max(0, pos - window + 1);
+  return window < 0 ? pos - pos % -window : 0;
 }
 
 // Softplus and exponential of the recurrences' walks, in the type the walk computes in (float, or double for the

@@ -12,11 +12,24 @@ namespace pmm {
 
 // norm_w != nullptr: the row is divided by its root mean square and multiplied by norm_w,
 //   h[t] = r / sqrt(mean(r^2) + eps) * norm_w with r = mult * E[tok[t]], all in float.
+// bigram.table != nullptr: r is mult * E[tok[t]] + B[row], row = (previous token * mul_prev + token * mul_cur) mod
+//   buckets, or `buckets` (the last row) for a sequence's first token.  previous [slots] holds a request's last token
+//   plus one (zero: none yet): the block of a sequence's first token of the step reads it and then leaves the step's
+//   last token there; the blocks of the other tokens read the token before theirs in the batch.
+struct Bigram {
+  const void* table;
+  long long mul_prev, mul_cur;
+  int buckets;
+  int* previous;
+  const int *seq_of, *cu, *slots;
+};
+
 template <typename S>
 __global__ void embed_kernel(float* __restrict__ out, const S* __restrict__ table,
                              const int* __restrict__ tokens, float mult, int D, int V,
-                             const float* __restrict__ norm_w, float eps) {
+                             const float* __restrict__ norm_w, float eps, const Bigram bg) {
   __shared__ float red[32];
+  __shared__ int s_row;
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
@@ -25,6 +38,33 @@ __global__ void embed_kernel(float* __restrict__ out, const S* __restrict__ tabl
   if (!ok) id = 0;
   const S* row = table + static_cast<size_t>(id) * D;
   float* o = out + static_cast<size_t>(t) * D;
+  if (bg.table) {
+    if (threadIdx.x == 0) {
+      const int seq = bg.seq_of[t], first = bg.cu[seq];
+      long long before;  // the token before this one plus one
+      if (t == first) {
+        int* keep = bg.previous + bg.slots[seq];
+        before = *keep;
+        *keep = tokens[bg.cu[seq + 1] - 1] + 1;
+      } else {
+        before = static_cast<long long>(tokens[t - 1]) + 1;
+      }
+      s_row = before <= 0 ? bg.buckets
+                          : static_cast<int>(((before - 1) * bg.mul_prev + static_cast<long long>(id) * bg.mul_cur) % bg.buckets);
+    }
+    __syncthreads();
+    const S* add = static_cast<const S*>(bg.table) + static_cast<size_t>(s_row) * D;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < D; i += blockDim.x) {
+      const float v = (ok ? mult * ldf(row + i) : 0.f) + ldf(add + i);
+      o[i] = v;
+      ss += v * v;
+    }
+    if (!norm_w) return;
+    const float inv = 1.0f / sqrtf(block_sum(ss, red) / static_cast<float>(D) + eps);
+    for (int i = threadIdx.x; i < D; i += blockDim.x) o[i] = o[i] * inv * norm_w[i];  // (own entries only)
+    return;
+  }
   if (!norm_w) {
     for (int i = threadIdx.x; i < D; i += blockDim.x) o[i] = ok ? mult * ldf(row + i) : 0.f;
     return;
@@ -123,7 +163,7 @@ __global__ void add_rmsnorm_vec_kernel(float* __restrict__ h, const S* __restric
 
 // A sublayer's result is normed once more before it joins the stream, and the stream is normed for the
 // next sublayer, in one launch (a block per row, the row kept in shared memory, float throughout):
-//   s   = sa * a + sb * b
+//   s   = sa * a + sb * b (+ bias, a float vector)
 //   u   = s / sqrt(mean(s^2) + post_eps) * post_w
 //   v   = h + u                      (h absent: v = u);  h = v when rows == nullptr
 //   out = v / sqrt(mean(v^2) + eps) * w          (when out is given; w absent: out = v)
@@ -132,7 +172,8 @@ template <typename S>
 __global__ void add_postnorm_rmsnorm_kernel(float* __restrict__ h, const S* __restrict__ a, float sa,
                                             const S* __restrict__ b, float sb, const float* __restrict__ post_w,
                                             float post_eps, const float* __restrict__ w, float eps,
-                                            S* __restrict__ out, const int* __restrict__ rows, int D) {
+                                            S* __restrict__ out, const int* __restrict__ rows, int D,
+                                            const float* __restrict__ bias) {
   extern __shared__ float buf[];
   __shared__ float red[32];
   pdl_launch_dependents();
@@ -143,6 +184,7 @@ __global__ void add_postnorm_rmsnorm_kernel(float* __restrict__ h, const S* __re
   for (int i = threadIdx.x; i < D; i += blockDim.x) {
     float s = sa * ldf(a + src + i);
     if (b) s = s + sb * ldf(b + src + i);
+    if (bias) s = s + bias[i];
     buf[i] = s;
     ss += s * s;
   }
@@ -174,7 +216,8 @@ template <typename S, int P>
 __global__ void add_postnorm_rmsnorm_vec_kernel(float* __restrict__ h, const S* __restrict__ a, float sa,
                                                 const S* __restrict__ b, float sb, const float* __restrict__ post_w,
                                                 float post_eps, const float* __restrict__ w, float eps,
-                                                S* __restrict__ out, const int* __restrict__ rows, int D) {
+                                                S* __restrict__ out, const int* __restrict__ rows, int D,
+                                                const float* __restrict__ bias) {
   extern __shared__ float buf[];
   __shared__ float red[32];
   pdl_launch_dependents();
@@ -188,6 +231,10 @@ __global__ void add_postnorm_rmsnorm_vec_kernel(float* __restrict__ h, const S* 
     if (b) {
       const float4 x = ld4(b + src + i);
       s.x += sb * x.x; s.y += sb * x.y; s.z += sb * x.z; s.w += sb * x.w;
+    }
+    if (bias) {
+      const float4 x = ld4(bias + i);
+      s.x += x.x; s.y += x.y; s.z += x.z; s.w += x.w;
     }
     return s;
   };
@@ -278,11 +325,15 @@ __global__ void cast_scale_kernel(float* __restrict__ out, const S* __restrict__
 }  // namespace pmm
 
 PMM_EXPORT int pmm_embed(void* out, const void* table, const int* tokens, float mult, int T, int D,
-                         int V, int dtype, const float* norm_w, float eps, cudaStream_t stream) {
+                         int V, int dtype, const float* norm_w, float eps, const void* bigram, long long mul_prev,
+                         long long mul_cur, int buckets, int* previous, const int* seq_of, const int* cu,
+                         const int* slots, cudaStream_t stream) {
   if (T <= 0) return 0;
+  if (bigram && (buckets <= 0 || mul_prev < 0 || mul_cur < 0 || !previous || !seq_of || !cu || !slots)) return PMM_ERR_BAD_ARGUMENT;
+  const pmm::Bigram bg{bigram, mul_prev, mul_cur, buckets, previous, seq_of, cu, slots};
   PMM_DISPATCH_DTYPE(dtype, S, pmm::launch_pdl(pmm::embed_kernel<S>, dim3(T), dim3(256), 0, stream,
                                                static_cast<float*>(out), static_cast<const S*>(table), tokens,
-                                               mult, D, V, norm_w, eps));
+                                               mult, D, V, norm_w, eps, bg));
   return pmm::launch_status();
 }
 
@@ -314,14 +365,14 @@ PMM_EXPORT int pmm_add_rmsnorm(void* h, const void* a, float sa, const void* b, 
 // type or nullptr; rows [R] or nullptr (then R = T).
 PMM_EXPORT int pmm_add_postnorm_rmsnorm(void* h, const void* a, float sa, const void* b, float sb, const float* post_w,
                                         float post_eps, const float* w, float eps, void* out, const int* rows, int R,
-                                        int D, int dtype, cudaStream_t stream) {
+                                        int D, int dtype, const float* bias, cudaStream_t stream) {
   if (R <= 0) return 0;
   if (D <= 0 || !a || !post_w || (rows && !out) || (!h && !out)) return PMM_ERR_BAD_ARGUMENT;
   const size_t smem = static_cast<size_t>(D) * sizeof(float);
   if (smem > 200 * 1024) return PMM_ERR_BAD_ARGUMENT;
   const int threads = D >= 1024 ? 256 : 128;
   auto aligned = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
-  const bool vec = D % 4 == 0 && aligned(h) && aligned(a) && aligned(b) && aligned(out) && aligned(w) && aligned(post_w);
+  const bool vec = D % 4 == 0 && aligned(h) && aligned(a) && aligned(b) && aligned(out) && aligned(w) && aligned(post_w) && aligned(bias);
   PMM_DISPATCH_DTYPE(dtype, S, {
     const int pieces = (D + threads * 4 - 1) / (threads * 4);
     auto kern = !vec ? pmm::add_postnorm_rmsnorm_kernel<S>
@@ -332,7 +383,7 @@ PMM_EXPORT int pmm_add_postnorm_rmsnorm(void* h, const void* a, float sa, const 
       if (e != cudaSuccess) return static_cast<int>(e);
     }
     pmm::launch_pdl(kern, dim3(R), dim3(threads), smem, stream, static_cast<float*>(h), static_cast<const S*>(a), sa,
-                    static_cast<const S*>(b), sb, post_w, post_eps, w, eps, static_cast<S*>(out), rows, D);
+                    static_cast<const S*>(b), sb, post_w, post_eps, w, eps, static_cast<S*>(out), rows, D, bias);
   });
   return pmm::launch_status();
 }

@@ -15,6 +15,11 @@
 //   read-out: o_i = (q_i * exp L_i)^T S_0 + sum_{j<=i} B_ij u_j,   B_ij = sum_c q_i[c] k_j[c] exp(L_i[c] - L_j[c])
 //   state after the chunk of n tokens: S = diag(exp L_{n-1}) S_0 + (K * exp(L_{n-1} - L))^T U
 //
+// Time mixing (kRuleWkv) is the decayed sum with a decay per channel and a read-out before the token's own write:
+//   o_i = (q_i * exp L_(i-1))^T S_0 + sum_{j<i} B_ij v_j + B_ii v_i,  B_ij = sum_c q_i[c] k_j[c] exp(L_(i-1)[c] - L_j[c]),
+//   B_ii = sum_c q_i[c] b[c] k_i[c] with the bonus b;  only `chunk_prepare` knows the difference.  Retention
+// (kRuleRetention) is the decayed sum whose q and k are rotated there.
+//
 // Only differences L_i - L_j with i >= j are ever exponentiated, so nothing overflows however strong
 // the decay.  `chunk_prepare` makes W, Uv, B, Q * exp L, K * exp(L_end - L) and exp L_end for every
 // (chunk, head) in parallel.  What follows keeps the chain from chunk to chunk as short as it can be
@@ -25,7 +30,7 @@
 // CUDA cores: scores, decays, the triangular solve and the state stay 32-bit in both storage types.
 // Chunks start at the portion's first token; results do not depend on where a portion is cut beyond
 // rounding.
-#include "common.cuh"
+#include "recurrence_rules.cuh"
 #include <utility>
 
 namespace pmm {
@@ -42,7 +47,10 @@ struct ChunkArgs {
   const void* v; long long ld_v;        // [T, H*dv]
   const void* beta; long long ld_beta;  // delta: [T, H]
   const void* a; long long ld_a;        // delta: [T, H*d]
-  const float* dt_bias; const float* a_log; const float* decay;
+  const float* dt_bias; const float* a_log; const float* decay;   // wkv: dt_bias is the bias of a, a is float
+  const float* bonus;                   // wkv: [H*d]
+  float k_scale;                        // retention
+  RecRotation rot;                      // retention
   const int* cu; int n_seq;
   int H, Hk, d, dv;
   float unit_eps, q_scale;
@@ -71,15 +79,17 @@ __device__ __forceinline__ bool locate_chunk(const int* __restrict__ cu, int n_s
   return false;
 }
 
-template <typename S, bool DELTA>
+template <typename S, int RULE>
 __global__ void __launch_bounds__(kPrepThreads)
     chunk_prepare_kernel(ChunkArgs p) {
   extern __shared__ float sm[];
+  constexpr bool DELTA = RULE == kRuleDelta, WKV = RULE == kRuleWkv, SILU = RULE == kRuleDecay;
+  constexpr bool CHANNEL = DELTA || WKV;  // a decay per key channel
   const int d = p.d, dv = p.dv, ds = d + 1;  // rows of stride d + 1: row i, column c sits in bank (i + c) mod 32
   float* sK = sm;                         // [C][ds]
   float* sQ = sK + kChunk * ds;           // [C][ds]   (later: the right-hand sides of the solve)
-  float* sL = sQ + kChunk * ds;           // delta: [C][ds]
-  float* sA = sL + (DELTA ? kChunk * ds : 0);  // delta: [C][C + 1]
+  float* sL = sQ + kChunk * ds;           // delta, wkv: [C][ds]
+  float* sA = sL + (CHANNEL ? kChunk * ds : 0);  // delta: [C][C + 1]
   __shared__ float s_beta[kChunk];
   pdl_launch_dependents();
   pdl_wait();
@@ -110,14 +120,23 @@ __global__ void __launch_bounds__(kPrepThreads)
       sK[i * ds + c] = kv;
       const float av = ldf(static_cast<const S*>(p.a) + t * p.ld_a + h * d + c) + p.dt_bias[h * d + c];
       sL[i * ds + c] = a_neg * softplus_f(av);
+    } else if (WKV) {
+      sQ[i * ds + c] = qv;
+      sK[i * ds + c] = kv;
+      // (the bound keeps the running sums finite; exp(-exp(80)) is zero by far)
+      sL[i * ds + c] = -expf(fminf(static_cast<const float*>(p.a)[t * p.ld_a + h * d + c] + p.dt_bias[h * d + c], 80.f));
     } else {
-      sQ[i * ds + c] = silu_f(qv);
-      sK[i * ds + c] = silu_f(kv);
+      sQ[i * ds + c] = SILU ? silu_f(qv) : qv;
+      sK[i * ds + c] = SILU ? silu_f(kv) : kv * p.k_scale;
     }
   }
   if (DELTA && tid < n) s_beta[tid] = sigmoid_c(ldf(static_cast<const S*>(p.beta) + static_cast<long long>(t0 + tid) * p.ld_beta + h));
   __syncthreads();
-  const float log_a = DELTA ? 0.f : logf(fmaxf(p.decay[h], 1e-38f));
+  if (RULE == kRuleRetention && p.rot.rot_dims > 0) {
+    rotate_rows(sQ, sK, ds, n, t0, p.rot, tid, kPrepThreads);
+    __syncthreads();
+  }
+  const float log_a = CHANNEL ? 0.f : logf(fmaxf(p.decay[h], 1e-38f));
   if (DELTA) {
     for (int i = warp; i < n; i += kPrepThreads / 32) {  // unit length per token
       float sq = 0.f, sk = 0.f;
@@ -133,6 +152,8 @@ __global__ void __launch_bounds__(kPrepThreads)
         sK[i * ds + c] *= fk;
       }
     }
+  }
+  if (CHANNEL) {
     for (int c = tid; c < d; c += kPrepThreads) {  // running sums of the logarithms
       float run = 0.f;
       for (int i = 0; i < n; ++i) {
@@ -144,26 +165,28 @@ __global__ void __launch_bounds__(kPrepThreads)
   }
 
   // ---- A (delta) and B
-  if (DELTA && p.sub_blocks) {
+  // wkv: the decays up to the token before i weaken what i reads: row i - 1 of the running sums (i > j >= 0)
+  const float* sLx = WKV ? sL - ds : sL;
+  if (CHANNEL && p.sub_blocks) {
     // Pairs inside one sub-block of 16 tokens: the exponential per channel.  A warp takes two rows,
     // 16 lanes each, a lane one column of the row's sub-block.
     for (int i2 = 2 * warp; i2 < n; i2 += 2 * (kPrepThreads / 32)) {
       const int i = i2 + (lane >> 4), j = (i & ~15) + (lane & 15);
       if (i < n && j <= i) {
-        const float *qi = sQ + i * ds, *ki = sK + i * ds, *li = sL + i * ds, *kj = sK + j * ds, *lj = sL + j * ds;
+        const float *qi = sQ + i * ds, *ki = sK + i * ds, *li = sLx + i * ds, *kj = sK + j * ds, *lj = sL + j * ds;
         float accA = 0.f, accB = 0.f;
         for (int c = 0; c < d; ++c) {
-          const float w = expf(li[c] - lj[c]) * kj[c];
-          accA += ki[c] * w;
+          const float w = (WKV && i == j ? p.bonus[h * d + c] : expf(li[c] - lj[c])) * kj[c];
+          if (DELTA) accA += ki[c] * w;
           accB += qi[c] * w;
         }
-        sA[i * (kChunk + 1) + j] = accA;
+        if (DELTA) sA[i * (kChunk + 1) + j] = accA;
         oB[i * kChunk + j] = accB;
       }
     }
     // Pairs across sub-blocks: with r the last row before i's sub-block, exp(L_i - L_j) = exp(L_i - L_r) exp(L_r - L_j),
     // both factors at most one, so the rows are scaled once per sub-block and the pairs are plain dot products.
-    float* sKd = sA + kChunk * (kChunk + 1);   // [48][ds]  k_j exp(L_r - L_j), j before the sub-block
+    float* sKd = sA + (DELTA ? kChunk * (kChunk + 1) : 0);   // [48][ds]  k_j exp(L_r - L_j), j before the sub-block
     float* sKp = sKd + 48 * ds;                // [16][ds]  k_i exp(L_i - L_r), i in the sub-block
     float* sQp = sKp + 16 * ds;                // [16][ds]  q_i exp(L_i - L_r)
     for (int blk = 1; 16 * blk < n; ++blk) {
@@ -175,8 +198,8 @@ __global__ void __launch_bounds__(kPrepThreads)
       }
       for (int e = tid; e < rows * d; e += kPrepThreads) {
         const int ii = e / d, c = e - ii * d, i = 16 * blk + ii;
-        const float pw = expf(sL[i * ds + c] - sL[r * ds + c]);
-        sKp[ii * ds + c] = sK[i * ds + c] * pw;
+        const float pw = expf(sLx[i * ds + c] - sL[r * ds + c]);
+        if (DELTA) sKp[ii * ds + c] = sK[i * ds + c] * pw;
         sQp[ii * ds + c] = sQ[i * ds + c] * pw;
       }
       __syncthreads();
@@ -190,10 +213,10 @@ __global__ void __launch_bounds__(kPrepThreads)
             const float* kd = sKd + j * ds;
             float accA = 0.f, accB = 0.f;
             for (int c = 0; c < d; ++c) {
-              accA += kp[c] * kd[c];
+              if (DELTA) accA += kp[c] * kd[c];
               accB += qp[c] * kd[c];
             }
-            sA[i * (kChunk + 1) + j] = accA;
+            if (DELTA) sA[i * (kChunk + 1) + j] = accA;
             oB[i * kChunk + j] = accB;
           }
         }
@@ -204,21 +227,21 @@ __global__ void __launch_bounds__(kPrepThreads)
   for (int i = warp; i < n; i += kPrepThreads / 32) {
     const float* qi = sQ + i * ds;
     const float* ki = sK + i * ds;
-    const float* li = sL + i * ds;
+    const float* li = sLx + i * ds;
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
       const int j = lane + 32 * half;
       if (j > i) continue;
       const float* kj = sK + j * ds;
       float accA = 0.f, accB = 0.f;
-      if (DELTA) {
+      if (CHANNEL) {
         const float* lj = sL + j * ds;
         for (int c = 0; c < d; ++c) {
-          const float w = expf(li[c] - lj[c]) * kj[c];
-          accA += ki[c] * w;
+          const float w = (WKV && i == j ? p.bonus[h * d + c] : expf(li[c] - lj[c])) * kj[c];
+          if (DELTA) accA += ki[c] * w;
           accB += qi[c] * w;
         }
-        sA[i * (kChunk + 1) + j] = accA;
+        if (DELTA) sA[i * (kChunk + 1) + j] = accA;
       } else {
         for (int c = 0; c < d; ++c) accB += qi[c] * kj[c];
         accB *= expf(log_a * static_cast<float>(i - j));
@@ -230,16 +253,17 @@ __global__ void __launch_bounds__(kPrepThreads)
   // ---- q * exp L, k * exp(L_end - L), exp L_end
   for (int e = tid; e < n * d; e += kPrepThreads) {
     const int i = e / d, c = e - i * d;
-    const float up = DELTA ? sL[i * ds + c] : log_a * static_cast<float>(i + 1);
-    const float end = DELTA ? sL[(n - 1) * ds + c] : log_a * static_cast<float>(n);
-    oQg[i * d + c] = sQ[i * ds + c] * expf(up);
+    const float up = CHANNEL ? sL[i * ds + c] : log_a * static_cast<float>(i + 1);
+    const float end = CHANNEL ? sL[(n - 1) * ds + c] : log_a * static_cast<float>(n);
+    oQg[i * d + c] = sQ[i * ds + c] * (WKV ? (i > 0 ? expf(sLx[i * ds + c]) : 1.f) : expf(up));
     oKe[i * d + c] = sK[i * ds + c] * expf(end - up);
   }
-  for (int c = tid; c < d; c += kPrepThreads) oEg[c] = expf(DELTA ? sL[(n - 1) * ds + c] : log_a * static_cast<float>(n));
+  for (int c = tid; c < d; c += kPrepThreads) oEg[c] = expf(CHANNEL ? sL[(n - 1) * ds + c] : log_a * static_cast<float>(n));
   if (!DELTA) {
     for (int e = tid; e < n * dv; e += kPrepThreads) {
       const int i = e / dv, c = e - i * dv;
-      oUv[i * dv + c] = silu_f(ldf(gv + static_cast<long long>(t0 + i) * p.ld_v + h * dv + c));
+      const float vv = ldf(gv + static_cast<long long>(t0 + i) * p.ld_v + h * dv + c);
+      oUv[i * dv + c] = SILU ? silu_f(vv) : vv;
     }
     return;
   }
@@ -825,8 +849,9 @@ __global__ void __launch_bounds__(kDecayThreads)
   }
 }
 
-inline size_t prepare_smem(int d, bool delta, bool sub_blocks = false) {
-  return sizeof(float) * (static_cast<size_t>(kChunk) * (d + 1) * (delta ? 3 : 2) + (delta ? kChunk * (kChunk + 1) : 0) +
+inline size_t prepare_smem(int d, int rule, bool sub_blocks = false) {
+  const bool delta = rule == kRuleDelta, channel = delta || rule == kRuleWkv;
+  return sizeof(float) * (static_cast<size_t>(kChunk) * (d + 1) * (channel ? 3 : 2) + (delta ? kChunk * (kChunk + 1) : 0) +
                           (sub_blocks ? static_cast<size_t>(48 + 32) * (d + 1) : 0));
 }
 inline size_t apply_smem(int d, bool delta, int nc = 16) {
@@ -834,11 +859,12 @@ inline size_t apply_smem(int d, bool delta, int nc = 16) {
                           static_cast<size_t>(d) * nc + d);
 }
 
-template <typename S, bool DELTA>
+template <typename S, int RULE>
 int launch_chunked(ChunkArgs a, int n_chunks, cudaStream_t stream) {
-  a.sub_blocks = DELTA && prepare_smem(a.d, true, true) <= 220 * 1024;
-  const size_t sp = prepare_smem(a.d, DELTA, a.sub_blocks != 0);
-  auto prep = chunk_prepare_kernel<S, DELTA>;
+  constexpr bool DELTA = RULE == kRuleDelta;
+  a.sub_blocks = (DELTA || RULE == kRuleWkv) && prepare_smem(a.d, RULE, true) <= 220 * 1024;
+  const size_t sp = prepare_smem(a.d, RULE, a.sub_blocks != 0);
+  auto prep = chunk_prepare_kernel<S, RULE>;
   if (sp > 48 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(prep, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(sp));
     if (e != cudaSuccess) return static_cast<int>(e);
@@ -919,17 +945,38 @@ int launch_chunked(ChunkArgs a, int n_chunks, cudaStream_t stream) {
 
 // Whether the chunked kernels take this key size (whole float4 rows, operands of a chunk in one block's
 // shared memory).
-PMM_EXPORT int pmm_recurrent_chunked_supported(int d, int delta) {
+// rule: kRuleDecay .. kRuleWkv (0: the decayed sum, 1: the delta rule, 2: retention, 3: time mixing).
+PMM_EXPORT int pmm_recurrent_chunked_supported(int d, int rule) {
   if (d <= 0 || d % 4) return 0;
-  return pmm::prepare_smem(d, delta != 0) <= 220 * 1024 && pmm::apply_smem(d, delta != 0) <= 220 * 1024 ? 1 : 0;
+  const bool delta = rule == pmm::kRuleDelta;
+  return pmm::prepare_smem(d, rule) <= 220 * 1024 && pmm::apply_smem(d, delta) <= 220 * 1024 ? 1 : 0;
 }
 
 // Floats of scratch per (chunk, head).
-PMM_EXPORT long long pmm_recurrent_chunked_scratch(int d, int dv, int delta) {
+PMM_EXPORT long long pmm_recurrent_chunked_scratch(int d, int dv, int rule) {
+  const bool delta = rule == pmm::kRuleDelta;
   // Ke, Qg, Uv, B, Eg; N (then every chunk's starting state); for the delta rule also W and M
   const long long w = delta ? static_cast<long long>(pmm::kChunk) * d + static_cast<long long>(d) * d : 0;
   return static_cast<long long>(pmm::kChunk) * (2 * d + dv + pmm::kChunk) + static_cast<long long>(d) * dv + w + d;
 }
+
+namespace pmm {
+// the arrays of the scratch; every one starts on a 16-byte boundary where d is a multiple of 4 (the copies in 16 bytes
+// need no more: the d * dv array is read with plain loads)
+inline void place_scratch(ChunkArgs& p, float* s, size_t ch, bool delta) {
+  const int d = p.d, dv = p.dv;
+  p.Ke = s; s += ch * kChunk * d;
+  p.Qg = s; s += ch * kChunk * d;
+  p.B = s; s += ch * kChunk * kChunk;
+  p.N = s; s += ch * static_cast<size_t>(d) * dv;
+  if (delta) {
+    p.W = s; s += ch * kChunk * d;
+    p.M = s; s += ch * static_cast<size_t>(d) * d;
+  }
+  p.Uv = s; s += ch * kChunk * dv;
+  p.Eg = s;
+}
+}  // namespace pmm
 
 // n_chunks = sum over sequences of ceil(tokens / 64) (an upper bound is fine: surplus blocks leave).
 // scratch: n_chunks * H * pmm_recurrent_chunked_scratch(...) floats, 16-byte aligned.  Other arguments as
@@ -943,7 +990,7 @@ PMM_EXPORT int pmm_recurrent_chunked(const void* q, long long ld_q, const void* 
   if (n_seq <= 0 || n_chunks <= 0) return 0;
   const bool delta = decay == nullptr;
   if (H <= 0 || Hk <= 0 || H % Hk || dv <= 0 || H > 65535 || n_seq > 65535 || !scratch ||
-      reinterpret_cast<uintptr_t>(scratch) % 16 || !pmm_recurrent_chunked_supported(d, delta))
+      reinterpret_cast<uintptr_t>(scratch) % 16 || !pmm_recurrent_chunked_supported(d, delta ? pmm::kRuleDelta : pmm::kRuleDecay))
     return PMM_ERR_BAD_ARGUMENT;
   pmm::ChunkArgs p{};
   p.q = q; p.ld_q = ld_q; p.k = k; p.ld_k = ld_k; p.v = v; p.ld_v = ld_v;
@@ -952,22 +999,36 @@ PMM_EXPORT int pmm_recurrent_chunked(const void* q, long long ld_q, const void* 
   p.cu = cu; p.n_seq = n_seq; p.H = H; p.Hk = Hk; p.d = d; p.dv = dv;
   p.unit_eps = unit_eps; p.q_scale = q_scale;
   const size_t ch = static_cast<size_t>(n_chunks) * H;
-  float* s = scratch;
-  // every array starts on a 16-byte boundary where d is a multiple of 4 (the copies in 16 bytes need no
-  // more: the decayed sum's d * dv array is read with plain loads)
-  p.Ke = s; s += ch * pmm::kChunk * d;
-  p.Qg = s; s += ch * pmm::kChunk * d;
-  p.B = s; s += ch * pmm::kChunk * pmm::kChunk;
-  p.N = s; s += ch * static_cast<size_t>(d) * dv;
-  if (delta) {
-    p.W = s; s += ch * pmm::kChunk * d;
-    p.M = s; s += ch * static_cast<size_t>(d) * d;
-  }
-  p.Uv = s; s += ch * pmm::kChunk * dv;
-  p.Eg = s;
+  pmm::place_scratch(p, scratch, ch, delta);
   p.state = state; p.slots = slots; p.out = out;
   PMM_DISPATCH_DTYPE(dtype, S, {
-    return delta ? pmm::launch_chunked<S, true>(p, n_chunks, stream) : pmm::launch_chunked<S, false>(p, n_chunks, stream);
+    return delta ? pmm::launch_chunked<S, pmm::kRuleDelta>(p, n_chunks, stream) : pmm::launch_chunked<S, pmm::kRuleDecay>(p, n_chunks, stream);
+  });
+  return 0;
+}
+
+// kRuleRetention (decay given) and kRuleWkv in chunks: arguments as pmm_recurrence, n_chunks and scratch as above.
+PMM_EXPORT int pmm_recurrence_chunked(const void* q, long long ld_q, const void* k, long long ld_k, const void* v, long long ld_v,
+                                      const float* decay, float k_scale, const int* positions, const float* inv_freq,
+                                      int rot_dims, int half_layout, const float* a, long long ld_a, const float* a_bias,
+                                      const float* bonus, float* state, const int* cu, const int* slots, float* out,
+                                      float* scratch, int n_seq, int n_chunks, int H, int d, int dv, int dtype,
+                                      cudaStream_t stream) {
+  if (n_seq <= 0 || n_chunks <= 0) return 0;
+  if (H <= 0 || dv <= 0 || H > 65535 || n_seq > 65535 || !scratch || reinterpret_cast<uintptr_t>(scratch) % 16 ||
+      !pmm_recurrent_chunked_supported(d, decay ? pmm::kRuleRetention : pmm::kRuleWkv) || rot_dims < 0 || rot_dims > d ||
+      rot_dims % 2 || (rot_dims > 0 && (!positions || !inv_freq)) || (!decay && (!a || !a_bias || !bonus)))
+    return PMM_ERR_BAD_ARGUMENT;
+  pmm::ChunkArgs p{};
+  p.q = q; p.ld_q = ld_q; p.k = k; p.ld_k = ld_k; p.v = v; p.ld_v = ld_v;
+  p.a = a; p.ld_a = ld_a; p.dt_bias = a_bias; p.decay = decay; p.bonus = bonus; p.k_scale = k_scale;
+  p.rot = {positions, inv_freq, rot_dims, half_layout};
+  p.cu = cu; p.n_seq = n_seq; p.H = H; p.Hk = H; p.d = d; p.dv = dv;
+  pmm::place_scratch(p, scratch, static_cast<size_t>(n_chunks) * H, false);
+  p.state = state; p.slots = slots; p.out = out;
+  PMM_DISPATCH_DTYPE(dtype, S, {
+    return decay ? pmm::launch_chunked<S, pmm::kRuleRetention>(p, n_chunks, stream)
+                 : pmm::launch_chunked<S, pmm::kRuleWkv>(p, n_chunks, stream);
   });
   return 0;
 }

@@ -111,6 +111,128 @@ __global__ void __launch_bounds__(256)
   }
 }
 
+// ------------------------------------------------------------------------------------------------------------
+// The same preparation with a norm per head: bias, the head's RMS norm (with a weight that all heads share, without
+// one, or none), rotation with sines and cosines times an amplitude, and values that are mixed with the values an
+// earlier layer left for the same tokens,  v <- (1 - l) v + l v0.  A warp takes one head row (a query, key or value
+// head of a token): it keeps the row in registers for the norm, in its own piece of shared memory for the rotation's
+// partner entries, and writes the padded row.  Blocks of 8 warps; the rows of a token are spread over gridDim.y.
+constexpr int kHeadRopeWarps = 8;
+constexpr int kHeadRopeMaxDim = 256;
+constexpr int kHeadRopePer = kHeadRopeMaxDim / 32;
+
+struct HeadRopeArgs {
+  const void *q, *k, *v;
+  long long ld_q, ld_k, ld_v;
+  const float* inv_freq;
+  const int *positions, *seq_of, *block_table;
+  int max_blocks, page_size;
+  void *pool, *q_out;
+  int H, G, d, dv, Dp, rot_dims, half_layout;
+  float amplitude;
+  const float *q_bias, *k_bias, *v_bias;
+  float norm_eps;                  // below zero: no norm
+  const float *q_w, *k_w;          // [d] or nullptr
+  void* values;                    // [T, G*dv] or nullptr: the earlier layer's values (mix given) or where to leave these
+  const float* mix;                // one value, or nullptr
+};
+
+template <typename S>
+__global__ void __launch_bounds__(kHeadRopeWarps * 32)
+    head_norm_rope_store_kernel(const HeadRopeArgs p) {
+  __shared__ float sn_t[kRopeMaxPairs], cs_t[kRopeMaxPairs];
+  __shared__ float rows[kHeadRopeWarps][kHeadRopeMaxDim];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int pos = p.positions[t];
+  const float fpos = static_cast<float>(pos);
+  const int half = p.rot_dims >> 1;
+  const int n_rows = p.H + 2 * p.G;
+  // (a block of value rows alone turns nothing)
+  if (static_cast<int>(blockIdx.y) * kHeadRopeWarps < p.H + p.G)
+    for (int f = threadIdx.x; f < half; f += blockDim.x) {
+      float s, c;
+      sincosf(fpos * p.inv_freq[f], &s, &c);
+      sn_t[f] = s * p.amplitude;
+      cs_t[f] = c * p.amplitude;
+    }
+  __syncthreads();
+  const int row = blockIdx.y * kHeadRopeWarps + warp;
+  if (row >= n_rows) return;
+  S* page_row = nullptr;
+  if (row >= p.H) {
+    const int page = p.block_table[static_cast<size_t>(p.seq_of[t]) * p.max_blocks + pos / p.page_size];
+    page_row = static_cast<S*>(p.pool) + (static_cast<size_t>(page) * 2 * p.page_size + pos % p.page_size) * (p.G * p.Dp);
+  }
+  if (row >= p.H + p.G) {  // ---- a value head
+    const int g = row - p.H - p.G;
+    const S* src = static_cast<const S*>(p.v) + static_cast<long long>(t) * p.ld_v + g * p.dv;
+    S* vals = p.values ? static_cast<S*>(p.values) + (static_cast<size_t>(t) * p.G + g) * p.dv : nullptr;
+    S* dst = page_row + static_cast<size_t>(p.page_size) * (p.G * p.Dp) + g * p.Dp;
+    const float l = p.mix ? *p.mix : 0.f;
+    for (int i = lane; i < p.Dp; i += 32) {
+      float x = 0.f;
+      if (i < p.dv) {
+        x = ldf(src + i) + (p.v_bias ? p.v_bias[g * p.dv + i] : 0.f);
+        if (p.mix) x = (1.f - l) * x + l * ldf(vals + i);
+        else if (vals) stf(vals + i, x);
+      }
+      stf(dst + i, x);
+    }
+    return;
+  }
+  const bool is_q = row < p.H;
+  const int h = is_q ? row : row - p.H;
+  const S* src = is_q ? static_cast<const S*>(p.q) + static_cast<long long>(t) * p.ld_q + h * p.d
+                      : static_cast<const S*>(p.k) + static_cast<long long>(t) * p.ld_k + h * p.d;
+  const float* bias = is_q ? p.q_bias : p.k_bias;
+  const float* w = is_q ? p.q_w : p.k_w;
+  float x[kHeadRopePer];
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < kHeadRopePer; ++j) {
+    const int i = lane + 32 * j;
+    x[j] = 0.f;
+    if (i < p.d) x[j] = ldf(src + i) + (bias ? bias[h * p.d + i] : 0.f);
+    ss += x[j] * x[j];
+  }
+  if (p.norm_eps >= 0.f) {
+    const float inv = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(p.d) + p.norm_eps);
+#pragma unroll
+    for (int j = 0; j < kHeadRopePer; ++j) {
+      const int i = lane + 32 * j;
+      if (i < p.d) x[j] *= w ? inv * w[i] : inv;
+    }
+  }
+  if (half > 0) {
+#pragma unroll
+    for (int j = 0; j < kHeadRopePer; ++j) {
+      const int i = lane + 32 * j;
+      if (i < p.rot_dims) rows[warp][i] = x[j];
+    }
+    __syncwarp();
+#pragma unroll
+    for (int j = 0; j < kHeadRopePer; ++j) {
+      const int i = lane + 32 * j;
+      if (i < p.rot_dims) {
+        const bool second = p.half_layout ? i >= half : (i & 1);
+        const int other = p.half_layout ? (second ? i - half : i + half) : (i ^ 1);
+        const int f = p.half_layout ? (second ? i - half : i) : (i >> 1);
+        const float y = rows[warp][other];
+        x[j] = second ? x[j] * cs_t[f] + y * sn_t[f] : x[j] * cs_t[f] - y * sn_t[f];
+      }
+    }
+  }
+  S* dst = is_q ? static_cast<S*>(p.q_out) + (static_cast<size_t>(t) * p.H + h) * p.Dp : page_row + h * p.Dp;
+#pragma unroll
+  for (int j = 0; j < kHeadRopePer; ++j) {
+    const int i = lane + 32 * j;
+    if (i < p.Dp) stf(dst + i, x[j]);  // (entries from d on are zero)
+  }
+}
+
 }  // namespace pmm
 
 // q [T, H*d], k [T, G*d], v [T, G*dv] rows of stride ld; inv_freq [rot_dims/2] floats (may be nullptr when
@@ -135,5 +257,27 @@ PMM_EXPORT int pmm_rope_pairs_store(const void* q, long long ld_q, const void* k
                                                block_table, max_blocks, static_cast<S*>(pool), page_size,
                                                static_cast<S*>(q_out), H, G, d, dv, Dp, rot_dims, half_layout, q_bias,
                                                k_bias, v_bias, q_norm_w, k_norm_w, norm_eps, v_norm_eps));
+  return pmm::launch_status();
+}
+
+// q [T, H*d], k [T, G*d], v [T, G*dv] rows of stride ld; pool [pages, 2, page_size, G*Dp]; q_out [T, H*Dp]; biases,
+// norm weights [d] floats or nullptr; norm_eps below zero: no norm; values [T, G*dv] or nullptr, mix one float or
+// nullptr (values are read where mix is given and written where it is not).  Dp up to 256.
+PMM_EXPORT int pmm_head_norm_rope_store(const void* q, long long ld_q, const void* k, long long ld_k, const void* v,
+                                        long long ld_v, const float* inv_freq, const int* positions, const int* seq_of,
+                                        const int* block_table, int max_blocks, void* pool, int page_size, void* q_out,
+                                        int T, int H, int G, int d, int dv, int Dp, int rot_dims, int half_layout,
+                                        float amplitude, const float* q_bias, const float* k_bias, const float* v_bias,
+                                        float norm_eps, const float* q_w, const float* k_w, void* values, const float* mix,
+                                        int dtype, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (H <= 0 || G <= 0 || d <= 0 || dv <= 0 || Dp < d || Dp < dv || Dp > pmm::kHeadRopeMaxDim || rot_dims < 0 || rot_dims > d ||
+      rot_dims % 2 || (rot_dims > 0 && !inv_freq) || page_size <= 0 || (mix && !values))
+    return PMM_ERR_BAD_ARGUMENT;
+  const pmm::HeadRopeArgs a{q, k, v, ld_q, ld_k, ld_v, inv_freq, positions, seq_of, block_table, max_blocks, page_size,
+                            pool, q_out, H, G, d, dv, Dp, rot_dims, half_layout, amplitude, q_bias, k_bias, v_bias,
+                            norm_eps, q_w, k_w, values, mix};
+  const dim3 grid(T, (H + 2 * G + pmm::kHeadRopeWarps - 1) / pmm::kHeadRopeWarps);
+  PMM_DISPATCH_DTYPE(dtype, S, pmm::launch_pdl(pmm::head_norm_rope_store_kernel<S>, grid, dim3(pmm::kHeadRopeWarps * 32), 0, stream, a));
   return pmm::launch_status();
 }

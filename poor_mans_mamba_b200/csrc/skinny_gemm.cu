@@ -35,7 +35,10 @@ constexpr int kSgWStride = kSgChunk + 8;
 constexpr int kSgThreads = 256;
 constexpr int kSgPieces = kSgRows * (kSgChunk / 8) / kSgThreads;  // 16-byte pieces per thread and chunk
 
-enum { kSgStore = 0, kSgSwiglu = 1, kSgResidual = 2, kSgStoreF32 = 3 };
+// MULTI: STORE for up to kSgProducts products with activations, weights, widths and outputs of their own (gridDim.z).
+// GELU: STORE with y = gelu(x W^T), the erf form.
+enum { kSgStore = 0, kSgSwiglu = 1, kSgResidual = 2, kSgStoreF32 = 3, kSgMulti = 4, kSgGelu = 5 };
+constexpr int kSgProducts = 6;
 
 struct SkinnyProblem {
   const bf16* x;       // [M, ldx] activations, or nullptr when the norm prologue is used
@@ -46,10 +49,14 @@ struct SkinnyProblem {
   const bf16* w;       // [N or 2F, K]
   int K;
   float scale;         // RESIDUAL: factor on y; SWIGLU: gate multiplier
+  int N;               // MULTI: this product's output columns
+  bf16* y;             // MULTI: [M, ldy]
+  long long ldy;
 };
 
-struct SkinnyArgs {
-  SkinnyProblem p[2];
+template <int NP>
+struct SkinnyArgsT {
+  SkinnyProblem p[NP];
   int n_problems;
   int M, N;            // tokens, output columns (SWIGLU: F)
   int k_slice;         // columns of K per block along gridDim.y (multiple of 256)
@@ -60,6 +67,9 @@ struct SkinnyArgs {
   float y_scale;
   float y_cap;         // > 0: y32 = y_cap * tanh(y_scale * y / y_cap)
 };
+using SkinnyArgs = SkinnyArgsT<2>;
+template <int MODE>
+using SkinnyArgsOf = SkinnyArgsT<MODE == kSgMulti ? kSgProducts : 2>;
 
 __device__ __forceinline__ void sg_cp16(void* smem, const void* gmem, bool pred) {
   const unsigned s = static_cast<unsigned>(__cvta_generic_to_shared(smem));
@@ -92,8 +102,10 @@ struct SkinnyBlock {
   static constexpr int MP = MT * 8;  // padded tokens
   static constexpr int kSgStages = sg_stages(MT);
   static constexpr int kTileCols = MODE == kSgSwiglu ? 16 : kSgRows;  // output columns of a row tile
-  const SkinnyArgs& args;
+  using Args = SkinnyArgsOf<MODE>;
+  const Args& args;
   const SkinnyProblem& pr;
+  int N;  // output columns
   int K, k0, k1, kx, xs, n_chunks;
   int t0, t_step, my_tiles, total;  // row tiles t0, t0 + t_step, ...; total = my_tiles * n_chunks copies
   bf16* sW;     // [stages][32][264]
@@ -104,9 +116,10 @@ struct SkinnyBlock {
   const bf16* src[kSgPieces];  // this thread's pieces of chunk 0 of the block's first tile
   size_t tile_stride;          // elements of W between one of the block's tiles and the next
 
-  __device__ SkinnyBlock(const SkinnyArgs& a, int bx, int bx_step, int by, int bz, unsigned char* smem_raw)
+  __device__ SkinnyBlock(const Args& a, int bx, int bx_step, int by, int bz, unsigned char* smem_raw)
       : args(a), pr(a.p[bz]) {
     K = pr.K;
+    N = MODE == kSgMulti ? pr.N : a.N;
     k0 = by * a.k_slice;
     k1 = min(K, k0 + a.k_slice);
     kx = k0 < K ? (k1 - k0 + kSgChunk - 1) / kSgChunk * kSgChunk : 0;  // slice length, whole chunks
@@ -117,7 +130,7 @@ struct SkinnyBlock {
     sNw = sRed + 3 * 32 * MP;
     sInv = sNw + kx;
     n_chunks = kx / kSgChunk;
-    const int n_tx = (a.N + kTileCols - 1) / kTileCols;
+    const int n_tx = (N + kTileCols - 1) / kTileCols;
     t0 = bx;
     t_step = bx_step;
     my_tiles = bx < n_tx ? (bx + bx_step < n_tx ? (n_tx - 1 - bx) / bx_step + 1 : 1) : 0;
@@ -129,7 +142,7 @@ struct SkinnyBlock {
     for (int j = 0; j < kSgPieces; ++j) {
       const int r = (tid >> 5) + j * (kSgThreads / 32);
       // global row of W behind row r of a tile (SWIGLU: 16 gate rows, then their 16 up rows)
-      const int wr = MODE == kSgSwiglu ? (r < 16 ? n0 + r : a.N + n0 + (r - 16)) : n0 + r;
+      const int wr = MODE == kSgSwiglu ? (r < 16 ? n0 + r : N + n0 + (r - 16)) : n0 + r;
       src[j] = pr.w + static_cast<size_t>(wr) * K + k0 + c8 * 8;
     }
   }
@@ -145,7 +158,7 @@ struct SkinnyBlock {
 #pragma unroll
     for (int j = 0; j < kSgPieces; ++j) {
       const int r = (tid >> 5) + j * (kSgThreads / 32);
-      const bool ok = col_ok && (MODE == kSgSwiglu ? n0 + (r & 15) < args.N : n0 + r < args.N);
+      const bool ok = col_ok && (MODE == kSgSwiglu ? n0 + (r & 15) < N : n0 + r < N);
       sg_cp16(dst + j * (kSgThreads / 32) * kSgWStride, ok ? src[j] + off : pr.w, ok);
     }
   }
@@ -377,7 +390,7 @@ __device__ void SkinnyBlock<MT, MODE>::finish_tile(float (&acc)[MT][4], int n0) 
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int f = n0 + g + (e >> 1) * 8, m = nt * 8 + t2 + (e & 1);
-          if (f < args.N && m < M) {
+          if (f < N && m < M) {
             const float inv = pr.h_in ? sInv[m] : 1.f;  // the row's norm factor (norm prologue)
             const float up = sRed[(g + (e >> 1) * 8) * MP + m] * inv;
             args.y[static_cast<size_t>(m) * args.ldy + f] = __float2bfloat16_rn(silu_fast(acc[nt][e] * inv * pr.scale) * up);
@@ -394,8 +407,12 @@ __device__ void SkinnyBlock<MT, MODE>::finish_tile(float (&acc)[MT][4], int n0) 
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int n = n0 + ft * 16 + g + (e >> 1) * 8, m = nt * 8 + t2 + (e & 1);
-        if (n < args.N && m < M) {
-          if (MODE == kSgStore) {
+        if (n < N && m < M) {
+          if (MODE == kSgMulti) {
+            pr.y[static_cast<size_t>(m) * pr.ldy + n] = __float2bfloat16_rn(acc[nt][e]);
+          } else if (MODE == kSgGelu) {
+            args.y[static_cast<size_t>(m) * args.ldy + n] = __float2bfloat16_rn(gelu_erf_f(acc[nt][e]));
+          } else if (MODE == kSgStore) {
             const float inv = pr.h_in ? sInv[m] : 1.f;  // the row's norm factor (norm prologue)
             args.y[static_cast<size_t>(m) * args.ldy + n] = __float2bfloat16_rn(acc[nt][e] * inv);
           } else if (MODE == kSgStoreF32) {
@@ -412,7 +429,7 @@ __device__ void SkinnyBlock<MT, MODE>::finish_tile(float (&acc)[MT][4], int n0) 
 
 // MT: token tiles of 8 (1, 2, 4 or 8 -> up to 8, 16, 32, 64 tokens).
 template <int MT, int MODE, bool ONE>
-__global__ void __launch_bounds__(kSgThreads) skinny_gemm_kernel(const SkinnyArgs args) {
+__global__ void __launch_bounds__(kSgThreads) skinny_gemm_kernel(const SkinnyArgsOf<MODE> args) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   pdl_launch_dependents();
   const SkinnyBlock<MT, MODE> blk(args, blockIdx.x, gridDim.x, blockIdx.y, blockIdx.z, smem_raw);
@@ -521,7 +538,7 @@ inline size_t skinny_smem(int MP, int kx) {
 }
 
 template <int MT, int MODE>
-int launch_skinny(const SkinnyArgs& a, int k_max, cudaStream_t stream) {
+int launch_skinny(const SkinnyArgsOf<MODE>& a, int k_max, cudaStream_t stream) {
   constexpr int MP = MT * 8;
   const int kx = (min(a.k_slice, k_max) + kSgChunk - 1) / kSgChunk * kSgChunk;
   const size_t smem = skinny_smem(MP, kx);
@@ -557,7 +574,7 @@ int launch_skinny(const SkinnyArgs& a, int k_max, cudaStream_t stream) {
 }
 
 template <int MODE>
-int dispatch_skinny(const SkinnyArgs& a, int k_max, cudaStream_t stream) {
+int dispatch_skinny(const SkinnyArgsOf<MODE>& a, int k_max, cudaStream_t stream) {
   if (a.M <= 8) return launch_skinny<1, MODE>(a, k_max, stream);
   if (a.M <= 16) return launch_skinny<2, MODE>(a, k_max, stream);
   if (a.M <= 32) return launch_skinny<4, MODE>(a, k_max, stream);
@@ -584,6 +601,7 @@ int launch_chain(const SkinnyChain& ch, size_t smem, int grid, cudaStream_t stre
 
 // mode 0 STORE (y bfloat16 [M, ldy]), 1 SWIGLU (w = [gate; up] rows, N = F, scale0 = gate multiplier),
 // 2 RESIDUAL (h_out[M, N] += scale * y, k_split blocks along K, one or two products).
+// 5 GELU (STORE with y = gelu(x W^T)).
 // x0/x1: bfloat16 activations, or nullptr with h_in/norm_w/eps for the RMSNorm prologue (K0 == width of h_in).
 PMM_EXPORT int pmm_skinny_gemm(int mode, int M, int N, const void* x0, long long ldx0, const float* h_in,
                                const float* norm_w, float eps, const void* w0, int K0, float scale0,
@@ -615,6 +633,7 @@ PMM_EXPORT int pmm_skinny_gemm(int mode, int M, int N, const void* x0, long long
     case pmm::kSgStore: return pmm::dispatch_skinny<pmm::kSgStore>(a, k_max, stream);
     case pmm::kSgSwiglu: return pmm::dispatch_skinny<pmm::kSgSwiglu>(a, k_max, stream);
     case pmm::kSgResidual: return pmm::dispatch_skinny<pmm::kSgResidual>(a, k_max, stream);
+    case pmm::kSgGelu: return x0 ? pmm::dispatch_skinny<pmm::kSgGelu>(a, k_max, stream) : PMM_ERR_BAD_ARGUMENT;
     default: return PMM_ERR_BAD_ARGUMENT;
   }
 }
@@ -636,6 +655,26 @@ PMM_EXPORT int pmm_skinny_gemm_f32out(int M, int N, const void* x, long long ldx
   a.y_scale = scale;
   a.y_cap = cap;
   return pmm::dispatch_skinny<pmm::kSgStoreF32>(a, K, stream);
+}
+
+// y_i[M, ldy_i] = x_i[M, ldx_i] w_i[N_i, K]^T for up to kSgProducts products of one K (a multiple of 8), bfloat16, up to 64 rows.
+PMM_EXPORT int pmm_skinny_multi(int n, int M, int K, const void* const* x, const long long* ldx, const void* const* w,
+                                const int* N, void* const* y, const long long* ldy, cudaStream_t stream) {
+  if (M <= 0 || n <= 0) return 0;
+  if (n > pmm::kSgProducts || M > 64 || K <= 0 || K % 8) return PMM_ERR_BAD_ARGUMENT;
+  pmm::SkinnyArgsT<pmm::kSgProducts> a{};
+  int widest = 0;
+  for (int i = 0; i < n; ++i) {
+    if (!x[i] || !w[i] || !y[i] || N[i] <= 0) return PMM_ERR_BAD_ARGUMENT;
+    a.p[i] = {static_cast<const pmm::bf16*>(x[i]), ldx[i], nullptr, nullptr, 0.f, static_cast<const pmm::bf16*>(w[i]), K, 1.f,
+              N[i], static_cast<pmm::bf16*>(y[i]), ldy[i]};
+    if (N[i] > widest) widest = N[i];
+  }
+  a.n_problems = n;
+  a.M = M;
+  a.N = widest;  // sizes the grid
+  a.k_slice = (K + pmm::kSgChunk - 1) / pmm::kSgChunk * pmm::kSgChunk;
+  return pmm::dispatch_skinny<pmm::kSgMulti>(a, K, stream);
 }
 
 // One phase of pmm_skinny_chain: the arguments of pmm_skinny_gemm without M, k_split and stream.

@@ -1,7 +1,7 @@
 // Weight-streaming matrix product for steps of 33..64 tokens (it takes 1..64) on the fifth-generation
 // tensor cores:
 //   y[T, N] = x[T, K] W[N, K]^T, bfloat16 operands, float accumulation,
-// with the same epilogues as the mma.sync form for fewer tokens (skinny_gemm.cu): STORE (bfloat16),
+// with the same epilogues as the mma.sync form for fewer tokens (skinny_gemm.cu): STORE (bfloat16; with gelu on it),
 // SWIGLU (W = [gate rows; up rows], act = silu(gate * mult) * up) and RESIDUAL (h += scale * y with
 // float atomics; K may be cut into slices over blocks, and two products may share a launch).
 // At these sizes the product is still a read of W at memory speed, but with mma.sync every warp
@@ -44,7 +44,7 @@ constexpr int kStWBox = kStRows * kStKB * 2;   // 4 KB
 constexpr int kStStageBytes = kStChunk * kStWBox;
 constexpr size_t kStSmem = 1024 /*alignment*/ + static_cast<size_t>(kStMaxKB + 1) * kStXBox + static_cast<size_t>(kStStages) * kStStageBytes;
 
-enum { kStStore = 0, kStSwiglu = 1, kStResidual = 2 };
+enum { kStStore = 0, kStSwiglu = 1, kStResidual = 2, kStGelu = 3 };  // GELU: STORE with y = gelu(x W^T), the erf form
 
 // kind::f16 instruction descriptor: float accumulate, bfloat16 A and B, both K-major, N = 32, M = 128.
 constexpr unsigned kStIdesc = (1u << 4) | (1u << 7) | (1u << 10) | ((kStRows >> 3) << 17) | ((128 >> 4) << 24);
@@ -260,7 +260,11 @@ __global__ void __launch_bounds__(kStThreads)
           for (int e = 0; e < 16; ++e)
             if (n0 + e < args.N) dst[e] = __float2bfloat16_rn(a[e]);
         }
-      } else if (MODE == kStStore) {
+      } else if (MODE == kStStore || MODE == kStGelu) {
+        if (MODE == kStGelu) {
+#pragma unroll
+          for (int e = 0; e < 32; ++e) v[e] = __float_as_uint(gelu_erf_f(__uint_as_float(v[e])));
+        }
         bf16* dst = args.y + static_cast<long long>(m) * args.ldy + n0;
         if (whole) {
 #pragma unroll
@@ -343,12 +347,13 @@ PMM_EXPORT int pmm_skinny_tc_supported(int mode, int T, int N, int K0, int K1, l
   if (T < 1 || T > pmm::kStTok || N < 1 || K0 < 8 || K0 % 8 || ldx0 % 8) return 0;
   if (K1 && (K1 < 8 || K1 % 8 || ldx1 % 8)) return 0;
   if (mode == pmm::kStResidual) return 1;
-  if (mode != pmm::kStStore && mode != pmm::kStSwiglu) return 0;
+  if (mode != pmm::kStStore && mode != pmm::kStSwiglu && mode != pmm::kStGelu) return 0;
   return (K1 == 0 && K0 <= pmm::kStMaxKB * pmm::kStKB && ldy % 8 == 0) ? 1 : 0;
 }
 
 // mode 0 STORE (y bfloat16 [T, ldy]), 1 SWIGLU (w0 = [gate; up] rows, N = F, scale0 = gate multiplier),
-// 2 RESIDUAL (h_out[T, N] += scale * y; one or two products; K cut into slices of at most 1,024 columns).
+// 2 RESIDUAL (h_out[T, N] += scale * y; one or two products; K cut into slices of at most 1,024 columns), 3 GELU
+// (STORE with y = gelu(x W^T)).
 // status: one int in device memory that stays 0 unless a bounded wait gave up.
 PMM_EXPORT int pmm_skinny_tc(int mode, int T, int N, const void* x0, long long ldx0, const void* w0, int K0, float scale0,
                              const void* x1, long long ldx1, const void* w1, int K1, float scale1, void* y,
@@ -390,6 +395,7 @@ PMM_EXPORT int pmm_skinny_tc(int mode, int T, int N, const void* x0, long long l
   switch (mode) {
     case pmm::kStStore: return pmm::launch_skinny_tc<pmm::kStStore>(maps, a, k_max, stream);
     case pmm::kStSwiglu: return pmm::launch_skinny_tc<pmm::kStSwiglu>(maps, a, k_max, stream);
+    case pmm::kStGelu: return pmm::launch_skinny_tc<pmm::kStGelu>(maps, a, k_max, stream);
     default: return pmm::launch_skinny_tc<pmm::kStResidual>(maps, a, k_max, stream);
   }
 }

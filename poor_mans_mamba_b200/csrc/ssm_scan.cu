@@ -248,6 +248,45 @@ __global__ void gated_norm_kernel(const Y* __restrict__ y, const S* __restrict__
   }
 }
 
+// The norm-before-gate form for narrow groups (at most 256 channels): a warp per (token, group), the row in registers.
+constexpr int kGroupWarps = 8;
+template <typename S, typename Y>
+__global__ void __launch_bounds__(kGroupWarps * 32)
+    gated_norm_narrow_kernel(const Y* __restrict__ y, const S* __restrict__ z_raw, long long ld_z, float z_scale,
+                             const float* __restrict__ z_bias, const float* __restrict__ w, float eps, S* __restrict__ out,
+                             long long ld_out, int T, int I, int group_width, int gate_sigmoid) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int groups = I / group_width;
+  const long long item = static_cast<long long>(blockIdx.x) * kGroupWarps + (threadIdx.x >> 5);
+  if (item >= static_cast<long long>(T) * groups) return;
+  const int t = static_cast<int>(item / groups), c0 = static_cast<int>(item % groups) * group_width;
+  const int lane = threadIdx.x & 31;
+  float v[8], zv[8];
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < 8; ++j) {
+    const int i = lane + 32 * j;
+    v[j] = zv[j] = 0.f;
+    if (i < group_width) {
+      v[j] = ldf(y + static_cast<size_t>(t) * I + c0 + i);
+      zv[j] = ldf(z_raw + static_cast<long long>(t) * ld_z + c0 + i);
+    }
+    ss += v[j] * v[j];
+  }
+  const float inv = 1.0f / sqrtf(warp_sum(ss) / static_cast<float>(group_width) + eps);
+#pragma unroll
+  for (int j = 0; j < 8; ++j) {
+    const int i = lane + 32 * j;
+    if (i < group_width) {
+      const int c = c0 + i;
+      const float z = zv[j] * z_scale + (z_bias ? z_bias[c] : 0.f);
+      const float gate = gate_sigmoid ? 1.f / (1.f + expf(-z)) : silu_f(z);
+      stf(out + static_cast<long long>(t) * ld_out + c, v[j] * inv * w[c] * gate);
+    }
+  }
+}
+
 template <typename S>
 int launch_scan(const void* xbc, int ld_xbc, const void* dt_raw, long long ld_dt, float dt_scale,
                 const float* dt_shift, const float* a_log, const float* d_skip, float* state,
@@ -317,6 +356,20 @@ PMM_EXPORT int pmm_gated_norm(const void* y, const void* z_raw, long long ld_z, 
   if (T <= 0) return 0;
   if (n_groups <= 0 || I % n_groups || n_groups > 65535) return PMM_ERR_BAD_ARGUMENT;
   const int gw = I / n_groups;
+  if (w && norm_before_gate && n_groups > 1 && gw <= 256) {
+    const long long items = static_cast<long long>(T) * n_groups;
+    const dim3 narrow(static_cast<unsigned>((items + pmm::kGroupWarps - 1) / pmm::kGroupWarps));
+#define PMM_NARROW_CASE(Y)                                                                                             \
+  pmm::launch_pdl(pmm::gated_norm_narrow_kernel<S, Y>, narrow, dim3(pmm::kGroupWarps * 32), 0, stream,                 \
+                  static_cast<const Y*>(y), static_cast<const S*>(z_raw), ld_z, z_scale, z_bias, w, eps,               \
+                  static_cast<S*>(out), ld_out, T, I, gw, gate_sigmoid)
+    PMM_DISPATCH_DTYPE(dtype, S, {
+      if (y_f32) PMM_NARROW_CASE(float);
+      else PMM_NARROW_CASE(S);
+    });
+#undef PMM_NARROW_CASE
+    return pmm::launch_status();
+  }
   const size_t smem = w ? static_cast<size_t>(gw) * sizeof(float) * (norm_before_gate ? 2 : 1) : 0;
   if (smem > 200 * 1024) return PMM_ERR_BAD_ARGUMENT;
   dim3 grid(T, n_groups);

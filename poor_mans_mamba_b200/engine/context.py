@@ -2,7 +2,7 @@
 from __future__ import annotations
 
 from dataclasses import dataclass, field
-from typing import List, Optional
+from typing import Dict, List, Optional
 
 import torch
 
@@ -44,6 +44,7 @@ class StepContext:
     a layer that streams its weights once may ask the memory system for them early).
     ``defer_output_bias``: a mixer that exposes `output_bias()` leaves the bias out while this is set (its
     caller folds it into the launch that reads the mixer's output).
+    ``carried``: rows [T, width] that mixers of earlier layers leave for later ones (`Mixer.carries`), by name.
     ``unjoined_stream``: a side stream on which a layer left work running that nothing has waited
     for yet (a fetch-ahead beside its products); the model joins it before a layer that would not
     (`joins_side_stream`) and at the end of the step.
@@ -65,4 +66,5 @@ class StepContext:
     past_lens: List[int] = field(default_factory=list)
     defer_output_bias: bool = False  # set by a caller that adds a mixer's `output_bias()` itself
     fetch_ahead: Optional[List[Tensor]] = None
+    carried: Dict[str, Tensor] = field(default_factory=dict)
     unjoined_stream: Optional["torch.cuda.Stream"] = None

@@ -180,7 +180,7 @@ class GraphDecoder:
         rows, seen, _ = entry
         for j, (g, row) in enumerate(zip(self.groups, rows)):
             table = g.tables[req]
-            if len(table) != seen[j] or g.window > 0:  # grown (or a window may have passed pages)
+            if len(table) != seen[j] or g.bounded:  # grown (or a window may have passed pages)
                 arr = np.asarray(table, dtype=np.int32)
                 arr[arr < 0] = g.num_pages
                 row[:len(table)] = arr

@@ -2,7 +2,7 @@
 order in which the layers run, final norm and output head.
 
 The forward pass is the same for every architecture:
-  h = multiplier * E[tokens]                       (float32 residual stream; then the embedding's norm, if any)
+  h = multiplier * E[tokens] (+ an addend's rows)  (float32 residual stream; then the embedding's norm, if any)
   for (layer, cache_of) in order: layers[layer](h, cache of cache_of)
   logits = (norm(h)[wanted rows] @ W_head^T) * head_multiplier       (float32; then the softcap, if any)
 (reference src/runtime/runner/falconh1_runner.cpp:129-228, which keeps the last row only).
@@ -16,7 +16,7 @@ from typing import Dict, List, Optional, Tuple
 import torch
 
 from ..kernels import ops as K
-from ..parts.base import LayerCache, ModelSpec, ParamSpec, Part, StateSpec, build_part, _REGISTRIES
+from ..parts.base import EMBEDDING_CACHE, LayerCache, ModelSpec, ParamSpec, Part, StateSpec, build_part, _REGISTRIES
 from ..parts.block import ResidualStream
 from .context import StepContext
 
@@ -53,6 +53,16 @@ class Model:
         self.embedding_norm = None
         if spec.embedding_norm is not None:
             self.embedding_norm = build_part("norm", spec.embedding_norm, width=spec.hidden_size)
+        self.embedding_addend = None
+        if spec.embedding_addend is not None:
+            self.embedding_addend = build_part("embedding_addend", spec.embedding_addend, hidden_size=spec.hidden_size)
+        # rows that mixers leave for later layers of the same step: name -> width
+        self._carried: Dict[str, int] = {}
+        for layer in self.layers:
+            for mixer in getattr(layer, "mixers", ()):
+                for name, width in mixer.carries().items():
+                    if self._carried.setdefault(name, int(width)) != int(width):
+                        raise ValueError(f"the carried rows '{name}' are declared with two widths")
         self.embedding: Optional[Tensor] = None
         self.head: Optional[Tensor] = None
         self.dtype: Optional[torch.dtype] = None
@@ -72,6 +82,8 @@ class Model:
         out.append((self.spec.final_norm.name, self.final_norm))
         if self.embedding_norm is not None:
             out.append((self.spec.embedding_norm.name, self.embedding_norm))
+        if self.embedding_addend is not None:
+            out.append((self.spec.embedding_addend.name, self.embedding_addend))
         if self.reentry is not None:
             out.append((self.spec.reentry.name, self.reentry))
         return out
@@ -114,6 +126,8 @@ class Model:
             self.embedding_norm.finalize(dtype, self.device)
             if self.embedding_norm.rms_prologue() is None:
                 raise ValueError("the embedding's norm must be an RMS norm")
+        if self.embedding_addend is not None:
+            self.embedding_addend.finalize(dtype, self.device)
         if self.reentry is not None:
             self.reentry.finalize(dtype, self.device)
 
@@ -123,6 +137,9 @@ class Model:
         the execution order's ``cache_of`` names: the states that the layers run with that id
         declare, each name once (a layer that only reads another's state declares none)."""
         out: Dict[int, List[Tuple[str, StateSpec]]] = {}
+        if self.embedding_addend is not None and self.embedding_addend.state_specs():
+            name = self.embedding_addend.name
+            out[EMBEDDING_CACHE] = [(f"{name}.{s.name}", s) for s in self.embedding_addend.state_specs()]
         for call in self.spec.order:
             have = out.setdefault(call.cache_of, [])
             for name, spec in self.layers[call.layer].state_specs():
@@ -141,11 +158,12 @@ class Model:
         ws = ctx.workspace
         T, D = ctx.n_tokens, self.hidden_size
         h = ws.alloc((T, D), torch.float32)
-        if self.embedding_norm is not None:
-            norm_w, norm_eps = self.embedding_norm.rms_prologue()
-            K.embed(h, self.embedding, ctx.tokens, self.spec.embedding_multiplier, norm_w, norm_eps)
-        else:
-            K.embed(h, self.embedding, ctx.tokens, self.spec.embedding_multiplier)
+        norm_w, norm_eps = self.embedding_norm.rms_prologue() if self.embedding_norm is not None else (None, 0.0)
+        addend = {}
+        if self.embedding_addend is not None:
+            addend = self.embedding_addend.arguments(ctx, caches.get(EMBEDDING_CACHE))
+        K.embed(h, self.embedding, ctx.tokens, self.spec.embedding_multiplier, norm_w, norm_eps, **addend)
+        ctx.carried = {name: ws.alloc((T, width), ctx.dtype) for name, width in self._carried.items()}
         stream = ResidualStream(h, ctx, self._branch_buffers, lanes=self.spec.residual_lanes,
                                 second_buffer=self._second_stream_buffer)
         if self.reentry is not None and self.reentry.reads_embedding:

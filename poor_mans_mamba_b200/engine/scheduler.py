@@ -150,7 +150,7 @@ class Scheduler:
 
     def _never_fits(self, req: Request) -> bool:
         total = len(req.prompt) + len(req.output)
-        return any(g.blocks_for(total) > g.num_pages for g in self.cache.groups.values() if g.window <= 0)
+        return any(g.blocks_for(total) > g.num_pages for g in self.cache.groups.values() if not g.bounded)
 
     def _preempt(self, req: Request, plan: StepPlan) -> None:
         self._release(req.id)

@@ -28,9 +28,10 @@ class KernelError(RuntimeError):
 
 
 _SIGNATURES = {
-    "pmm_embed": [c_void_p, c_void_p, c_void_p, c_float, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p],
+    "pmm_embed": [c_void_p, c_void_p, c_void_p, c_float, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p,
+                  c_longlong, c_longlong, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p],
     "pmm_add_postnorm_rmsnorm": [c_void_p, c_void_p, c_float, c_void_p, c_float, c_void_p, c_float, c_void_p, c_float,
-                                 c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
+                                 c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p],
     "pmm_add_rmsnorm": [c_void_p, c_void_p, c_float, c_void_p, c_float, c_void_p, c_float, c_void_p,
                         c_void_p, c_int, c_int, c_int, c_void_p],
     "pmm_fold_norm": [c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_float, c_void_p, c_void_p, c_float, c_int, c_void_p,
@@ -157,6 +158,21 @@ _SIGNATURES = {
     "pmm_token_gated_update": [c_void_p, c_void_p, c_float, c_void_p, c_float, c_void_p, c_void_p, c_longlong, c_int,
                                c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_int, c_int, c_int, c_int, c_void_p],
     "pmm_cast_rows": [c_void_p, c_void_p, c_float, c_void_p, c_float, c_void_p, c_longlong, c_int, c_int, c_int, c_void_p],
+    "pmm_unary": [c_int, c_void_p, c_longlong, c_int, c_int, c_int, c_void_p],
+    "pmm_skinny_multi": [c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p],
+    "pmm_shifted_mixes": [c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong,
+                          c_int, c_int, c_int, c_void_p],
+    "pmm_low_rank_tanh": [c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+    "pmm_head_norm_rope_store": [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p,
+                                 c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+                                 c_int, c_float, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_void_p,
+                                 c_int, c_void_p],
+    "pmm_recurrence": [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_float, c_void_p, c_void_p,
+                       c_int, c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+                       c_int, c_int, c_int, c_int, c_void_p],
+    "pmm_recurrence_chunked": [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_float, c_void_p,
+                               c_void_p, c_int, c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                               c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
     "pmm_relu_squared": [c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_int, c_int, c_void_p],
     "pmm_sample_rows": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
                         c_void_p, c_void_p, c_void_p],
@@ -363,6 +379,19 @@ def linear(x: Tensor, weight: Tensor, out: Tensor) -> Tensor:
     return out
 
 
+def batched_linear(x: Tensor, weight: Tensor, out: Tensor) -> None:
+    """out[b] [T, N] = x[b] [T, K] @ weight[b] [N, K]^T through the GEMM library, one call."""
+    _cuda(x, weight, out)
+    if not (x.dim() == weight.dim() == out.dim() == 3 and x.dtype == weight.dtype == out.dtype):
+        raise KernelError("batched_linear: x [B, T, K], weight [B, N, K], out [B, T, N] of one type")
+    prev = torch.backends.cuda.matmul.allow_tf32
+    torch.backends.cuda.matmul.allow_tf32 = False
+    try:
+        torch.bmm(x, weight.transpose(1, 2), out=out)
+    finally:
+        torch.backends.cuda.matmul.allow_tf32 = prev
+
+
 _MM_F32_OUT: Optional[bool] = None
 
 
@@ -397,10 +426,14 @@ def linear_f32_out(x: Tensor, weight: Tensor, out: Tensor, scratch_low: Optional
 
 # ----------------------------------------------------------------------------- own kernels
 def embed(out: Tensor, table: Tensor, tokens: Tensor, mult: float, norm_weight: Optional[Tensor] = None,
-          eps: float = 0.0) -> None:
+          eps: float = 0.0, bigram: Optional[Tuple[Tensor, int, int]] = None, previous: Optional[Tensor] = None,
+          seq_of: Optional[Tensor] = None, cu: Optional[Tensor] = None, slots: Optional[Tensor] = None) -> None:
     """out[t] = mult * table[tokens[t]] (float32); with ``norm_weight`` [D] the row is then divided by its root
-    mean square (eps inside the root) and multiplied by the weight, all in float."""
-    _cuda(out, table, tokens, norm_weight)
+    mean square (eps inside the root) and multiplied by the weight, all in float.  ``bigram`` (table [buckets + 1, D],
+    mul_prev, mul_cur): before the norm, row (previous token * mul_prev + token * mul_cur) mod buckets of that table
+    joins, the last row for a sequence's first token; ``previous`` (int32 [slots, 1], the requests' last tokens plus
+    one, zero: none) is read and brought up to date."""
+    _cuda(out, table, tokens, norm_weight, previous, seq_of, cu, slots)
     T, D = out.shape
     if not (out.dtype == torch.float32 and out.is_contiguous()):
         raise KernelError("embed: out must be contiguous float32")
@@ -410,16 +443,33 @@ def embed(out: Tensor, table: Tensor, tokens: Tensor, mult: float, norm_weight: 
     if not (tokens.numel() == T):
         raise KernelError("embed: one token per output row")
     _f32vec(norm_weight, D, "embed: norm weight")
+    extra, mul_prev, mul_cur, buckets = None, 0, 0, 0
+    if bigram is not None:
+        extra, mul_prev, mul_cur = bigram
+        buckets = extra.shape[0] - 1
+        _cuda(extra)
+        if not (extra.dim() == 2 and extra.shape[1] == D and buckets >= 1 and extra.is_contiguous() and extra.dtype == table.dtype
+                and mul_prev >= 0 and mul_cur >= 0):
+            raise KernelError("embed: the bigram table must be [buckets + 1, D] of the table's type, its multipliers not negative")
+        for t, what in ((previous, "previous"), (seq_of, "seq_of"), (cu, "cu"), (slots, "slots")):
+            if t is None:
+                raise KernelError(f"embed: a bigram table needs {what}")
+            _i32(t, f"embed: {what}")
+        if not (seq_of.numel() == T):
+            raise KernelError("embed: seq_of [T]")
     _call("pmm_embed", out.data_ptr(), table.data_ptr(), tokens.data_ptr(), float(mult), T, D,
-          table.shape[0], _dt(table), _ptr(norm_weight), float(eps), _stream())
+          table.shape[0], _dt(table), _ptr(norm_weight), float(eps), _ptr(extra), mul_prev, mul_cur, buckets, _ptr(previous),
+          _ptr(seq_of), _ptr(cu), _ptr(slots), _stream())
 
 
 def add_postnorm_rmsnorm(h: Optional[Tensor], branches: Sequence[Tuple[Tensor, float]], post_weight: Tensor, post_eps: float,
-                         weight: Optional[Tensor], eps: float, out: Optional[Tensor], rows: Optional[Tensor] = None) -> None:
-    """u = rmsnorm(s0*b0 + s1*b1) * post_weight;  h <- h + u (rows is None and h given);  out = rmsnorm(h + u) * weight
+                         weight: Optional[Tensor], eps: float, out: Optional[Tensor], rows: Optional[Tensor] = None,
+                         bias: Optional[Tensor] = None) -> None:
+    """u = rmsnorm(s0*b0 + s1*b1 (+ bias)) * post_weight;  h <- h + u (rows is None and h given);  out = rmsnorm(h + u) * weight
     (``weight`` None: out = h + u, or u alone without h).  With ``rows`` h is left as it is and out[r] comes from row
     rows[r].  One or two branches in the storage type; every statistic and sum is float."""
-    _cuda(h, post_weight, weight, out, rows)
+    _cuda(h, post_weight, weight, out, rows, bias)
+    _f32vec(bias, branches[0][0].shape[-1], "add_postnorm_rmsnorm: bias")
     if not (1 <= len(branches) <= 2):
         raise KernelError("add_postnorm_rmsnorm: one or two branches")
     T, D = branches[0][0].shape
@@ -446,7 +496,7 @@ def add_postnorm_rmsnorm(h: Optional[Tensor], branches: Sequence[Tuple[Tensor, f
     if out is None and (h is None or rows is not None):
         raise KernelError("add_postnorm_rmsnorm: nothing to write")
     _call("pmm_add_postnorm_rmsnorm", _ptr(h), ptrs[0], scales[0], ptrs[1], scales[1], post_weight.data_ptr(),
-          float(post_eps), _ptr(weight), float(eps), _ptr(out), _ptr(rows), R, D, dtype, _stream())
+          float(post_eps), _ptr(weight), float(eps), _ptr(out), _ptr(rows), R, D, dtype, _ptr(bias), _stream())
 
 
 def add_rmsnorm(h: Tensor, branches: Sequence[Tuple[Tensor, float]], weight: Optional[Tensor],
@@ -1331,8 +1381,9 @@ def _skinny_x(x: Tensor, M: int, K: int, what: str) -> None:
         raise KernelError(f"{what}: x must be bfloat16 [M, K] with 16-byte aligned rows")
 
 
-def skinny_linear(x: Tensor, weight: Tensor, out: Tensor) -> None:
-    """out[M, N] = x @ weight^T for M <= 64 rows of bfloat16 activations (weights streamed once)."""
+def skinny_linear(x: Tensor, weight: Tensor, out: Tensor, gelu: bool = False) -> None:
+    """out[M, N] = x @ weight^T for M <= 64 rows of bfloat16 activations (weights streamed once); ``gelu``: the exact
+    form of GELU on the result."""
     _cuda(x, weight, out)
     M, K = x.shape
     _skinny_check(M, weight, K, "skinny_linear")
@@ -1342,8 +1393,29 @@ def skinny_linear(x: Tensor, weight: Tensor, out: Tensor) -> None:
     N = weight.shape[0]
     if not (out.dtype == torch.bfloat16 and out.shape == (M, N) and out.stride(1) == 1):
         raise KernelError("skinny_linear: out [M, N] bfloat16")
-    _call("pmm_skinny_gemm", 0, M, N, x.data_ptr(), x.stride(0), None, None, 0.0, weight.data_ptr(), K,
+    _call("pmm_skinny_gemm", 5 if gelu else 0, M, N, x.data_ptr(), x.stride(0), None, None, 0.0, weight.data_ptr(), K,
           1.0, None, 0, None, 0, 0.0, out.data_ptr(), out.stride(0), None, 1, _stream())
+
+
+SKINNY_MAX_PRODUCTS = 6
+
+
+def skinny_linears(xs: Sequence[Tensor], weights: Sequence[Tensor], outs: Sequence[Tensor]) -> None:
+    """outs[i] [M, N_i] = xs[i] @ weights[i]^T for up to six products of one K, M <= 64 rows, in one launch."""
+    n = len(xs)
+    _cuda(*xs, *weights, *outs)
+    M, K = xs[0].shape
+    if not (1 <= n <= SKINNY_MAX_PRODUCTS and len(weights) == n and len(outs) == n and skinny_fits(M, K)):
+        raise KernelError("skinny_linears: one to six products whose activations fit in shared memory")
+    for x, w, o in zip(xs, weights, outs):
+        _skinny_check(M, w, K, "skinny_linears")
+        _skinny_x(x, M, K, "skinny_linears")
+        if not (o.dtype == torch.bfloat16 and o.shape == (M, w.shape[0]) and o.stride(1) == 1):
+            raise KernelError("skinny_linears: outs [M, N] bfloat16")
+    px, pw, po = ((ctypes.c_void_p * n)(*[t.data_ptr() for t in ts]) for ts in (xs, weights, outs))
+    lx, lo = ((ctypes.c_longlong * n)(*[t.stride(0) for t in ts]) for ts in (xs, outs))
+    ns = (ctypes.c_int * n)(*[w.shape[0] for w in weights])
+    _call("pmm_skinny_multi", n, M, K, *(ctypes.cast(a, ctypes.c_void_p) for a in (px, lx, pw, ns, po, lo)), _stream())
 
 
 def skinny_linear_f32(x: Tensor, weight: Tensor, out: Tensor, scale: float, cap: float = 0.0) -> None:
@@ -1546,14 +1618,15 @@ def skinny_tc_supported(kind: str, x: Tensor, weight: Tensor, out: Optional[Tens
     return bool(_fn("pmm_skinny_tc_supported")(mode, T, n, K, 0, x.stride(0), 0, ldy))
 
 
-def skinny_tc_linear(x: Tensor, weight: Tensor, out: Tensor) -> None:
-    """out[T, N] (bfloat16) = x @ weight^T for up to 64 tokens on the tcgen05 tensor cores."""
+def skinny_tc_linear(x: Tensor, weight: Tensor, out: Tensor, gelu: bool = False) -> None:
+    """out[T, N] (bfloat16) = x @ weight^T for up to 64 tokens on the tcgen05 tensor cores; ``gelu``: the exact form of
+    GELU on the result."""
     _cuda(x, weight, out)
     if not (skinny_tc_supported("store", x, weight, out) and out.shape == (x.shape[0], weight.shape[0])):
         raise KernelError("skinny_tc_linear: operands not supported (bfloat16, <= 64 tokens, K <= 1024 and a "
                           "multiple of 8, aligned rows)")
     T, K = x.shape
-    _call("pmm_skinny_tc", 0, T, weight.shape[0], x.data_ptr(), x.stride(0), weight.data_ptr(), K, 1.0, None, 0, None, 0,
+    _call("pmm_skinny_tc", 3 if gelu else 0, T, weight.shape[0], x.data_ptr(), x.stride(0), weight.data_ptr(), K, 1.0, None, 0, None, 0,
           0.0, out.data_ptr(), out.stride(0), None, _tc_status(x.device).data_ptr(), _stream())
 
 
@@ -1641,8 +1714,9 @@ def tc_gemm_clamped_glu(x: Tensor, gate_up: Tensor, limit: float, alpha: float, 
           float(limit), float(alpha), float(shift), _tc_status(x.device).data_ptr(), _stream())
 
 
-def tc_gemm(x: Tensor, weight: Tensor, out: Tensor) -> None:
-    """out[T, N] = x @ weight^T on tcgen05 (bfloat16 in and out, float accumulation)."""
+def tc_gemm(x: Tensor, weight: Tensor, out: Tensor, gelu: bool = False) -> None:
+    """out[T, N] = x @ weight^T on tcgen05 (bfloat16 in and out, float accumulation); ``gelu``: the exact form of GELU in
+    the epilogue."""
     _cuda(x, weight, out)
     T, K = x.shape
     N = weight.shape[0]
@@ -1651,6 +1725,10 @@ def tc_gemm(x: Tensor, weight: Tensor, out: Tensor) -> None:
         raise KernelError("tc_gemm: out must be bfloat16 [T, N], rows 16-byte aligned")
     if not (tc_gemm_supported(x, weight, N, False)):
         raise KernelError("tc_gemm: sizes or alignment outside what the kernel takes")
+    if gelu:
+        _call("pmm_tc_gemm_act", 4, x.data_ptr(), x.stride(0), weight.data_ptr(), out.data_ptr(), out.stride(0), T, K, N,
+              1.0, 0.0, 0.0, _tc_status(x.device).data_ptr(), _stream())
+        return
     _call("pmm_tc_gemm", 0, x.data_ptr(), x.stride(0), weight.data_ptr(), out.data_ptr(), out.stride(0), T, K, N,
           1.0, _tc_status(x.device).data_ptr(), _stream())
 
@@ -1711,6 +1789,21 @@ def attention_tc(q: Tensor, pool: Tensor, block_table: Tensor, positions: Tensor
     if keep > 0:
         kept_first_merge(q, pool, block_table, positions, seq_of, out, lse, n_q_heads, n_kv_heads, head_dim, softmax_scale,
                          window, keep)
+
+
+def _unary(op: int, x: Tensor, what: str) -> None:
+    _cuda(x)
+    _call("pmm_unary", op, x.data_ptr(), _rows_view(x, what), x.shape[0], x.shape[1], _dt(x), _stream())
+
+
+def gelu_(x: Tensor) -> None:
+    """x = gelu(x) in place on a [T, F] view, the exact form z/2 (1 + erf(z / sqrt 2))."""
+    _unary(0, x, "gelu_")
+
+
+def tanh_(x: Tensor) -> None:
+    """x = tanh(x) in place on a [T, F] view."""
+    _unary(1, x, "tanh_")
 
 
 def silu_mul(gate_up: Tensor, gate_mult: float, out: Tensor) -> None:
@@ -2292,6 +2385,92 @@ def rope_pairs_store(q: Tensor, k: Tensor, v: Tensor, inv_freq: Optional[Tensor]
           -1.0 if v_norm_eps is None else float(v_norm_eps), _dt(q), _stream())
 
 
+def head_norm_rope_store(q: Tensor, k: Tensor, v: Tensor, inv_freq: Optional[Tensor], rot_dims: int, positions: Tensor,
+                         seq_of: Tensor, block_table: Tensor, pool: Tensor, q_out: Tensor, n_heads: int, n_kv_heads: int,
+                         dim: int, vdim: int, padded_dim: int, half_layout: bool = False, amplitude: float = 1.0,
+                         biases: Optional[Tuple[Tensor, Tensor, Tensor]] = None, norm_eps: Optional[float] = None,
+                         norm_weights: Optional[Tuple[Tensor, Tensor]] = None, values: Optional[Tensor] = None,
+                         mix_weight: Optional[Tensor] = None) -> None:
+    """The preparation of `rope_pairs_store` with a norm per head: biases, then (``norm_eps``) every query and key head
+    over its own root mean square, times ``norm_weights`` [dim] (queries', keys') where given, then rotation with
+    sines and cosines times ``amplitude``; queries to q_out [T, H*Dp], keys and values into their pages.  ``values`` [T,
+    G*dv]: with ``mix_weight`` (one float l) the values become (1 - l) v + l values, without it they are left there."""
+    _cuda(q, k, v, inv_freq, positions, seq_of, block_table, pool, q_out, values, mix_weight)
+    what = "head_norm_rope_store"
+    qb = kb = vb = qw = kw = None
+    if biases is not None:
+        qb, kb, vb = biases
+        _cuda(qb, kb, vb)
+        _f32vec(qb, n_heads * dim, f"{what}: q bias")
+        _f32vec(kb, n_kv_heads * dim, f"{what}: k bias")
+        _f32vec(vb, n_kv_heads * vdim, f"{what}: v bias")
+    if norm_weights is not None:
+        qw, kw = norm_weights
+        _cuda(qw, kw)
+        _f32vec(qw, dim, f"{what}: q norm weight")
+        _f32vec(kw, dim, f"{what}: k norm weight")
+        if norm_eps is None:
+            raise KernelError(f"{what}: norm weights need norm_eps")
+    T = q.shape[0]
+    ld_q, ld_k, ld_v = (_rows_view(t, what) for t in (q, k, v))
+    if not (q.shape[1] == n_heads * dim and k.shape == (T, n_kv_heads * dim) and v.shape == (T, n_kv_heads * vdim)
+            and q.dtype == k.dtype == v.dtype == pool.dtype == q_out.dtype):
+        raise KernelError(f"{what}: q [T, H*d], k [T, G*d], v [T, G*dv] of the pool's type")
+    if not (pool.dim() == 4 and pool.shape[1] == 2 and pool.shape[3] == n_kv_heads * padded_dim and pool.is_contiguous()
+            and q_out.shape == (T, n_heads * padded_dim) and q_out.is_contiguous()):
+        raise KernelError(f"{what}: pool [pages, 2, page_size, G*Dp], q_out [T, H*Dp]")
+    if values is not None and not (values.shape == (T, n_kv_heads * vdim) and values.is_contiguous() and values.dtype == v.dtype):
+        raise KernelError(f"{what}: values must be contiguous [T, G*dv] of v's type")
+    if mix_weight is not None:
+        _f32vec(mix_weight, 1, f"{what}: mix weight")
+        if values is None:
+            raise KernelError(f"{what}: a mix weight needs values to mix with")
+    if rot_dims > 0:
+        _f32vec(inv_freq, rot_dims // 2, f"{what}: inv_freq")
+    for t in (positions, seq_of, block_table):
+        _i32(t, what)
+    _call("pmm_head_norm_rope_store", q.data_ptr(), ld_q, k.data_ptr(), ld_k, v.data_ptr(), ld_v, _ptr(inv_freq),
+          positions.data_ptr(), seq_of.data_ptr(), block_table.data_ptr(), block_table.shape[1], pool.data_ptr(), pool.shape[2],
+          q_out.data_ptr(), T, n_heads, n_kv_heads, dim, vdim, padded_dim, int(rot_dims), int(bool(half_layout)),
+          float(amplitude), _ptr(qb), _ptr(kb), _ptr(vb), -1.0 if norm_eps is None else float(norm_eps), _ptr(qw), _ptr(kw),
+          _ptr(values), _ptr(mix_weight), _dt(q), _stream())
+
+
+# ----------------------------------------------------------------------------- inputs that look one token back
+def shifted_mixes(x: Tensor, mu: Tensor, state: Tensor, cu: Tensor, slots: Tensor, seq_of: Tensor, out: Tensor) -> None:
+    """out[s, t] = x_t + (x_(t-1) - x_t) mu[s] with x_(t-1) the row before of the same request: ``state`` (float32
+    [slots, D], zero for a new request) holds it for the first token of a step and is brought up to date.  out [n, >= T, D]
+    contiguous, of x's type; mu [n, D] float32, n <= 8."""
+    _cuda(x, mu, state, cu, slots, seq_of, out)
+    T, D = x.shape
+    n = mu.shape[0]
+    if not (mu.dtype == torch.float32 and mu.is_contiguous() and mu.shape == (n, D) and state.dtype == torch.float32
+            and state.is_contiguous() and state.dim() == 2 and state.shape[1] == D):
+        raise KernelError("shifted_mixes: mu [n, D] and state [slots, D], contiguous float32")
+    if not (out.dim() == 3 and out.shape[0] == n and out.shape[1] >= T and out.shape[2] == D and out.is_contiguous()
+            and out.dtype == x.dtype and seq_of.numel() == T):
+        raise KernelError("shifted_mixes: out [n, >= T, D] of x's type")
+    for t in (cu, slots, seq_of):
+        _i32(t, "shifted_mixes")
+    _call("pmm_shifted_mixes", x.data_ptr(), _rows_view(x, "shifted_mixes"), mu.data_ptr(), n, state.data_ptr(), cu.data_ptr(),
+          slots.data_ptr(), seq_of.data_ptr(), out.data_ptr(), out.stride(0), T, D, _dt(x), _stream())
+
+
+LOW_RANK_TANH_MAX_TOKENS = 128  # bfloat16 steps of more tokens take the library's product on tanh'd rows
+
+
+def low_rank_tanh(z: Tensor, w: Tensor, out: Tensor) -> None:
+    """out [T, C] (float32) = tanh(z) [T, R] @ w [C, R]^T in float arithmetic."""
+    _cuda(z, w, out)
+    T, R = z.shape
+    C = w.shape[0]
+    if not (w.shape == (C, R) and w.is_contiguous() and w.dtype == z.dtype and out.shape == (T, C) and out.is_contiguous()
+            and out.dtype == torch.float32):
+        raise KernelError("low_rank_tanh: w [C, R] of z's type, out contiguous float32 [T, C]")
+    _call("pmm_low_rank_tanh", z.data_ptr(), _rows_view(z, "low_rank_tanh"), w.data_ptr(), out.data_ptr(), T, C, R, _dt(z),
+          _stream())
+
+
 # ----------------------------------------------------------------------------- matrix-state recurrences
 RECURRENT_MAX_KEY_DIM = 256
 
@@ -2345,6 +2524,69 @@ def decay_scan(q: Tensor, k: Tensor, v: Tensor, decay: Tensor, state: Tensor, cu
 
 
 RECURRENT_CHUNK = 64  # tokens per chunk of the chunked recurrences
+
+
+RECURRENCE_RULES = {"retention": 2, "wkv": 3}
+
+
+def recurrence_chunked_supported(rule: str, dim: int) -> bool:
+    """Whether the chunked kernels take this key size (a multiple of 4 whose operands fit one block)."""
+    return bool(_fn("pmm_recurrent_chunked_supported")(int(dim), RECURRENCE_RULES[rule]))
+
+
+def recurrence_scratch_floats(rule: str, new_lens: Sequence[int], n_heads: int, dim: int, vdim: int) -> int:
+    f = _fn("pmm_recurrent_chunked_scratch")
+    f.restype = c_longlong
+    return recurrent_chunks(new_lens) * n_heads * int(f(int(dim), int(vdim), RECURRENCE_RULES[rule])) + 4
+
+
+def recurrence(rule: str, q: Tensor, k: Tensor, v: Tensor, state: Tensor, cu: Tensor, slots: Tensor, new_lens: Sequence[int],
+               out: Tensor, n_heads: int, dim: int, vdim: int, scratch: Optional[Tensor] = None, decay: Optional[Tensor] = None,
+               k_scale: float = 1.0, positions: Optional[Tensor] = None, inv_freq: Optional[Tensor] = None, rot_dims: int = 0,
+               half_layout: bool = True, a: Optional[Tensor] = None, a_bias: Optional[Tensor] = None,
+               bonus: Optional[Tensor] = None) -> None:
+    """A matrix-state recurrence over the step's tokens, state [slots, H, d, dv] float32 carried between steps; q, k [T, H*d],
+    v [T, H*dv] of one type, out [T, H*dv] float32.  ``rule`` "retention": q and k turn in pairs by ``positions`` and
+    ``inv_freq`` (rot_dims entries of every head, pairs (i, i + rot_dims/2) with ``half_layout``, else (2i, 2i+1)), k is
+    multiplied by ``k_scale``, S <- decay_h S + k v^T, o = S^T q.  "wkv": o = (S + diag(bonus) k v^T)^T q, S <- diag(w) S +
+    k v^T, w = exp(-exp(a + a_bias)) with a [T, H*d] float32, a_bias and bonus [H*d].  With ``scratch``
+    (`recurrence_scratch_floats` floats) in chunks of 64 tokens, else token by token."""
+    what = f"recurrence '{rule}'"
+    _cuda(q, k, v, state, cu, slots, out, scratch, decay, positions, inv_freq, a, a_bias, bonus)
+    T, ld_q, ld_k, ld_v = _recurrent_common(q, k, v, state, cu, slots, out, n_heads, n_heads, dim, vdim, what)
+    ld_a = 0
+    if rule == "retention":
+        if decay is None:
+            raise KernelError(f"{what}: needs a decay per head")
+        _f32vec(decay, n_heads, f"{what}: decay")
+        if rot_dims > 0:
+            if not (rot_dims % 2 == 0 and rot_dims <= dim and positions is not None and inv_freq is not None):
+                raise KernelError(f"{what}: rotation needs an even number of entries, positions and frequencies")
+            _f32vec(inv_freq, rot_dims // 2, f"{what}: inv_freq")
+            _i32(positions, f"{what}: positions")
+    elif rule == "wkv":
+        if a is None or a_bias is None or bonus is None or decay is not None:
+            raise KernelError(f"{what}: needs a, a_bias and bonus")
+        if not (a.dtype == torch.float32 and a.shape == (T, n_heads * dim)):
+            raise KernelError(f"{what}: a must be float32 [T, H*d]")
+        ld_a = _rows_view(a, f"{what}: a")
+        _f32vec(a_bias, n_heads * dim, f"{what}: a_bias")
+        _f32vec(bonus, n_heads * dim, f"{what}: bonus")
+    else:
+        raise KernelError(f"unknown recurrence rule '{rule}'")
+    args = (q.data_ptr(), ld_q, k.data_ptr(), ld_k, v.data_ptr(), ld_v, _ptr(decay), float(k_scale), _ptr(positions),
+            _ptr(inv_freq), int(rot_dims), int(bool(half_layout)), _ptr(a), ld_a, _ptr(a_bias), _ptr(bonus), state.data_ptr(),
+            cu.data_ptr(), slots.data_ptr(), out.data_ptr())
+    if scratch is None:
+        _call("pmm_recurrence", *args, len(new_lens), n_heads, dim, vdim, _dt(q), _stream())
+        return
+    need = recurrence_scratch_floats(rule, new_lens, n_heads, dim, vdim)
+    if not (recurrence_chunked_supported(rule, dim) and scratch.dtype == torch.float32 and scratch.is_contiguous()
+            and scratch.numel() >= need):
+        raise KernelError(f"{what}: key size {dim} in chunks needs {need} floats of scratch")
+    base = scratch.data_ptr()
+    base += (-base) % 16
+    _call("pmm_recurrence_chunked", *args, base, len(new_lens), recurrent_chunks(new_lens), n_heads, dim, vdim, _dt(q), _stream())
 
 
 def recurrent_chunked_supported(dim: int, delta: bool) -> bool:

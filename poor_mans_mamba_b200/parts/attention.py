@@ -28,11 +28,11 @@ _TC_ATTENTION = os.environ.get("PMM_TCGEN05_ATTENTION", "1") == "1"
 
 
 def plan_key_splits_tc(num_heads: int, num_kv_heads: int, window: int, new_lens, kv_len_bound: int):
-    """Key ranges for the tcgen05 kernel (128 rows a block, two blocks an SM): one range when
+    """(``window`` below zero: chunks of -window positions.)  Key ranges for the tcgen05 kernel (128 rows a block, two blocks an SM): one range when
     the row tiles alone give a block per SM, else enough ranges of at least 256 keys to get there."""
     per_tile = 128 // (num_heads // num_kv_heads)
     blocks = sum((n + per_tile - 1) // per_tile for n in new_lens) * num_kv_heads
-    reach = min(kv_len_bound, window) if window > 0 else kv_len_bound
+    reach = min(kv_len_bound, abs(window)) if window != 0 else kv_len_bound
     want = min(_TC_BLOCKS // max(blocks, 1), (reach + 255) // 256)
     if want <= 1:
         return 1, 0
@@ -59,7 +59,7 @@ def plan_key_splits(num_heads: int, num_kv_heads: int, head_dim: int, window: in
         blocks = sum(new_lens) * ((num_heads + 3) // 4)
         min_len = 128
         target = _TARGET_BLOCKS
-    reach = min(kv_len_bound, window) if window > 0 else kv_len_bound
+    reach = min(kv_len_bound, abs(window)) if window != 0 else kv_len_bound
     if blocks >= target or reach <= min_len:
         return 1, 0
     if dtype == torch.bfloat16 and min_len == 256:

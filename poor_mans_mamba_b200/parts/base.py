@@ -49,9 +49,10 @@ class StateSpec:
     kind "paged": ``planes`` rows of ``width`` elements per token (keys and values: 2
     planes), kept in pages through a block table; ``window`` > 0 means only the last
     ``window`` tokens are ever read, so older pages can be given back; ``keep_first`` > 0: the first
-    ``keep_first`` tokens are read for ever as well, so the pages they lie in stay.
+    ``keep_first`` tokens are read for ever as well, so the pages they lie in stay.  ``chunk`` > 0 instead: a token
+    only reads its own chunk of ``chunk`` positions (chunks counted from position 0), so the pages before it can go.
     kind "fixed": one tensor of ``shape`` per request, kept in a slot; zero for a new
-    request.  dtype "compute" follows the engine's storage type, "float32" stays 32-bit.
+    request.  dtype "compute" follows the engine's storage type, "float32" stays 32-bit, "int32" holds integers.
     """
     name: str
     kind: str
@@ -59,13 +60,15 @@ class StateSpec:
     width: int = 0
     window: int = 0
     keep_first: int = 0
+    chunk: int = 0
     shape: Tuple[int, ...] = ()
     dtype: str = "compute"
 
     @staticmethod
-    def paged(name: str, planes: int, width: int, window: int = 0, keep_first: int = 0) -> "StateSpec":
+    def paged(name: str, planes: int, width: int, window: int = 0, keep_first: int = 0,
+              chunk: int = 0) -> "StateSpec":
         return StateSpec(name=name, kind="paged", planes=planes, width=width, window=window,
-                         keep_first=keep_first if window > 0 else 0)
+                         keep_first=keep_first if window > 0 else 0, chunk=chunk)
 
     @staticmethod
     def fixed(name: str, shape: Sequence[int], dtype: str = "float32") -> "StateSpec":
@@ -127,6 +130,11 @@ class Norm(Part):
     # launch of its own (``apply``) and the result waits as an ordinary branch.
     def folds_post(self, post: "Norm") -> bool:
         """Whether `forward(..., post=post)` applies ``post`` to the sum of the pending branches itself."""
+        return False
+
+    def folds_post_bias(self) -> bool:
+        """As a post norm: whether `forward(..., post=this, post_bias=b)`, `apply` and `fold` take a vector b [D] (float32)
+        that joins the sublayer's result before it is normed (an output projection's bias)."""
         return False
 
     def apply(self, pending, out: Tensor, ctx) -> None:
@@ -203,6 +211,12 @@ class Mixer(Part):
         columns, sum_m scale_m * y_m W_m^T = [scale_0 y_0 | scale_1 y_1 | ...] [W_0 | W_1 | ...]^T."""
         return False
 
+    def carries(self) -> Dict[str, int]:
+        """Rows [T, width] in the storage type, by name, that this mixer leaves for (or takes from) mixers of later
+        layers of the same step: the model makes one matrix per name for the step and hands them over as
+        ``ctx.carried``."""
+        return {}
+
     def joins_output_products(self) -> bool:
         """Whether `pre_output_into` is available for this mixer as it is configured."""
         return False
@@ -256,6 +270,21 @@ class InputMap(Part):
 
     def forward(self, x: Tensor, ctx, cache: "LayerCache", out: Tensor) -> None:
         raise NotImplementedError
+
+
+class EmbeddingAddend(Part):
+    """A row that joins the embedding's row of every token and may depend on the tokens before it, through state of
+    its own (kept under the cache id EMBEDDING_CACHE): ``arguments(ctx, cache)`` are what the embedding's launch needs
+    to add it (see `kernels.ops.embed`)."""
+
+    def state_specs(self) -> List[StateSpec]:
+        return []
+
+    def arguments(self, ctx, cache: "LayerCache") -> Dict[str, Any]:
+        raise NotImplementedError
+
+
+EMBEDDING_CACHE = -1   # the cache id of what the embedding keeps per request
 
 
 class StreamUpdate(Part):
@@ -328,6 +357,8 @@ class ModelSpec:
     # A norm applied to the embedding's output before the first layer (in float, inside the embedding launch;
     # an RMS norm: one whose `rms_prologue` answers).
     embedding_norm: Optional[PartSpec] = None
+    # Rows that join the embedding's (`register_embedding_addend`), added in the embedding's launch before its norm.
+    embedding_addend: Optional[PartSpec] = None
     # > 0: logits <- logit_softcap * tanh(logits / logit_softcap), after the head's multiplier.
     logit_softcap: float = 0.0
     # None: one residual stream [T, D].  n >= 1: the residual state is n lanes [n, T, D], all equal to
@@ -339,7 +370,7 @@ class ModelSpec:
 # ----------------------------------------------------------------------------- registries
 _REGISTRIES: Dict[str, Dict[str, Callable[..., Part]]] = {
     "mixer": {}, "feed_forward": {}, "norm": {}, "position_encoding": {}, "arrangement": {}, "stream_update": {},
-    "input_map": {},
+    "input_map": {}, "embedding_addend": {},
 }
 
 
@@ -376,6 +407,10 @@ def register_stream_update(kind: str, factory: Callable[..., "StreamUpdate"]) ->
 
 def register_input_map(kind: str, factory: Callable[..., "InputMap"]) -> None:
     _register("input_map", kind, factory)
+
+
+def register_embedding_addend(kind: str, factory: Callable[..., "EmbeddingAddend"]) -> None:
+    _register("embedding_addend", kind, factory)
 
 
 def build_part(family: str, spec: PartSpec, **extra: Any) -> Any:

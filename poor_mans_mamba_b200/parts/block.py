@@ -78,6 +78,7 @@ class ResidualStream:
         self.pending: List[Tuple[Tensor, float]] = []
         self.pending_vector: Optional[Tensor] = None  # [D] float32, waits to join every row of the stream
         self.pending_post: Optional[Norm] = None  # normed once more before the pending branches join (see Norm.folds_post)
+        self.pending_bias: Optional[Tensor] = None  # [D] float32, part of what waits with the post norm (inside that norm)
         self._buffers = [ctx.workspace.alloc(tuple(h.shape), ctx.dtype) for _ in range(n_branch_buffers)]
         self._taken = 0
         # Residual state in lanes [n, T, D] (see ModelSpec.residual_lanes): every lane starts as h, so
@@ -122,12 +123,18 @@ class ResidualStream:
             self._settle_post()  # what waits with a post norm is one sublayer's result: settle it first
         self.pending.append((branch, float(scale)))
 
-    def add_normed(self, branches: Sequence[Tuple[Tensor, float]], post: Norm) -> None:
-        """A sublayer's result sum(scale_i * branch_i) waits to join the stream as post(that sum)."""
+    def add_normed(self, branches: Sequence[Tuple[Tensor, float]], post: Norm, bias: Optional[Tensor] = None) -> None:
+        """A sublayer's result sum(scale_i * branch_i) (+ ``bias``, with a post norm that `folds_post_bias`) waits to
+        join the stream as post(that sum)."""
         if self.pending or self.pending_vector is not None:
             self.flush()
         self.pending = [(b, float(s)) for b, s in branches]
-        self.pending_post = post
+        self.pending_post, self.pending_bias = post, bias
+
+    def _post_bias(self) -> dict:
+        """The waiting bias as an argument of the waiting post norm's launch (which takes it over)."""
+        bias, self.pending_bias = self.pending_bias, None
+        return {} if bias is None else {"post_bias": bias}
 
     def _settle_post(self) -> None:
         """Apply the waiting post norm by a launch of its own; its result waits as an ordinary branch."""
@@ -135,7 +142,7 @@ class ResidualStream:
         if post is None or not self.pending:
             return
         out = self.take_branch()  # (arrangements with post norms ask for one buffer more)
-        post.apply(self.pending, out, self.ctx)
+        post.apply(self.pending, out, self.ctx, **self._post_bias())
         self.pending = [(out, 1.0)]
 
     def lane_add(self, y: Tensor, mix: Tensor, out_w: Tensor) -> None:
@@ -178,13 +185,14 @@ class ResidualStream:
                 return out
             self._settle_vector()
         if self.pending_post is not None and self.pending and norm.folds_post(self.pending_post):
-            norm.forward(self.h, self.pending, out, rows, self.ctx, post=self.pending_post)
+            bias = {} if self.pending_bias is None else {"post_bias": self.pending_bias}
+            norm.forward(self.h, self.pending, out, rows, self.ctx, post=self.pending_post, **bias)
         else:
             self._settle_post()
             norm.forward(self.h, self.pending, out, rows, self.ctx)
         if rows is None:
             self.pending = []
-            self.pending_post = None
+            self.pending_post = self.pending_bias = None
             self._taken = 0
         return out
 
@@ -235,7 +243,7 @@ class ResidualStream:
             raise RuntimeError("a residual state in lanes has no single stream to flush into")
         self._settle_vector()
         if self.pending_post is not None and self.pending:
-            self.pending_post.fold(self.h, self.pending, self.ctx)
+            self.pending_post.fold(self.h, self.pending, self.ctx, **self._post_bias())
         else:
             fold_branches(self.h, self.pending)
         self.pending = []
@@ -422,6 +430,7 @@ class ParallelPreNormBlock(Part):
             return
         ws = ctx.workspace
         mark = ws.mark()
+        bias: Optional[Tensor] = None
         n = stream.normed_mapped(self.mixer_norm, self.mixer_input, cache)
         if self._fused_in is not None:
             proj = ws.alloc((n.shape[0], self._fused_in.shape[0]), n.dtype)
@@ -459,15 +468,20 @@ class ParallelPreNormBlock(Part):
                 streaming.linear(joined, self._fused_out, outs[0], ctx)
         else:
             outs = []
+            # a lone mixer's output bias is added where its result is normed
+            if len(self.mixers) == 1 and self.mixer_post_norm is not None and self.mixer_post_norm.folds_post_bias():
+                bias = self.mixers[0].output_bias()
+            ctx.defer_output_bias = bias is not None
             for m in self.mixers:
                 outs.append(stream.take_branch())
                 m.forward(n, ctx, cache, outs[-1])
+            ctx.defer_output_bias = False
         if self._fused_in is not None and self._fused_out is not None:
             results = [(outs[0], 1.0)]
         else:
             results = [(out, m.out_scale) for m, out in zip(self.mixers, outs)]
         if self.mixer_post_norm is not None:
-            stream.add_normed(results, self.mixer_post_norm)
+            stream.add_normed(results, self.mixer_post_norm, bias)
         else:
             for out, scale in results:
                 stream.add(out, scale)

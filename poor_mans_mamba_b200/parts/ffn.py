@@ -1,4 +1,4 @@
-"""Dense gated feed-forward (SwiGLU, or the same with the tanh form of GELU on the gate).
+"""Dense feed-forwards: gated (SwiGLU, or the same with the tanh form of GELU on the gate) and plain (`MLP`).
 
 g = (x Wg^T) * gate_multiplier; u = x Wu^T; out = (act(g) * u) Wd^T with act = silu, or with
 ``activation`` "gelu_tanh" act(z) = 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))); the down
@@ -95,4 +95,41 @@ class SwiGLU(FeedForward):
         return [self.gate_up, self.down]
 
 
+class MLP(FeedForward):
+    """Dense feed-forward without a gate: out = act(x Wu^T) Wd^T with ``activation`` "gelu", the exact form
+    act(z) = z/2 (1 + erf(z / sqrt 2)).  The activation is in the first product's epilogue: of the weight-streaming
+    product in steps of few tokens, of the tcgen05 product in steps of many."""
+
+    def __init__(self, hidden_size: int, intermediate_size: int, activation: str = "gelu", tensors=("up", "down"),
+                 down_multiplier: float = 1.0):
+        if activation != "gelu":
+            raise ValueError("activation is 'gelu'")
+        self.hidden_size, self.intermediate_size = int(hidden_size), int(intermediate_size)
+        self.tensors = tuple(tensors)
+        self.out_scale = float(down_multiplier)
+
+    def param_specs(self) -> List[ParamSpec]:
+        f, d = self.intermediate_size, self.hidden_size
+        return [ParamSpec(self.tensors[0], (f, d)), ParamSpec(self.tensors[1], (d, f))]
+
+    def bind(self, params: Dict[str, Tensor]) -> None:
+        self.up, self.down = (params[n].contiguous() for n in self.tensors)
+
+    def forward(self, x: Tensor, ctx, out: Tensor) -> None:
+        T, f = x.shape[0], self.intermediate_size
+        act = ctx.workspace.alloc((T, f), x.dtype)
+        if not streaming.gelu_linear(x, self.up, act, ctx):
+            tiles = ((T + 255) // 256) * (f // 256)
+            if _TC_ENABLED and tiles >= _TC_FROM_TILES and K.tc_gemm_supported(x, self.up, f, False):
+                K.tc_gemm(x, self.up, act, gelu=True)
+            else:
+                K.linear(x, self.up, act)
+                K.gelu_(act)
+        streaming.linear(act, self.down, out, ctx)
+
+    def streamed_weights(self) -> List[Tensor]:
+        return [self.up, self.down]
+
+
 register_feed_forward("swiglu", SwiGLU)
+register_feed_forward("mlp", MLP)

@@ -32,17 +32,20 @@ def fold_branches(h: Tensor, pending) -> None:
 
 class RMSNorm(Norm):
     """``offset``: the stored weight is kept around zero and the norm multiplies by offset + w (the sum
-    is made once, in float32, when the tensors are bound).  ``tensor``: the weight's name within the
+    is made once, in float32, when the tensors are bound).  ``multiplier``: a constant that the weight takes in (as a
+    post norm: the factor with which the normed result joins the stream).  ``tensor``: the weight's name within the
     part ("" where the part's own name is the tensor's).  ``groups``: the row is cut into that many equal
     neighbouring parts and each is divided by its own root mean square."""
 
-    def __init__(self, width: int, eps: float, offset: float = 0.0, tensor: str = "weight", groups: int = 1):
+    def __init__(self, width: int, eps: float, offset: float = 0.0, tensor: str = "weight", groups: int = 1,
+                 multiplier: float = 1.0):
         if groups < 1 or width % groups:
             raise ValueError("the norm's groups must divide the width")
         self.groups = int(groups)
         self.width = int(width)
         self.eps = float(eps)
         self.offset = float(offset)
+        self.multiplier = float(multiplier)
         self.tensor = str(tensor)
         self.weight: Optional[Tensor] = None
 
@@ -52,7 +55,11 @@ class RMSNorm(Norm):
 
     def bind(self, params: Dict[str, Tensor]) -> None:
         w = params[self.tensor]
-        self.weight = w if self.offset == 0.0 else (w + self.offset).contiguous()
+        if self.offset != 0.0:
+            w = w + self.offset
+        if self.multiplier != 1.0:
+            w = w * self.multiplier
+        self.weight = w.contiguous()
 
     def rms_prologue(self):
         return (self.weight, self.eps) if self.groups == 1 else None
@@ -63,13 +70,17 @@ class RMSNorm(Norm):
     def folds_post(self, post: Norm) -> bool:
         return isinstance(post, RMSNorm) and self.groups == 1 and post.groups == 1
 
-    def forward(self, h: Tensor, pending, out: Tensor, rows: Optional[Tensor], ctx, post: Optional[Norm] = None) -> None:
+    def folds_post_bias(self) -> bool:
+        return self.groups == 1
+
+    def forward(self, h: Tensor, pending, out: Tensor, rows: Optional[Tensor], ctx, post: Optional[Norm] = None,
+                post_bias: Optional[Tensor] = None) -> None:
         items = list(pending)
         if post is not None and items:
             # a sublayer's result, normed once more before it joins: x <- x + post(sum), out = norm(x), one launch
             if not self.folds_post(post) or len(items) > 2:
                 raise ValueError("the RMS norm folds a post norm of its own kind over at most two branches")
-            K.add_postnorm_rmsnorm(h, items, post.weight, post.eps, self.weight, self.eps, out, rows)
+            K.add_postnorm_rmsnorm(h, items, post.weight, post.eps, self.weight, self.eps, out, rows, bias=post_bias)
             return
         while len(items) > 2:  # more than two branches: fold the surplus first
             if rows is not None:
@@ -85,13 +96,13 @@ class RMSNorm(Norm):
         if self.groups > 1:
             raise NotImplementedError("an RMS norm over groups of channels cannot norm a sublayer's result")
 
-    def apply(self, pending, out: Tensor, ctx) -> None:
+    def apply(self, pending, out: Tensor, ctx, post_bias: Optional[Tensor] = None) -> None:
         self._whole_row()
-        K.add_postnorm_rmsnorm(None, list(pending), self.weight, self.eps, None, 0.0, out)
+        K.add_postnorm_rmsnorm(None, list(pending), self.weight, self.eps, None, 0.0, out, bias=post_bias)
 
-    def fold(self, h: Tensor, pending, ctx) -> None:
+    def fold(self, h: Tensor, pending, ctx, post_bias: Optional[Tensor] = None) -> None:
         self._whole_row()
-        K.add_postnorm_rmsnorm(h, list(pending), self.weight, self.eps, None, 0.0, None)
+        K.add_postnorm_rmsnorm(h, list(pending), self.weight, self.eps, None, 0.0, None, bias=post_bias)
 
 
 class TanhNorm(Norm):

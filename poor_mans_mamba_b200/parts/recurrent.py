@@ -10,6 +10,11 @@
 ``DecayLinearAttention`` ("decay_linear_attention"): linear attention with a fixed decay per head.
     q, k = silu(W x) (heads x dim), v = silu(Wv x) (heads x vdim);  S <- decay_h S + k v^T;  o = S^T q;
     out = Wo [ rmsnorm(o over all heads) * norm * sigmoid(Wg x) ].
+``Retention`` ("retention"): linear attention with a fixed decay per head and rotated queries and keys.
+    q = Wq x, k = Wk x (heads x dim), v = Wv x (heads x vdim);  among the first rot_dims entries of every q and k
+    head, entry i and entry i + rot_dims/2 turn together by the angle p * rot_base^(-2i / rot_dims) (``rot_layout``
+    "pairs": entries 2i and 2i+1);  k * dim^-1/2;  S <- decay_h S + k v^T;  o = S^T q;
+    out = Wo [ (o / sqrt(mean(o^2) + eps) per head) * silu(Wg x) ].
 
 State per request (float32, in a slot, zero for a new request): S [heads, dim, vdim]; the gated
 delta mixer also keeps the last taps - 1 inputs of its convolution.  Decays, gates, unit lengths,
@@ -26,12 +31,23 @@ from ..kernels import ops as K
 from . import streaming
 from . import branches
 from .base import Mixer, ParamSpec, StateSpec, register_mixer
+from .rope import rotary_frequencies
 
 Tensor = torch.Tensor
 
 # Steps whose longest portion has at least this many tokens walk it in chunks (two launches with a
 # fixed cost of tens of microseconds) instead of token by token (about a microsecond a token).
 _CHUNKED_FROM = 32
+
+
+def run_recurrence(rule: str, q: Tensor, k: Tensor, v: Tensor, state: Tensor, ctx, o: Tensor, heads: int, dim: int, vdim: int,
+                   **operands) -> None:
+    """The recurrence ``rule`` ("retention" or "wkv", see `kernels.ops.recurrence`) over the step's tokens into o [T,
+    heads * vdim] (float32): prompt portions in chunks, short steps token by token."""
+    scratch = None
+    if not ctx.decode_only and max(ctx.new_lens) >= _CHUNKED_FROM and K.recurrence_chunked_supported(rule, dim):
+        scratch = ctx.workspace.alloc((K.recurrence_scratch_floats(rule, ctx.new_lens, heads, dim, vdim),), torch.float32)
+    K.recurrence(rule, q, k, v, state, ctx.cu_seqlens, ctx.slots, ctx.new_lens, o, heads, dim, vdim, scratch=scratch, **operands)
 
 
 def _chunked(ctx, dim: int, delta: bool) -> bool:
@@ -207,5 +223,59 @@ class DecayLinearAttention(_StackedInput):
         streaming.linear(y, self.w_out, out, ctx)
 
 
+class Retention(_StackedInput):
+    def __init__(self, hidden_size: int, heads: int, dim: int, vdim: int, decay: Sequence[float], norm_eps: float,
+                 rot_dims: int = 0, rot_base: float = 1.0, rot_layout: str = "halves", out_multiplier: float = 1.0):
+        if len(decay) != heads:
+            raise ValueError("one decay per head")
+        if dim > K.RECURRENT_MAX_KEY_DIM:
+            raise ValueError(f"the recurrence kernels take key sizes up to {K.RECURRENT_MAX_KEY_DIM}, got {dim}")
+        if rot_dims % 2 or not 0 <= rot_dims <= dim:
+            raise ValueError("rot_dims must be even and at most dim")
+        if rot_layout not in ("halves", "pairs"):
+            raise ValueError("rot_layout is 'halves' or 'pairs'")
+        self.hidden_size = int(hidden_size)
+        self.heads, self.dim, self.vdim = int(heads), int(dim), int(vdim)
+        self.decay_values, self.norm_eps = tuple(float(a) for a in decay), float(norm_eps)
+        self.rot_dims, self.rot_base, self.half_layout = int(rot_dims), float(rot_base), rot_layout == "halves"
+        self.out_scale = float(out_multiplier)
+        self.qk_dim, self.v_dim = self.heads * self.dim, self.heads * self.vdim
+        self.inv_freq: Optional[Tensor] = None
+
+    def param_specs(self) -> List[ParamSpec]:
+        D = self.hidden_size
+        return [ParamSpec("q", (self.qk_dim, D)), ParamSpec("k", (self.qk_dim, D)), ParamSpec("v", (self.v_dim, D)),
+                ParamSpec("g", (self.v_dim, D)), ParamSpec("o", (D, self.v_dim))]
+
+    def state_specs(self) -> List[StateSpec]:
+        return [StateSpec.fixed("S", (self.heads, self.dim, self.vdim), "float32")]
+
+    def bind(self, params: Dict[str, Tensor]) -> None:
+        self.w_in = torch.cat([params["q"], params["k"], params["v"], params["g"]], dim=0).contiguous()
+        self.w_out = params["o"].contiguous()
+        self.decay = torch.tensor(self.decay_values, dtype=torch.float32, device=self.w_out.device)
+        self.unit_w = torch.ones(self.v_dim, dtype=torch.float32, device=self.w_out.device)
+
+    def finalize(self, dtype: torch.dtype, device: torch.device) -> None:
+        if self.rot_dims > 0:
+            self.inv_freq = rotary_frequencies(self.rot_dims, self.rot_base).to(device).contiguous()
+
+    def output_weight(self) -> Tensor:
+        return self.w_out
+
+    def forward_projected(self, proj: Tensor, ctx, cache, out: Tensor) -> None:
+        T = proj.shape[0]
+        ws = ctx.workspace
+        qk, vd = self.qk_dim, self.v_dim
+        o = ws.alloc((T, vd), torch.float32)
+        run_recurrence("retention", proj[:, :qk], proj[:, qk:2 * qk], proj[:, 2 * qk:2 * qk + vd], cache.fixed(f"{self.name}.S"),
+                       ctx, o, self.heads, self.dim, self.vdim, decay=self.decay, k_scale=float(self.dim) ** -0.5,
+                       positions=ctx.positions, inv_freq=self.inv_freq, rot_dims=self.rot_dims, half_layout=self.half_layout)
+        y = ws.alloc((T, vd), proj.dtype)
+        K.gated_norm(o, proj[:, 2 * qk + vd:], 1.0, None, self.unit_w, self.norm_eps, self.heads, True, y, gate="silu")
+        streaming.linear(y, self.w_out, out, ctx)
+
+
+register_mixer("retention", Retention)
 register_mixer("gated_delta", GatedDeltaMixer)
 register_mixer("decay_linear_attention", DecayLinearAttention)

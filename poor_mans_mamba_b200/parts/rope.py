@@ -8,7 +8,7 @@ The whole head is rotated; there is no scaling of positions.
 from __future__ import annotations
 
 import math
-from typing import Optional, Sequence
+from typing import Optional, Sequence, Tuple
 
 import torch
 
@@ -31,6 +31,23 @@ def rotary_frequencies(dims: int, base: float, factor: float = 1.0,
         s = (n - low) / (high - low) if high != low else torch.zeros_like(n)
         f = torch.where(n > high, f, torch.where(n < low, f / by, (1.0 - s) * f / by + s * f))
     return f.to(torch.float32)
+
+
+def yarn_frequencies(dims: int, base: float, factor: float, original: float, fast: float,
+                     slow: float) -> Tuple[Tensor, float]:
+    """(frequencies, factor on the sines and cosines) of YaRN scaling.  Pair i turns original * f_i / (2 pi) times within
+    ``original`` positions; t(n) = dims * ln(original / (2 pi n)) / (2 ln base) is the (fractional) pair that turns n
+    times.  Pairs up to lo = max(floor t(fast), 0) keep their frequency, those from hi = min(ceil t(slow), dims - 1) on
+    are divided by the factor, between them the two are blended linearly in i; the sines and cosines are multiplied by
+    0.1 ln(factor) + 1.  Made in float64 and rounded to float32 once."""
+    def pair_turning(n: float) -> float:
+        return dims * math.log(original / (2.0 * math.pi * n)) / (2.0 * math.log(base))
+
+    i = torch.arange(dims // 2, dtype=torch.float64)
+    f = torch.pow(torch.tensor(float(base), dtype=torch.float64), -2.0 * i / float(max(dims, 1)))
+    lo, hi = max(math.floor(pair_turning(fast)), 0), min(math.ceil(pair_turning(slow)), dims - 1)
+    r = torch.clamp((i - lo) / max(hi - lo, 0.001), 0.0, 1.0)
+    return (f / factor * r + f * (1.0 - r)).to(torch.float32), 0.1 * math.log(factor) + 1.0
 
 
 class RotaryEncoding(PositionEncoding):

@@ -17,6 +17,8 @@ is handed normed rows):
 
     linear(x, w, out, ctx)                              out = x @ w^T
     swiglu(x, gate_up, gate_mult, out, ctx)             out = silu(g * gate_mult) * u,  [g | u] = x @ gate_up^T
+    gelu_linear(x, w, out, ctx)                         out = gelu(x @ w^T), the exact (erf) form
+    linears(xs, ws, outs, ctx)                          out_i = x_i @ w_i^T, several products in one launch
 
 h is the float32 residual stream [T, D]; x, w and out are bfloat16.
 """
@@ -123,4 +125,25 @@ def swiglu(x: Tensor, gate_up: Tensor, gate_mult: float, out: Tensor, ctx) -> bo
         K.skinny_tc_swiglu(x, gate_up, gate_mult, out)
     else:
         K.skinny_swiglu(x, gate_up, gate_mult, out)
+    return True
+
+
+def gelu_linear(x: Tensor, w: Tensor, out: Tensor, ctx) -> bool:
+    """out = gelu(x @ w^T) in one weight-streaming launch; False (nothing done) where the step or the operands do not
+    allow it."""
+    if not _streams(x, w, out, ctx):
+        return False
+    if _tensor_core(x.shape[0]) and K.skinny_tc_supported("store", x, w, out):
+        K.skinny_tc_linear(x, w, out, gelu=True)
+    else:
+        K.skinny_linear(x, w, out, gelu=True)
+    return True
+
+
+def linears(xs: Sequence[Tensor], ws: Sequence[Tensor], outs: Sequence[Tensor], ctx) -> bool:
+    """out_i = x_i @ w_i^T, each with its own activations, in one weight-streaming launch (all with the same number of
+    columns); False (nothing done) where the step or the operands do not allow it."""
+    if len(xs) > K.SKINNY_MAX_PRODUCTS or not all(_streams(x, w, o, ctx) for x, w, o in zip(xs, ws, outs)):
+        return False
+    K.skinny_linears(xs, ws, outs)
     return True
