@@ -24,7 +24,8 @@ L2 flush is needed between timed iterations.
 `--design tafesun`, a Tafesun model) and a Falcon-H1 model of equal width, feed-forward size, layer count and
 vocabulary, one prompt step and decode steps of each with the L2 flushed before every timed step, and every
 kernel's device time.  `--design sorovik` measures a Sorovik model beside the Tafesun and the Gikovik models,
-`--design piladra` a Piladra model beside the Sorovik and the Falcon-H1 models.
+`--design piladra` a Piladra model beside the Sorovik and the Falcon-H1 models, `--design nikodra` a Nikodra model
+beside the Boketar and the Falcon-H1 models.
 `--design gikovik` measures a Gikovik model beside the Tafesun model (the closest one:
 paged softmax attention and routed experts) in the same way.
 """
@@ -603,6 +604,28 @@ def piladra_config(falcon, mixer_sizes, ff_sizes, layers, dense_ff):
             "loop": {"start": 0, "stop": layers, "times": 1}, "layers": out}
 
 
+# `--workload compare --design nikodra`: a Nikodra model beside the Boketar model and the Falcon-H1 model above (equal
+# width, layers and vocabulary; as many feed-forward weights).  Of every four layers the first and the last are
+# attention layers with Falcon-H1's head counts and head size (scaled rotation, mixed values), the second is a parallel
+# layer with the Boketar layer's sizes (chunks in its window's place, retention beside it), the third a time-mixing layer
+# with heads of 64 over the whole width.  The plain feed-forwards are one and a half times as wide as the gated ones.
+def nikodra_config(falcon, sizes, layers, dense_ff):
+    hd, width = falcon["head_dim"], falcon["hidden_size"]
+    att = {"heads": falcon["num_attention_heads"], "kv_heads": falcon["num_key_value_heads"], "dim": hd, "vdim": hd,
+           "scale": hd ** -0.5, "v_mix": True,
+           "rot": {"dims": hd, "base": 5e5, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    l, r = dict(sizes["left"]), sizes["right"]
+    l.pop("conv")
+    left = dict(l, mask={"size": l.pop("window")}, scale=l["dim"] ** -0.5)
+    right = dict(r, decay=[1.0 - 2.0 ** -(4 + 6 * h / max(1, r["heads"] - 1)) for h in range(r["heads"])],
+                 rot={"dims": r["dim"], "base": 1e6})
+    mix = {"heads": width // 64, "dim": 64, "decay_rank": 64 if width < 2048 else 128}
+    kinds = [("attention", att), ("parallel", {"left": left, "right": right}), ("wkv", mix), ("attention", att)]
+    out = [dict(zip(("type", "mixer"), kinds[i % 4]), mlp={"kind": "dense", "ff": dense_ff * 3 // 2}) for i in range(layers)]
+    return {"architecture": "Nikodra", "vocab": falcon["vocab_size"], "width": width, "norm": {"eps": 1e-6},
+            "embedding": {"bigram": {"buckets": 50021, "mul_prev": 8191, "mul_cur": 131}}, "residual_mult": 0.5, "layers": out}
+
+
 def compare_workload(args, peaks) -> int:
     import torch
 
@@ -617,7 +640,11 @@ def compare_workload(args, peaks) -> int:
     falcon.update(falcon_keys)
     falcon["num_hidden_layers"] = layers
     vocab = falcon["vocab_size"]
-    if args.design == "piladra":
+    if args.design == "nikodra":
+        configs = {"nikodra": nikodra_config(falcon, bk_sizes, layers, ff), "boketar": boketar_config(width, ff, vocab, bk_sizes, layers),
+                   "falcon_h1": falcon}
+        design_sizes = {"boketar_sizes": bk_sizes, "nikodra_layers": [l["mixer"] for l in configs["nikodra"]["layers"][:4]]}
+    elif args.design == "piladra":
         sizes = (falcon, GIKOVIK_MIXER[args.sizes], TAFESUN_FF[args.sizes], layers, ff)
         configs = {"piladra": piladra_config(*sizes), "sorovik": sorovik_config(*sizes), "falcon_h1": falcon}
         design_sizes = {"routed_ff": dict(zip(("experts", "top", "expert_ff", "shared_ff"), TAFESUN_FF[args.sizes])),
@@ -660,7 +687,7 @@ def compare_workload(args, peaks) -> int:
         """name -> device microseconds of every kernel of this repository and every library product that
         `fn` issues (launch by launch, an event pair around each)."""
         marks = []
-        call, mm = K._call, K._mm
+        call, mm, bmm = K._call, K._mm, K._bmm
 
         def wrap(inner, label):
             def go(*a, **k):
@@ -672,11 +699,12 @@ def compare_workload(args, peaks) -> int:
                 return r
             return go
         K._call, K._mm = wrap(call, lambda a: a[0]), wrap(mm, lambda a: "library product")
+        K._bmm = wrap(bmm, lambda a: "library product (batched)")
         try:
             fn()
             torch.cuda.synchronize()
         finally:
-            K._call, K._mm = call, mm
+            K._call, K._mm, K._bmm = call, mm, bmm
         out = {}
         for name, e0, e1 in marks:
             out[name] = out.get(name, 0.0) + e0.elapsed_time(e1) * 1e3
@@ -758,9 +786,10 @@ def main() -> int:
                          "count (--layers, default 4) and vocabulary at --sizes 0.5b or 7b: one prompt step of "
                          "--prompt-tokens and decode steps of --batch requests at --context, device-timed with the "
                          "L2 flushed, and the device time of every kernel of one step of each")
-    ap.add_argument("--design", default="boketar", choices=["boketar", "tafesun", "gikovik", "sorovik", "piladra"],
+    ap.add_argument("--design", default="boketar", choices=["boketar", "tafesun", "gikovik", "sorovik", "piladra", "nikodra"],
                     help="--workload compare: the model that is measured beside Falcon-H1 (gikovik: beside Tafesun; "
-                         "sorovik: beside Tafesun and Gikovik; piladra: beside Sorovik and Falcon-H1)")
+                         "sorovik: beside Tafesun and Gikovik; piladra: beside Sorovik and Falcon-H1; "
+                         "nikodra: beside Boketar and Falcon-H1)")
     ap.add_argument("--no-check", dest="check", action="store_false",
                     help="skip the comparison with the plain implementation that runs before the timing: the first "
                          "two layers of the run's model, in the run's dtype, on the benchmark's schedule (a "

@@ -17,7 +17,7 @@
 //
 // Time mixing (kRuleWkv) is the decayed sum with a decay per channel and a read-out before the token's own write:
 //   o_i = (q_i * exp L_(i-1))^T S_0 + sum_{j<i} B_ij v_j + B_ii v_i,  B_ij = sum_c q_i[c] k_j[c] exp(L_(i-1)[c] - L_j[c]),
-//   B_ii = sum_c q_i[c] b[c] k_i[c] with the bonus b;  only `chunk_prepare` knows the difference.  Retention
+//   B_ii = sum_c q_i[c] b[c] k_i[c] with the bonus b;  `wkv_prepare` makes these operands, what follows is the decayed sum's.  Retention
 // (kRuleRetention) is the decayed sum whose q and k are rotated there.
 //
 // Only differences L_i - L_j with i >= j are ever exponentiated, so nothing overflows however strong
@@ -83,13 +83,12 @@ template <typename S, int RULE>
 __global__ void __launch_bounds__(kPrepThreads)
     chunk_prepare_kernel(ChunkArgs p) {
   extern __shared__ float sm[];
-  constexpr bool DELTA = RULE == kRuleDelta, WKV = RULE == kRuleWkv, SILU = RULE == kRuleDecay;
-  constexpr bool CHANNEL = DELTA || WKV;  // a decay per key channel
+  constexpr bool DELTA = RULE == kRuleDelta, SILU = RULE == kRuleDecay;
   const int d = p.d, dv = p.dv, ds = d + 1;  // rows of stride d + 1: row i, column c sits in bank (i + c) mod 32
   float* sK = sm;                         // [C][ds]
   float* sQ = sK + kChunk * ds;           // [C][ds]   (later: the right-hand sides of the solve)
-  float* sL = sQ + kChunk * ds;           // delta, wkv: [C][ds]
-  float* sA = sL + (CHANNEL ? kChunk * ds : 0);  // delta: [C][C + 1]
+  float* sL = sQ + kChunk * ds;           // delta: [C][ds]
+  float* sA = sL + (DELTA ? kChunk * ds : 0);  // delta: [C][C + 1]
   __shared__ float s_beta[kChunk];
   pdl_launch_dependents();
   pdl_wait();
@@ -120,11 +119,6 @@ __global__ void __launch_bounds__(kPrepThreads)
       sK[i * ds + c] = kv;
       const float av = ldf(static_cast<const S*>(p.a) + t * p.ld_a + h * d + c) + p.dt_bias[h * d + c];
       sL[i * ds + c] = a_neg * softplus_f(av);
-    } else if (WKV) {
-      sQ[i * ds + c] = qv;
-      sK[i * ds + c] = kv;
-      // (the bound keeps the running sums finite; exp(-exp(80)) is zero by far)
-      sL[i * ds + c] = -expf(fminf(static_cast<const float*>(p.a)[t * p.ld_a + h * d + c] + p.dt_bias[h * d + c], 80.f));
     } else {
       sQ[i * ds + c] = SILU ? silu_f(qv) : qv;
       sK[i * ds + c] = SILU ? silu_f(kv) : kv * p.k_scale;
@@ -136,7 +130,7 @@ __global__ void __launch_bounds__(kPrepThreads)
     rotate_rows(sQ, sK, ds, n, t0, p.rot, tid, kPrepThreads);
     __syncthreads();
   }
-  const float log_a = CHANNEL ? 0.f : logf(fmaxf(p.decay[h], 1e-38f));
+  const float log_a = DELTA ? 0.f : logf(fmaxf(p.decay[h], 1e-38f));
   if (DELTA) {
     for (int i = warp; i < n; i += kPrepThreads / 32) {  // unit length per token
       float sq = 0.f, sk = 0.f;
@@ -152,8 +146,6 @@ __global__ void __launch_bounds__(kPrepThreads)
         sK[i * ds + c] *= fk;
       }
     }
-  }
-  if (CHANNEL) {
     for (int c = tid; c < d; c += kPrepThreads) {  // running sums of the logarithms
       float run = 0.f;
       for (int i = 0; i < n; ++i) {
@@ -165,28 +157,26 @@ __global__ void __launch_bounds__(kPrepThreads)
   }
 
   // ---- A (delta) and B
-  // wkv: the decays up to the token before i weaken what i reads: row i - 1 of the running sums (i > j >= 0)
-  const float* sLx = WKV ? sL - ds : sL;
-  if (CHANNEL && p.sub_blocks) {
+  if (DELTA && p.sub_blocks) {
     // Pairs inside one sub-block of 16 tokens: the exponential per channel.  A warp takes two rows,
     // 16 lanes each, a lane one column of the row's sub-block.
     for (int i2 = 2 * warp; i2 < n; i2 += 2 * (kPrepThreads / 32)) {
       const int i = i2 + (lane >> 4), j = (i & ~15) + (lane & 15);
       if (i < n && j <= i) {
-        const float *qi = sQ + i * ds, *ki = sK + i * ds, *li = sLx + i * ds, *kj = sK + j * ds, *lj = sL + j * ds;
+        const float *qi = sQ + i * ds, *ki = sK + i * ds, *li = sL + i * ds, *kj = sK + j * ds, *lj = sL + j * ds;
         float accA = 0.f, accB = 0.f;
         for (int c = 0; c < d; ++c) {
-          const float w = (WKV && i == j ? p.bonus[h * d + c] : expf(li[c] - lj[c])) * kj[c];
-          if (DELTA) accA += ki[c] * w;
+          const float w = expf(li[c] - lj[c]) * kj[c];
+          accA += ki[c] * w;
           accB += qi[c] * w;
         }
-        if (DELTA) sA[i * (kChunk + 1) + j] = accA;
+        sA[i * (kChunk + 1) + j] = accA;
         oB[i * kChunk + j] = accB;
       }
     }
     // Pairs across sub-blocks: with r the last row before i's sub-block, exp(L_i - L_j) = exp(L_i - L_r) exp(L_r - L_j),
     // both factors at most one, so the rows are scaled once per sub-block and the pairs are plain dot products.
-    float* sKd = sA + (DELTA ? kChunk * (kChunk + 1) : 0);   // [48][ds]  k_j exp(L_r - L_j), j before the sub-block
+    float* sKd = sA + kChunk * (kChunk + 1);   // [48][ds]  k_j exp(L_r - L_j), j before the sub-block
     float* sKp = sKd + 48 * ds;                // [16][ds]  k_i exp(L_i - L_r), i in the sub-block
     float* sQp = sKp + 16 * ds;                // [16][ds]  q_i exp(L_i - L_r)
     for (int blk = 1; 16 * blk < n; ++blk) {
@@ -198,8 +188,8 @@ __global__ void __launch_bounds__(kPrepThreads)
       }
       for (int e = tid; e < rows * d; e += kPrepThreads) {
         const int ii = e / d, c = e - ii * d, i = 16 * blk + ii;
-        const float pw = expf(sLx[i * ds + c] - sL[r * ds + c]);
-        if (DELTA) sKp[ii * ds + c] = sK[i * ds + c] * pw;
+        const float pw = expf(sL[i * ds + c] - sL[r * ds + c]);
+        sKp[ii * ds + c] = sK[i * ds + c] * pw;
         sQp[ii * ds + c] = sQ[i * ds + c] * pw;
       }
       __syncthreads();
@@ -213,10 +203,10 @@ __global__ void __launch_bounds__(kPrepThreads)
             const float* kd = sKd + j * ds;
             float accA = 0.f, accB = 0.f;
             for (int c = 0; c < d; ++c) {
-              if (DELTA) accA += kp[c] * kd[c];
+              accA += kp[c] * kd[c];
               accB += qp[c] * kd[c];
             }
-            if (DELTA) sA[i * (kChunk + 1) + j] = accA;
+            sA[i * (kChunk + 1) + j] = accA;
             oB[i * kChunk + j] = accB;
           }
         }
@@ -227,21 +217,21 @@ __global__ void __launch_bounds__(kPrepThreads)
   for (int i = warp; i < n; i += kPrepThreads / 32) {
     const float* qi = sQ + i * ds;
     const float* ki = sK + i * ds;
-    const float* li = sLx + i * ds;
+    const float* li = sL + i * ds;
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
       const int j = lane + 32 * half;
       if (j > i) continue;
       const float* kj = sK + j * ds;
       float accA = 0.f, accB = 0.f;
-      if (CHANNEL) {
+      if (DELTA) {
         const float* lj = sL + j * ds;
         for (int c = 0; c < d; ++c) {
-          const float w = (WKV && i == j ? p.bonus[h * d + c] : expf(li[c] - lj[c])) * kj[c];
-          if (DELTA) accA += ki[c] * w;
+          const float w = expf(li[c] - lj[c]) * kj[c];
+          accA += ki[c] * w;
           accB += qi[c] * w;
         }
-        if (DELTA) sA[i * (kChunk + 1) + j] = accA;
+        sA[i * (kChunk + 1) + j] = accA;
       } else {
         for (int c = 0; c < d; ++c) accB += qi[c] * kj[c];
         accB *= expf(log_a * static_cast<float>(i - j));
@@ -253,12 +243,12 @@ __global__ void __launch_bounds__(kPrepThreads)
   // ---- q * exp L, k * exp(L_end - L), exp L_end
   for (int e = tid; e < n * d; e += kPrepThreads) {
     const int i = e / d, c = e - i * d;
-    const float up = CHANNEL ? sL[i * ds + c] : log_a * static_cast<float>(i + 1);
-    const float end = CHANNEL ? sL[(n - 1) * ds + c] : log_a * static_cast<float>(n);
-    oQg[i * d + c] = sQ[i * ds + c] * (WKV ? (i > 0 ? expf(sLx[i * ds + c]) : 1.f) : expf(up));
+    const float up = DELTA ? sL[i * ds + c] : log_a * static_cast<float>(i + 1);
+    const float end = DELTA ? sL[(n - 1) * ds + c] : log_a * static_cast<float>(n);
+    oQg[i * d + c] = sQ[i * ds + c] * expf(up);
     oKe[i * d + c] = sK[i * ds + c] * expf(end - up);
   }
-  for (int c = tid; c < d; c += kPrepThreads) oEg[c] = expf(CHANNEL ? sL[(n - 1) * ds + c] : log_a * static_cast<float>(n));
+  for (int c = tid; c < d; c += kPrepThreads) oEg[c] = expf(DELTA ? sL[(n - 1) * ds + c] : log_a * static_cast<float>(n));
   if (!DELTA) {
     for (int e = tid; e < n * dv; e += kPrepThreads) {
       const int i = e / dv, c = e - i * dv;
@@ -307,6 +297,136 @@ __global__ void __launch_bounds__(kPrepThreads)
       }
     }
     __syncthreads();  // the next pass loads further columns of V over these
+  }
+}
+
+// ----------------------------------------------------------------------------------------------
+// The same operands for time mixing.  Sums of logarithms are kept within sub-blocks of 16 tokens only (sL: up to and
+// including the token; sT: a sub-block's total), so that strong decays do not drown the weak ones behind them, and a
+// token's logarithm is bounded at -40 (4e-18: below the rounding of anything it could stand beside).  Rows of stride
+// d + 4: sixteen-byte reads of neighbouring rows fall into different banks.
+//   pairs within a sub-block:  B_ij = sum_c q_i[c] k_j[c] exp(L_(i-1) - L_j),  B_ii with the bonus;
+//   then in place  q_i <- q_i exp(L_(i-1) of its sub-block),  k_j <- k_j exp(T - L_j)  (weakened to its sub-block's end);
+//   sub-block by sub-block, all rows of k before it are weakened to its start: pairs across are dot products.
+// What is left of q and k at the end is, up to whole sub-blocks' totals, Q * exp L and K * exp(L_end - L).
+constexpr float kLogDecayFloor = -40.f;
+
+inline size_t wkv_prepare_smem(int d) { return sizeof(float) * (static_cast<size_t>(3 * kChunk) * (d + 4) + 4 * static_cast<size_t>(d)); }
+
+template <typename S>
+__global__ void __launch_bounds__(kPrepThreads)
+    wkv_prepare_kernel(ChunkArgs p) {
+  extern __shared__ __align__(16) float sm[];
+  const int d = p.d, dv = p.dv, ds = d + 4;
+  float* sK = sm;                  // [C][ds]
+  float* sQ = sK + kChunk * ds;    // [C][ds]
+  float* sL = sQ + kChunk * ds;    // [C][ds]
+  float* sT = sL + kChunk * ds;    // [4][d]
+  pdl_launch_dependents();
+  pdl_wait();
+  const int chunk = blockIdx.x, h = blockIdx.y;
+  int seq, t0, n;
+  if (!locate_chunk(p.cu, p.n_seq, chunk, &seq, &t0, &n)) return;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const size_t ch = static_cast<size_t>(chunk) * p.H + h;
+  float* oB = p.B + ch * kChunk * kChunk;
+  float* oQg = p.Qg + ch * kChunk * d;
+  float* oKe = p.Ke + ch * kChunk * d;
+  float* oUv = p.Uv + ch * kChunk * dv;
+  const int nb = (n + 15) >> 4;
+
+  for (int e = tid; e < n * d; e += kPrepThreads) {
+    const int i = e / d, c = e - i * d;
+    const long long t = t0 + i;
+    sQ[i * ds + c] = ldf(static_cast<const S*>(p.q) + t * p.ld_q + h * d + c);
+    sK[i * ds + c] = ldf(static_cast<const S*>(p.k) + t * p.ld_k + h * d + c);
+    sL[i * ds + c] = fmaxf(-expf(static_cast<const float*>(p.a)[t * p.ld_a + h * d + c] + p.dt_bias[h * d + c]), kLogDecayFloor);
+  }
+  for (int e = tid; e < n * dv; e += kPrepThreads) {
+    const int i = e / dv, c = e - i * dv;
+    oUv[e] = ldf(static_cast<const S*>(p.v) + static_cast<long long>(t0 + i) * p.ld_v + h * dv + c);
+  }
+  __syncthreads();
+  for (int e = tid; e < nb * d; e += kPrepThreads) {
+    const int blk = e / d, c = e - blk * d;
+    float run = 0.f;
+    for (int i = 16 * blk; i < min(16 * blk + 16, n); ++i) {
+      run += sL[i * ds + c];
+      sL[i * ds + c] = run;
+    }
+    sT[blk * d + c] = run;
+  }
+  __syncthreads();
+
+  // ---- pairs within a sub-block: a warp takes two rows, 16 lanes each, a lane one column of the row's sub-block
+  for (int i2 = 2 * warp; i2 < n; i2 += 2 * (kPrepThreads / 32)) {
+    const int i = i2 + (lane >> 4), j = (i & ~15) + (lane & 15);
+    if (i < n && j <= i) {
+      const float *qi = sQ + i * ds, *kj = sK + j * ds, *lj = sL + j * ds, *li = sL + (i > 0 ? i - 1 : 0) * ds;  // (i > j: row i - 1 is in the sub-block)
+      const float* u = p.bonus + h * d;
+      float acc = 0.f;
+      for (int c = 0; c < d; c += 4) {
+        const float4 q4 = *reinterpret_cast<const float4*>(qi + c), k4 = *reinterpret_cast<const float4*>(kj + c);
+        if (i == j) {
+          acc += q4.x * u[c] * k4.x + q4.y * u[c + 1] * k4.y + q4.z * u[c + 2] * k4.z + q4.w * u[c + 3] * k4.w;
+        } else {
+          const float4 a4 = *reinterpret_cast<const float4*>(li + c), b4 = *reinterpret_cast<const float4*>(lj + c);
+          acc += q4.x * k4.x * expf(a4.x - b4.x) + q4.y * k4.y * expf(a4.y - b4.y) + q4.z * k4.z * expf(a4.z - b4.z) +
+                 q4.w * k4.w * expf(a4.w - b4.w);
+        }
+      }
+      oB[i * kChunk + j] = acc;
+    }
+  }
+  __syncthreads();
+  for (int e = tid; e < n * d; e += kPrepThreads) {
+    const int i = e / d, c = e - i * d;
+    if (i & 15) sQ[i * ds + c] *= expf(sL[(i - 1) * ds + c]);
+    sK[i * ds + c] *= expf(sT[(i >> 4) * d + c] - sL[i * ds + c]);
+  }
+  // ---- pairs across: four rows of the sub-block and 32 columns a warp
+  for (int blk = 1; blk < nb; ++blk) {
+    __syncthreads();
+    if (blk > 1) {  // rows before the last sub-block reach this one through its total
+      for (int e = tid; e < 16 * (blk - 1) * d; e += kPrepThreads) {
+        const int j = e / d, c = e - j * d;
+        sK[j * ds + c] *= expf(sT[(blk - 1) * d + c]);
+      }
+      __syncthreads();
+    }
+    const int rg = warp & 3, j = (warp >> 2) * 32 + lane;  // warps 8.. have no columns (at most 48 are before a sub-block)
+    const int i0 = 16 * blk + 4 * rg;
+    if (j < 16 * blk && i0 < n) {
+      const float* kj = sK + j * ds;
+      const float* q0 = sQ + i0 * ds;   // (rows at and beyond n hold stale values that are not stored)
+      float acc[4] = {0.f, 0.f, 0.f, 0.f};
+      for (int c = 0; c < d; c += 4) {
+        const float4 k4 = *reinterpret_cast<const float4*>(kj + c);
+#pragma unroll
+        for (int r = 0; r < 4; ++r) {
+          const float4 q4 = *reinterpret_cast<const float4*>(q0 + r * ds + c);
+          acc[r] += q4.x * k4.x + q4.y * k4.y + q4.z * k4.z + q4.w * k4.w;
+        }
+      }
+#pragma unroll
+      for (int r = 0; r < 4; ++r)
+        if (i0 + r < n) oB[(i0 + r) * kChunk + j] = acc[r];
+    }
+  }
+  __syncthreads();
+  // ---- what the other launches read: q weakened from the chunk's start, k to its end, the whole chunk's decay
+  for (int e = tid; e < n * d; e += kPrepThreads) {
+    const int i = e / d, c = e - i * d, blk = i >> 4;
+    float before = 0.f;
+    for (int b = 0; b < blk; ++b) before += sT[b * d + c];
+    oQg[e] = sQ[i * ds + c] * expf(before);
+    oKe[e] = sK[i * ds + c] * (blk < nb - 1 ? expf(sT[(nb - 1) * d + c]) : 1.f);
+  }
+  float* oEg = p.Eg + ch * d;
+  for (int c = tid; c < d; c += kPrepThreads) {
+    float all = 0.f;
+    for (int b = 0; b < nb; ++b) all += sT[b * d + c];
+    oEg[c] = expf(all);
   }
 }
 
@@ -850,8 +970,9 @@ __global__ void __launch_bounds__(kDecayThreads)
 }
 
 inline size_t prepare_smem(int d, int rule, bool sub_blocks = false) {
-  const bool delta = rule == kRuleDelta, channel = delta || rule == kRuleWkv;
-  return sizeof(float) * (static_cast<size_t>(kChunk) * (d + 1) * (channel ? 3 : 2) + (delta ? kChunk * (kChunk + 1) : 0) +
+  if (rule == kRuleWkv) return wkv_prepare_smem(d);
+  const bool delta = rule == kRuleDelta;
+  return sizeof(float) * (static_cast<size_t>(kChunk) * (d + 1) * (delta ? 3 : 2) + (delta ? kChunk * (kChunk + 1) : 0) +
                           (sub_blocks ? static_cast<size_t>(48 + 32) * (d + 1) : 0));
 }
 inline size_t apply_smem(int d, bool delta, int nc = 16) {
@@ -862,9 +983,11 @@ inline size_t apply_smem(int d, bool delta, int nc = 16) {
 template <typename S, int RULE>
 int launch_chunked(ChunkArgs a, int n_chunks, cudaStream_t stream) {
   constexpr bool DELTA = RULE == kRuleDelta;
-  a.sub_blocks = (DELTA || RULE == kRuleWkv) && prepare_smem(a.d, RULE, true) <= 220 * 1024;
+  a.sub_blocks = DELTA && prepare_smem(a.d, RULE, true) <= 220 * 1024;
   const size_t sp = prepare_smem(a.d, RULE, a.sub_blocks != 0);
-  auto prep = chunk_prepare_kernel<S, RULE>;
+  void (*prep)(ChunkArgs) = nullptr;
+  if constexpr (RULE == kRuleWkv) prep = wkv_prepare_kernel<S>;
+  else prep = chunk_prepare_kernel<S, RULE>;
   if (sp > 48 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(prep, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(sp));
     if (e != cudaSuccess) return static_cast<int>(e);

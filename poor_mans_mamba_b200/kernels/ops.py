@@ -379,6 +379,10 @@ def linear(x: Tensor, weight: Tensor, out: Tensor) -> Tensor:
     return out
 
 
+def _bmm(x: Tensor, weight: Tensor, out: Tensor) -> None:
+    torch.bmm(x, weight.transpose(1, 2), out=out)
+
+
 def batched_linear(x: Tensor, weight: Tensor, out: Tensor) -> None:
     """out[b] [T, N] = x[b] [T, K] @ weight[b] [N, K]^T through the GEMM library, one call."""
     _cuda(x, weight, out)
@@ -387,7 +391,7 @@ def batched_linear(x: Tensor, weight: Tensor, out: Tensor) -> None:
     prev = torch.backends.cuda.matmul.allow_tf32
     torch.backends.cuda.matmul.allow_tf32 = False
     try:
-        torch.bmm(x, weight.transpose(1, 2), out=out)
+        _bmm(x, weight, out)
     finally:
         torch.backends.cuda.matmul.allow_tf32 = prev
 

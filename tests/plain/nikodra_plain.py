@@ -95,7 +95,9 @@ def causal_mask(T: int) -> Tensor:
 
 
 def chunk_mask(T: int, size: int) -> Tensor:
-    """i sees j <= i of its own chunk of ``size`` positions."""
+    """i sees j <= i of its own chunk of ``size`` positions (0: every j <= i)."""
+    if size == 0:
+        return causal_mask(T)
     i = torch.arange(T)
     return causal_mask(T) & (i[:, None] // size == i[None, :] // size)
 
@@ -142,7 +144,7 @@ def chunked_attention(x: Tensor, W: Dict[str, Tensor], pre: str, m: dict, eps: f
     q = rms(linear(x, W[pre + "q"]).reshape(T, H, d), eps)
     k = rms(linear(x, W[pre + "k"]).reshape(T, G, d), eps)
     v = linear(x, W[pre + "v"]).reshape(T, G, dv)
-    heads = attend_with_one_more(q, k, v, m["scale"], chunk_mask(T, m["mask"]["size"]))
+    heads = attend_with_one_more(q, k, v, m["scale"], chunk_mask(T, (m.get("mask") or {}).get("size", 0)))
     return linear(heads.reshape(T, H * dv), W[pre + "o"])
 
 
