@@ -204,8 +204,12 @@ PMM_EXPORT int pmm_clamped_glu(const void* gu, long long ld, float limit, float 
 namespace pmm {
 enum { kUnaryGelu = 0, kUnaryTanh = 1 };
 
+// `low`: the result is stored as bfloat16
 template <int OP>
-__device__ __forceinline__ float unary_f(float z) { return OP == kUnaryGelu ? gelu_erf_f(z) : tanhf(z); }
+__device__ __forceinline__ float unary_f(float z, bool low) {
+  if (OP == kUnaryTanh) return tanhf(z);
+  return low ? gelu_erf_fast(z) : gelu_erf_f(z);
+}
 
 // x = f(x) in place on rows of stride ld
 template <typename S, int OP>
@@ -213,7 +217,7 @@ __global__ void unary_kernel(S* __restrict__ x, long long ld, int F) {
   pdl_launch_dependents();
   pdl_wait();
   S* row = x + static_cast<long long>(blockIdx.x) * ld;
-  for (int f = blockIdx.y * blockDim.x + threadIdx.x; f < F; f += gridDim.y * blockDim.x) stf(row + f, unary_f<OP>(ldf(row + f)));
+  for (int f = blockIdx.y * blockDim.x + threadIdx.x; f < F; f += gridDim.y * blockDim.x) stf(row + f, unary_f<OP>(ldf(row + f), sizeof(S) == 2));
 }
 
 // bfloat16, F and ld multiples of 8, 16-byte aligned rows: eight elements per thread
@@ -228,7 +232,7 @@ __global__ void unary_bf16x8_kernel(__nv_bfloat16* __restrict__ x, long long ld,
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const float2 z = __bfloat1622float2(v2[i]);
-      v2[i] = __floats2bfloat162_rn(unary_f<OP>(z.x), unary_f<OP>(z.y));
+      v2[i] = __floats2bfloat162_rn(unary_f<OP>(z.x, true), unary_f<OP>(z.y, true));
     }
     *reinterpret_cast<uint4*>(row + f) = v;
   }

@@ -20,6 +20,26 @@ __device__ __forceinline__ float ldf(const __nv_bfloat16* p) { return __bfloat16
 __device__ __forceinline__ void stf(float* p, float v) { *p = v; }
 __device__ __forceinline__ void stf(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
 
+// Two and four neighbouring elements (the pointer on a boundary of as many).
+__device__ __forceinline__ float2 ldf2(const float* p) { return *reinterpret_cast<const float2*>(p); }
+__device__ __forceinline__ float2 ldf2(const __nv_bfloat16* p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p)); }
+__device__ __forceinline__ void stf2(float* p, float2 v) { *reinterpret_cast<float2*>(p) = v; }
+__device__ __forceinline__ void stf2(__nv_bfloat16* p, float2 v) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(v.x, v.y); }
+__device__ __forceinline__ float4 ldf4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 ldf4(const __nv_bfloat16* p) {
+  const uint2 raw = *reinterpret_cast<const uint2*>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void stf4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void stf4(__nv_bfloat16* p, float4 v) {
+  uint2 raw;
+  *reinterpret_cast<__nv_bfloat162*>(&raw.x) = __floats2bfloat162_rn(v.x, v.y);
+  *reinterpret_cast<__nv_bfloat162*>(&raw.y) = __floats2bfloat162_rn(v.z, v.w);
+  *reinterpret_cast<uint2*>(p) = raw;
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
@@ -44,6 +64,21 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
   return t;
 }
 
+// Two sums over the block at once; `red` is shared memory for 64 floats.
+__device__ __forceinline__ float2 block_sum2(float2 v, float* red) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int nwarp = (blockDim.x + 31) >> 5;
+  v.x = warp_sum(v.x);
+  v.y = warp_sum(v.y);
+  __syncthreads();  // protects `red` against a previous use
+  if (lane == 0) {
+    red[warp] = v.x;
+    red[32 + warp] = v.y;
+  }
+  __syncthreads();
+  return make_float2(warp_sum(lane < nwarp ? red[lane] : 0.f), warp_sum(lane < nwarp ? red[32 + lane] : 0.f));
+}
+
 __device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
 // For results that are stored as bfloat16: relative error about 1e-6, three instructions' worth
 // of special-function work instead of a full-precision exponential and division.
@@ -51,6 +86,15 @@ __device__ __forceinline__ float silu_fast(float x) { return __fdividef(x, 1.f +
 
 // The exact (erf) form of GELU: z/2 (1 + erf(z / sqrt 2)).
 __device__ __forceinline__ float gelu_erf_f(float z) { return 0.5f * z * (1.f + erff(z * 0.70710678118654752f)); }
+// For results that are stored as bfloat16: with x = |z| / sqrt 2 and t = 1 / (1 + 0.3275911 x),
+// erfc(x) = (a1 t + ... + a5 t^5) e^(-x^2) to 1.5e-7 (Abramowitz and Stegun, Handbook of Mathematical Functions, 7.1.26).
+__device__ __forceinline__ float gelu_erf_fast(float z) {
+  const float x = fabsf(z) * 0.70710678118654752f;
+  const float t = __fdividef(1.f, 1.f + 0.3275911f * x);
+  const float poly = t * (0.254829592f + t * (-0.284496736f + t * (1.421413741f + t * (-1.453152027f + t * 1.061405429f))));
+  const float half = 0.5f * z * poly * __expf(-x * x);  // z/2 erfc(x)
+  return z >= 0.f ? z - half : half;
+}
 
 // v if v>20; exp(v) if v<-20; log1p(exp(v)) otherwise.
 __device__ __forceinline__ float softplus_f(float v) {

@@ -27,7 +27,7 @@ struct Bigram {
 template <typename S>
 __global__ void embed_kernel(float* __restrict__ out, const S* __restrict__ table,
                              const int* __restrict__ tokens, float mult, int D, int V,
-                             const float* __restrict__ norm_w, float eps, const Bigram bg) {
+                             const float* __restrict__ norm_w, float eps, const Bigram bg, int vec) {
   __shared__ float red[32];
   __shared__ int s_row;
   pdl_launch_dependents();
@@ -54,6 +54,14 @@ __global__ void embed_kernel(float* __restrict__ out, const S* __restrict__ tabl
     }
     __syncthreads();
     const S* add = static_cast<const S*>(bg.table) + static_cast<size_t>(s_row) * D;
+    if (vec && !norm_w) {
+      const float m = ok ? mult : 0.f;
+      for (int i = threadIdx.x * 4; i < D; i += blockDim.x * 4) {
+        const float4 x = ldf4(row + i), y = ldf4(add + i);
+        stf4(o + i, make_float4(m * x.x + y.x, m * x.y + y.y, m * x.z + y.z, m * x.w + y.w));
+      }
+      return;
+    }
     float ss = 0.f;
     for (int i = threadIdx.x; i < D; i += blockDim.x) {
       const float v = (ok ? mult * ldf(row + i) : 0.f) + ldf(add + i);
@@ -66,6 +74,14 @@ __global__ void embed_kernel(float* __restrict__ out, const S* __restrict__ tabl
     return;
   }
   if (!norm_w) {
+    if (vec) {
+      const float m = ok ? mult : 0.f;
+      for (int i = threadIdx.x * 4; i < D; i += blockDim.x * 4) {
+        const float4 x = ldf4(row + i);
+        stf4(o + i, make_float4(m * x.x, m * x.y, m * x.z, m * x.w));
+      }
+      return;
+    }
     for (int i = threadIdx.x; i < D; i += blockDim.x) o[i] = ok ? mult * ldf(row + i) : 0.f;
     return;
   }
@@ -108,21 +124,6 @@ __global__ void add_rmsnorm_kernel(float* __restrict__ h, const S* __restrict__ 
   for (int i = threadIdx.x; i < D; i += blockDim.x) stf(o + i, buf[i] * inv * w[i]);
 }
 
-__device__ __forceinline__ float4 ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
-__device__ __forceinline__ float4 ld4(const __nv_bfloat16* p) {
-  const uint2 raw = *reinterpret_cast<const uint2*>(p);
-  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
-  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
-  return make_float4(a.x, a.y, b.x, b.y);
-}
-__device__ __forceinline__ void st4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
-__device__ __forceinline__ void st4(__nv_bfloat16* p, float4 v) {
-  uint2 raw;
-  *reinterpret_cast<__nv_bfloat162*>(&raw.x) = __floats2bfloat162_rn(v.x, v.y);
-  *reinterpret_cast<__nv_bfloat162*>(&raw.y) = __floats2bfloat162_rn(v.z, v.w);
-  *reinterpret_cast<uint2*>(p) = raw;
-}
-
 // The same for widths that are a multiple of 4: four elements per thread and access.
 template <typename S>
 __global__ void add_rmsnorm_vec_kernel(float* __restrict__ h, const S* __restrict__ a, float sa,
@@ -137,18 +138,18 @@ __global__ void add_rmsnorm_vec_kernel(float* __restrict__ h, const S* __restric
   const size_t src = static_cast<size_t>(rows ? rows[r] : r) * D;
   float ss = 0.f;
   for (int i = threadIdx.x * 4; i < D; i += blockDim.x * 4) {
-    float4 v = ld4(h + src + i);
+    float4 v = ldf4(h + src + i);
     if (a) {
-      const float4 x = ld4(a + src + i);
+      const float4 x = ldf4(a + src + i);
       v.x += sa * x.x; v.y += sa * x.y; v.z += sa * x.z; v.w += sa * x.w;
     }
     if (b) {
-      const float4 x = ld4(b + src + i);
+      const float4 x = ldf4(b + src + i);
       v.x += sb * x.x; v.y += sb * x.y; v.z += sb * x.z; v.w += sb * x.w;
     }
     *reinterpret_cast<float4*>(buf + i) = v;
     ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
-    if (!rows && (a || b)) st4(h + src + i, v);
+    if (!rows && (a || b)) stf4(h + src + i, v);
   }
   if (!out) return;
   const float total = block_sum(ss, red);
@@ -156,8 +157,8 @@ __global__ void add_rmsnorm_vec_kernel(float* __restrict__ h, const S* __restric
   S* o = out + static_cast<size_t>(r) * D;
   for (int i = threadIdx.x * 4; i < D; i += blockDim.x * 4) {
     const float4 v = *reinterpret_cast<const float4*>(buf + i);
-    const float4 g = ld4(w + i);
-    st4(o + i, make_float4(v.x * inv * g.x, v.y * inv * g.y, v.z * inv * g.z, v.w * inv * g.w));
+    const float4 g = ldf4(w + i);
+    stf4(o + i, make_float4(v.x * inv * g.x, v.y * inv * g.y, v.z * inv * g.z, v.w * inv * g.w));
   }
 }
 
@@ -226,14 +227,14 @@ __global__ void add_postnorm_rmsnorm_vec_kernel(float* __restrict__ h, const S* 
   const size_t src = static_cast<size_t>(rows ? rows[r] : r) * D;
   const int step = blockDim.x * 4;
   auto branches = [&](int i) {
-    float4 s = ld4(a + src + i);
+    float4 s = ldf4(a + src + i);
     s.x *= sa; s.y *= sa; s.z *= sa; s.w *= sa;
     if (b) {
-      const float4 x = ld4(b + src + i);
+      const float4 x = ldf4(b + src + i);
       s.x += sb * x.x; s.y += sb * x.y; s.z += sb * x.z; s.w += sb * x.w;
     }
     if (bias) {
-      const float4 x = ld4(bias + i);
+      const float4 x = ldf4(bias + i);
       s.x += x.x; s.y += x.y; s.z += x.z; s.w += x.w;
     }
     return s;
@@ -247,7 +248,7 @@ __global__ void add_postnorm_rmsnorm_vec_kernel(float* __restrict__ h, const S* 
     const int i = threadIdx.x * 4 + c * step;
     v[c] = i < D ? branches(i) : zero;
     // (the stream's row is asked for before the reduction, so that its latency hides behind it)
-    hv[c] = (h && i < D) ? ld4(h + src + i) : zero;
+    hv[c] = (h && i < D) ? ldf4(h + src + i) : zero;
     ss += sq(v[c]);
   }
   if (P == 4) {
@@ -260,9 +261,9 @@ __global__ void add_postnorm_rmsnorm_vec_kernel(float* __restrict__ h, const S* 
   const float inv_p = 1.0f / sqrtf(block_sum(ss, red) / static_cast<float>(D) + post_eps);
   float sv = 0.f;
   auto join = [&](int i, float4 s, float4 x) {
-    const float4 g = ld4(post_w + i);
+    const float4 g = ldf4(post_w + i);
     float4 y = make_float4(s.x * inv_p * g.x + x.x, s.y * inv_p * g.y + x.y, s.z * inv_p * g.z + x.z, s.w * inv_p * g.w + x.w);
-    if (h && !rows) st4(h + src + i, y);
+    if (h && !rows) stf4(h + src + i, y);
     sv += sq(y);
     return y;
   };
@@ -273,7 +274,7 @@ __global__ void add_postnorm_rmsnorm_vec_kernel(float* __restrict__ h, const S* 
   }
   if (P == 4) {
     for (int i = threadIdx.x * 4 + 4 * step; i < D; i += step)
-      *reinterpret_cast<float4*>(buf + i) = join(i, *reinterpret_cast<const float4*>(buf + i), h ? ld4(h + src + i) : zero);
+      *reinterpret_cast<float4*>(buf + i) = join(i, *reinterpret_cast<const float4*>(buf + i), h ? ldf4(h + src + i) : zero);
   }
   if (!out) return;
   S* o = out + static_cast<size_t>(r) * D;
@@ -281,10 +282,10 @@ __global__ void add_postnorm_rmsnorm_vec_kernel(float* __restrict__ h, const S* 
   if (w) inv = 1.0f / sqrtf(block_sum(sv, red) / static_cast<float>(D) + eps);
   auto write = [&](int i, float4 y) {
     if (w) {
-      const float4 g = ld4(w + i);
+      const float4 g = ldf4(w + i);
       y = make_float4(y.x * inv * g.x, y.y * inv * g.y, y.z * inv * g.z, y.w * inv * g.w);
     }
-    st4(o + i, y);
+    stf4(o + i, y);
   };
 #pragma unroll
   for (int c = 0; c < P; ++c) {
@@ -330,10 +331,12 @@ PMM_EXPORT int pmm_embed(void* out, const void* table, const int* tokens, float 
                          const int* slots, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (bigram && (buckets <= 0 || mul_prev < 0 || mul_cur < 0 || !previous || !seq_of || !cu || !slots)) return PMM_ERR_BAD_ARGUMENT;
+  const int vec = D % 4 == 0 && reinterpret_cast<uintptr_t>(out) % 16 == 0 && reinterpret_cast<uintptr_t>(table) % 16 == 0 &&
+                  reinterpret_cast<uintptr_t>(bigram) % 16 == 0;
   const pmm::Bigram bg{bigram, mul_prev, mul_cur, buckets, previous, seq_of, cu, slots};
   PMM_DISPATCH_DTYPE(dtype, S, pmm::launch_pdl(pmm::embed_kernel<S>, dim3(T), dim3(256), 0, stream,
                                                static_cast<float*>(out), static_cast<const S*>(table), tokens,
-                                               mult, D, V, norm_w, eps, bg));
+                                               mult, D, V, norm_w, eps, bg, vec));
   return pmm::launch_status();
 }
 

@@ -150,6 +150,66 @@ __global__ void __launch_bounds__(256)
   }
 }
 
+// The same for one or two branches of a width that is a multiple of 4, up to 1,024 * P: the rows stay in registers from
+// their one read to the sum, and both root mean squares come from one reduction.
+template <typename S, typename O, int P>
+__global__ void __launch_bounds__(256)
+    normed_sum_vec_kernel(Branches b, int n, float eps, float scale, O* __restrict__ out, int D) {
+  __shared__ float red[64];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x;
+  float4 v[2][P];
+  float ss[2] = {0.f, 0.f};
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+#pragma unroll
+    for (int c = 0; c < P; ++c) {
+      const int d = (threadIdx.x + 256 * c) * 4;
+      float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (i < n && d < D) {
+        x = ldf4(static_cast<const S*>(b.x[i]) + static_cast<long long>(t) * b.ld[i] + d);
+        if (b.bias[i]) {
+          const float4 y = ldf4(b.bias[i] + d);
+          x = make_float4(x.x + y.x, x.y + y.y, x.z + y.z, x.w + y.w);
+        }
+      }
+      v[i][c] = x;
+      ss[i] += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+    }
+  }
+  const float2 tot = block_sum2(make_float2(ss[0], ss[1]), red);
+  const float inv[2] = {scale / sqrtf(tot.x / static_cast<float>(D) + eps), scale / sqrtf(tot.y / static_cast<float>(D) + eps)};
+#pragma unroll
+  for (int c = 0; c < P; ++c) {
+    const int d = (threadIdx.x + 256 * c) * 4;
+    if (d >= D) continue;
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      if (i < n) {
+        const float4 w = ldf4(b.w[i] + d);
+        a.x += v[i][c].x * inv[i] * w.x;
+        a.y += v[i][c].y * inv[i] * w.y;
+        a.z += v[i][c].z * inv[i] * w.z;
+        a.w += v[i][c].w * inv[i] * w.w;
+      }
+    }
+    stf4(out + static_cast<size_t>(t) * D + d, a);
+  }
+}
+
+template <typename S, typename O>
+void launch_normed_sum(const Branches& b, int n, float eps, float scale, O* out, int T, int D, cudaStream_t stream) {
+  auto aligned = [](const void* p, size_t bytes) { return reinterpret_cast<uintptr_t>(p) % bytes == 0; };
+  bool vec = n <= 2 && D % 4 == 0 && D <= 4096 && aligned(out, 4 * sizeof(O));
+  for (int i = 0; i < n && vec; ++i)
+    vec = aligned(b.x[i], 4 * sizeof(S)) && b.ld[i] % 4 == 0 && aligned(b.w[i], 16) && aligned(b.bias[i], 16);
+  auto kern = !vec ? normed_sum_kernel<S, O>
+            : D <= 1024 ? normed_sum_vec_kernel<S, O, 1> : D <= 2048 ? normed_sum_vec_kernel<S, O, 2> : normed_sum_vec_kernel<S, O, 4>;
+  launch_pdl(kern, dim3(T), dim3(256), 0, stream, b, n, eps, scale, out, D);
+}
+
 }  // namespace pmm
 
 // x_in: lane s at x_in + s*in_lane_stride (stride 0: every lane reads the same [T, D]); x_out likewise
@@ -199,12 +259,8 @@ PMM_EXPORT int pmm_normed_sum(const void* const* x, const long long* ld, const f
     b.bias[i] = bias ? bias[i] : nullptr;
   }
   PMM_DISPATCH_DTYPE(dtype, S, {
-    if (out_f32)
-      pmm::launch_pdl(pmm::normed_sum_kernel<S, float>, dim3(T), dim3(256), 0, stream, b, n, eps, scale,
-                      static_cast<float*>(out), D);
-    else
-      pmm::launch_pdl(pmm::normed_sum_kernel<S, S>, dim3(T), dim3(256), 0, stream, b, n, eps, scale,
-                      static_cast<S*>(out), D);
+    if (out_f32) pmm::launch_normed_sum<S, float>(b, n, eps, scale, static_cast<float*>(out), T, D, stream);
+    else pmm::launch_normed_sum<S, S>(b, n, eps, scale, static_cast<S*>(out), T, D, stream);
   });
   return pmm::launch_status();
 }

@@ -18,7 +18,8 @@
 // Time mixing (kRuleWkv) is the decayed sum with a decay per channel and a read-out before the token's own write:
 //   o_i = (q_i * exp L_(i-1))^T S_0 + sum_{j<i} B_ij v_j + B_ii v_i,  B_ij = sum_c q_i[c] k_j[c] exp(L_(i-1)[c] - L_j[c]),
 //   B_ii = sum_c q_i[c] b[c] k_i[c] with the bonus b;  `wkv_prepare` makes these operands, what follows is the decayed sum's.  Retention
-// (kRuleRetention) is the decayed sum whose q and k are rotated there.
+// (kRuleRetention) is the decayed sum whose q and k are rotated as they are read.  The decayed sums' operands are made by
+// `decay_prepare`.
 //
 // Only differences L_i - L_j with i >= j are ever exponentiated, so nothing overflows however strong
 // the decay.  `chunk_prepare` makes W, Uv, B, Q * exp L, K * exp(L_end - L) and exp L_end for every
@@ -56,6 +57,7 @@ struct ChunkArgs {
   float unit_eps, q_scale;
   // per (chunk, head), chunk-major: W [C, d] (delta), Uv [C, dv], B [C, C], Qg [C, d], Ke [C, d], Eg [d]
   float *W, *Uv, *B, *Qg, *Ke, *Eg;
+  int vec_in;                           // q, k, v (and a) rows and heads start on boundaries of four elements
   int sub_blocks;                       // chunk_prepare scales rows once per sub-block of 16 tokens (its shared memory allows it)
   float *N, *M;                         // [d, dv] and (delta) [d, d] per (chunk, head): see the kernels that use them
   float* state; const int* slots; float* out;
@@ -79,16 +81,15 @@ __device__ __forceinline__ bool locate_chunk(const int* __restrict__ cu, int n_s
   return false;
 }
 
-template <typename S, int RULE>
+template <typename S>
 __global__ void __launch_bounds__(kPrepThreads)
     chunk_prepare_kernel(ChunkArgs p) {
   extern __shared__ float sm[];
-  constexpr bool DELTA = RULE == kRuleDelta, SILU = RULE == kRuleDecay;
   const int d = p.d, dv = p.dv, ds = d + 1;  // rows of stride d + 1: row i, column c sits in bank (i + c) mod 32
   float* sK = sm;                         // [C][ds]
   float* sQ = sK + kChunk * ds;           // [C][ds]   (later: the right-hand sides of the solve)
-  float* sL = sQ + kChunk * ds;           // delta: [C][ds]
-  float* sA = sL + (DELTA ? kChunk * ds : 0);  // delta: [C][C + 1]
+  float* sL = sQ + kChunk * ds;           // [C][ds]
+  float* sA = sL + kChunk * ds;           // [C][C + 1]
   __shared__ float s_beta[kChunk];
   pdl_launch_dependents();
   pdl_wait();
@@ -109,55 +110,43 @@ __global__ void __launch_bounds__(kPrepThreads)
   float* oEg = p.Eg + ch * d;
 
   // ---- q, k (and the logarithms of the decays) of the chunk's tokens
-  const float a_neg = DELTA ? -expf(p.a_log[h]) : 0.f;
+  const float a_neg = -expf(p.a_log[h]);
   for (int e = tid; e < n * d; e += kPrepThreads) {
     const int i = e / d, c = e - i * d;
     const long long t = t0 + i;
     const float qv = ldf(gq + t * p.ld_q + hk * d + c), kv = ldf(gk + t * p.ld_k + hk * d + c);
-    if (DELTA) {
-      sQ[i * ds + c] = qv;
-      sK[i * ds + c] = kv;
-      const float av = ldf(static_cast<const S*>(p.a) + t * p.ld_a + h * d + c) + p.dt_bias[h * d + c];
-      sL[i * ds + c] = a_neg * softplus_f(av);
-    } else {
-      sQ[i * ds + c] = SILU ? silu_f(qv) : qv;
-      sK[i * ds + c] = SILU ? silu_f(kv) : kv * p.k_scale;
-    }
+    sQ[i * ds + c] = qv;
+    sK[i * ds + c] = kv;
+    const float av = ldf(static_cast<const S*>(p.a) + t * p.ld_a + h * d + c) + p.dt_bias[h * d + c];
+    sL[i * ds + c] = a_neg * softplus_f(av);
   }
-  if (DELTA && tid < n) s_beta[tid] = sigmoid_c(ldf(static_cast<const S*>(p.beta) + static_cast<long long>(t0 + tid) * p.ld_beta + h));
+  if (tid < n) s_beta[tid] = sigmoid_c(ldf(static_cast<const S*>(p.beta) + static_cast<long long>(t0 + tid) * p.ld_beta + h));
   __syncthreads();
-  if (RULE == kRuleRetention && p.rot.rot_dims > 0) {
-    rotate_rows(sQ, sK, ds, n, t0, p.rot, tid, kPrepThreads);
-    __syncthreads();
-  }
-  const float log_a = DELTA ? 0.f : logf(fmaxf(p.decay[h], 1e-38f));
-  if (DELTA) {
-    for (int i = warp; i < n; i += kPrepThreads / 32) {  // unit length per token
-      float sq = 0.f, sk = 0.f;
-      for (int c = lane; c < d; c += 32) {
-        sq += sQ[i * ds + c] * sQ[i * ds + c];
-        sk += sK[i * ds + c] * sK[i * ds + c];
-      }
-      sq = warp_sum(sq);
-      sk = warp_sum(sk);
-      const float fq = p.q_scale / sqrtf(sq + p.unit_eps), fk = 1.f / sqrtf(sk + p.unit_eps);
-      for (int c = lane; c < d; c += 32) {
-        sQ[i * ds + c] *= fq;
-        sK[i * ds + c] *= fk;
-      }
+  for (int i = warp; i < n; i += kPrepThreads / 32) {  // unit length per token
+    float sq = 0.f, sk = 0.f;
+    for (int c = lane; c < d; c += 32) {
+      sq += sQ[i * ds + c] * sQ[i * ds + c];
+      sk += sK[i * ds + c] * sK[i * ds + c];
     }
-    for (int c = tid; c < d; c += kPrepThreads) {  // running sums of the logarithms
-      float run = 0.f;
-      for (int i = 0; i < n; ++i) {
-        run += sL[i * ds + c];
-        sL[i * ds + c] = run;
-      }
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    const float fq = p.q_scale / sqrtf(sq + p.unit_eps), fk = 1.f / sqrtf(sk + p.unit_eps);
+    for (int c = lane; c < d; c += 32) {
+      sQ[i * ds + c] *= fq;
+      sK[i * ds + c] *= fk;
     }
-    __syncthreads();
   }
+  for (int c = tid; c < d; c += kPrepThreads) {  // running sums of the logarithms
+    float run = 0.f;
+    for (int i = 0; i < n; ++i) {
+      run += sL[i * ds + c];
+      sL[i * ds + c] = run;
+    }
+  }
+  __syncthreads();
 
   // ---- A (delta) and B
-  if (DELTA && p.sub_blocks) {
+  if (p.sub_blocks) {
     // Pairs inside one sub-block of 16 tokens: the exponential per channel.  A warp takes two rows,
     // 16 lanes each, a lane one column of the row's sub-block.
     for (int i2 = 2 * warp; i2 < n; i2 += 2 * (kPrepThreads / 32)) {
@@ -224,18 +213,13 @@ __global__ void __launch_bounds__(kPrepThreads)
       if (j > i) continue;
       const float* kj = sK + j * ds;
       float accA = 0.f, accB = 0.f;
-      if (DELTA) {
-        const float* lj = sL + j * ds;
-        for (int c = 0; c < d; ++c) {
-          const float w = expf(li[c] - lj[c]) * kj[c];
-          accA += ki[c] * w;
-          accB += qi[c] * w;
-        }
-        sA[i * (kChunk + 1) + j] = accA;
-      } else {
-        for (int c = 0; c < d; ++c) accB += qi[c] * kj[c];
-        accB *= expf(log_a * static_cast<float>(i - j));
+      const float* lj = sL + j * ds;
+      for (int c = 0; c < d; ++c) {
+        const float w = expf(li[c] - lj[c]) * kj[c];
+        accA += ki[c] * w;
+        accB += qi[c] * w;
       }
+      sA[i * (kChunk + 1) + j] = accA;
       oB[i * kChunk + j] = accB;
     }
   }
@@ -243,20 +227,11 @@ __global__ void __launch_bounds__(kPrepThreads)
   // ---- q * exp L, k * exp(L_end - L), exp L_end
   for (int e = tid; e < n * d; e += kPrepThreads) {
     const int i = e / d, c = e - i * d;
-    const float up = DELTA ? sL[i * ds + c] : log_a * static_cast<float>(i + 1);
-    const float end = DELTA ? sL[(n - 1) * ds + c] : log_a * static_cast<float>(n);
+    const float up = sL[i * ds + c], end = sL[(n - 1) * ds + c];
     oQg[i * d + c] = sQ[i * ds + c] * expf(up);
     oKe[i * d + c] = sK[i * ds + c] * expf(end - up);
   }
-  for (int c = tid; c < d; c += kPrepThreads) oEg[c] = expf(DELTA ? sL[(n - 1) * ds + c] : log_a * static_cast<float>(n));
-  if (!DELTA) {
-    for (int e = tid; e < n * dv; e += kPrepThreads) {
-      const int i = e / dv, c = e - i * dv;
-      const float vv = ldf(gv + static_cast<long long>(t0 + i) * p.ld_v + h * dv + c);
-      oUv[i * dv + c] = SILU ? silu_f(vv) : vv;
-    }
-    return;
-  }
+  for (int c = tid; c < d; c += kPrepThreads) oEg[c] = expf(sL[(n - 1) * ds + c]);
   __syncthreads();  // A is whole; q is no longer needed: its rows become the right-hand sides
 
   // ---- T X = diag(beta) R by forward substitution in place, a thread per column.  R = K * exp L
@@ -301,6 +276,114 @@ __global__ void __launch_bounds__(kPrepThreads)
 }
 
 // ----------------------------------------------------------------------------------------------
+// Four neighbouring elements of a row in the storage type (`vec`: the row starts on a boundary of four elements).
+template <typename S>
+__device__ __forceinline__ float4 load4(const S* p, bool vec) {
+  if (!vec) return make_float4(ldf(p), ldf(p + 1), ldf(p + 2), ldf(p + 3));
+  return ldf4(p);
+}
+
+// The values of the chunk's tokens as floats (silu of them for kRuleDecay), eight or four bytes at a time where they lie so
+template <typename S, bool SILU>
+__device__ __forceinline__ void widen_values(const ChunkArgs& p, float* __restrict__ oUv, int h, int t0, int n, int tid, int n_threads) {
+  const int dv = p.dv;
+  const S* gv = static_cast<const S*>(p.v) + static_cast<long long>(t0) * p.ld_v + h * dv;
+  if (dv % 4 == 0) {
+    for (int e = tid; e < n * (dv / 4); e += n_threads) {
+      const int i = e / (dv / 4), c = 4 * (e - i * (dv / 4));
+      float4 v = load4(gv + static_cast<long long>(i) * p.ld_v + c, p.vec_in != 0);
+      if (SILU) v = make_float4(silu_f(v.x), silu_f(v.y), silu_f(v.z), silu_f(v.w));
+      *reinterpret_cast<float4*>(oUv + static_cast<size_t>(i) * dv + c) = v;
+    }
+    return;
+  }
+  for (int e = tid; e < n * dv; e += n_threads) {
+    const int i = e / dv, c = e - i * dv;
+    const float v = ldf(gv + static_cast<long long>(i) * p.ld_v + c);
+    oUv[e] = SILU ? silu_f(v) : v;
+  }
+}
+
+// The operands of the decayed sum (kRuleDecay, kRuleRetention): B_ij = (q_i . k_j) a^(i-j), Q * a^(i+1), K * a^(n-1-i), a^n.
+// Rows of stride d + 4: sixteen-byte reads of neighbouring rows fall into different banks.  A thread makes a 4 x 4
+// piece of B.
+constexpr int kDecayPrepThreads = 256;
+
+inline size_t decay_prepare_smem(int d) { return sizeof(float) * (static_cast<size_t>(2 * kChunk) * (d + 4)); }
+
+template <typename S, int RULE>
+__global__ void __launch_bounds__(kDecayPrepThreads)
+    decay_prepare_kernel(ChunkArgs p) {
+  extern __shared__ __align__(16) float sm[];
+  constexpr bool SILU = RULE == kRuleDecay;
+  const int d = p.d, d4 = d / 4, ds = d + 4;
+  float* sK = sm;                  // [C][ds]
+  float* sQ = sK + kChunk * ds;    // [C][ds]
+  __shared__ float s_pow[kChunk + 1];  // a^0 .. a^C
+  pdl_launch_dependents();
+  pdl_wait();
+  const int chunk = blockIdx.x, h = blockIdx.y;
+  int seq, t0, n;
+  if (!locate_chunk(p.cu, p.n_seq, chunk, &seq, &t0, &n)) return;
+  const int tid = threadIdx.x;
+  const size_t ch = static_cast<size_t>(chunk) * p.H + h;
+  if (tid <= kChunk) s_pow[tid] = expf(logf(fmaxf(p.decay[h], 1e-38f)) * static_cast<float>(tid));
+  for (int e = tid; e < n * d4; e += kDecayPrepThreads) {
+    const int i = e / d4, c = 4 * (e - i * d4);
+    const long long t = t0 + i;
+    float4 q = load4(static_cast<const S*>(p.q) + t * p.ld_q + h * d + c, p.vec_in != 0);
+    float4 k = load4(static_cast<const S*>(p.k) + t * p.ld_k + h * d + c, p.vec_in != 0);
+    if (SILU) {
+      q = make_float4(silu_f(q.x), silu_f(q.y), silu_f(q.z), silu_f(q.w));
+      k = make_float4(silu_f(k.x), silu_f(k.y), silu_f(k.z), silu_f(k.w));
+    } else {
+      k = make_float4(k.x * p.k_scale, k.y * p.k_scale, k.z * p.k_scale, k.w * p.k_scale);
+    }
+    *reinterpret_cast<float4*>(sQ + i * ds + c) = q;
+    *reinterpret_cast<float4*>(sK + i * ds + c) = k;
+  }
+  widen_values<S, SILU>(p, p.Uv + ch * kChunk * p.dv, h, t0, n, tid, kDecayPrepThreads);
+  __syncthreads();
+  if (RULE == kRuleRetention && p.rot.rot_dims > 0) {
+    rotate_rows(sQ, sK, ds, n, t0, p.rot, tid, kDecayPrepThreads);
+    __syncthreads();
+  }
+  float* oB = p.B + ch * kChunk * kChunk;
+  // (rows at and beyond n hold stale values whose results are not stored)
+  const int i0 = 4 * (tid / 16), j0 = 4 * (tid % 16);
+  if (j0 <= i0 && i0 < n) {
+    float acc[4][4] = {};
+    for (int c = 0; c < d; c += 4) {
+      float4 q[4], k[4];
+#pragma unroll
+      for (int r = 0; r < 4; ++r) {
+        q[r] = *reinterpret_cast<const float4*>(sQ + (i0 + r) * ds + c);
+        k[r] = *reinterpret_cast<const float4*>(sK + (j0 + r) * ds + c);
+      }
+#pragma unroll
+      for (int r = 0; r < 4; ++r)
+#pragma unroll
+        for (int s = 0; s < 4; ++s) acc[r][s] += q[r].x * k[s].x + q[r].y * k[s].y + q[r].z * k[s].z + q[r].w * k[s].w;
+    }
+#pragma unroll
+    for (int r = 0; r < 4; ++r)
+#pragma unroll
+      for (int s = 0; s < 4; ++s)
+        if (i0 + r < n && j0 + s <= i0 + r) oB[(i0 + r) * kChunk + j0 + s] = acc[r][s] * s_pow[i0 + r - j0 - s];
+  }
+  float* oQg = p.Qg + ch * kChunk * d;
+  float* oKe = p.Ke + ch * kChunk * d;
+  for (int e = tid; e < n * d4; e += kDecayPrepThreads) {
+    const int i = e / d4, c = 4 * (e - i * d4);
+    const float up = s_pow[i + 1], down = s_pow[n - 1 - i];
+    const float4 q = *reinterpret_cast<const float4*>(sQ + i * ds + c), k = *reinterpret_cast<const float4*>(sK + i * ds + c);
+    *reinterpret_cast<float4*>(oQg + i * d + c) = make_float4(q.x * up, q.y * up, q.z * up, q.w * up);
+    *reinterpret_cast<float4*>(oKe + i * d + c) = make_float4(k.x * down, k.y * down, k.z * down, k.w * down);
+  }
+  for (int c = tid; c < d; c += kDecayPrepThreads) p.Eg[ch * d + c] = s_pow[n];
+}
+
+// ----------------------------------------------------------------------------------------------
 // The same operands for time mixing.  Sums of logarithms are kept within sub-blocks of 16 tokens only (sL: up to and
 // including the token; sT: a sub-block's total), so that strong decays do not drown the weak ones behind them, and a
 // token's logarithm is bounded at -40 (4e-18: below the rounding of anything it could stand beside).  Rows of stride
@@ -308,16 +391,20 @@ __global__ void __launch_bounds__(kPrepThreads)
 //   pairs within a sub-block:  B_ij = sum_c q_i[c] k_j[c] exp(L_(i-1) - L_j),  B_ii with the bonus;
 //   then in place  q_i <- q_i exp(L_(i-1) of its sub-block),  k_j <- k_j exp(T - L_j)  (weakened to its sub-block's end);
 //   sub-block by sub-block, all rows of k before it are weakened to its start: pairs across are dot products.
+// Logarithms are to base 2 (one instruction less for every exponential).
 // What is left of q and k at the end is, up to whole sub-blocks' totals, Q * exp L and K * exp(L_end - L).
 constexpr float kLogDecayFloor = -40.f;
+constexpr float kLog2E = 1.4426950408889634f;
+
+constexpr int kWkvThreads = 256;
 
 inline size_t wkv_prepare_smem(int d) { return sizeof(float) * (static_cast<size_t>(3 * kChunk) * (d + 4) + 4 * static_cast<size_t>(d)); }
 
 template <typename S>
-__global__ void __launch_bounds__(kPrepThreads)
+__global__ void __launch_bounds__(kWkvThreads)
     wkv_prepare_kernel(ChunkArgs p) {
   extern __shared__ __align__(16) float sm[];
-  const int d = p.d, dv = p.dv, ds = d + 4;
+  const int d = p.d, d4 = d / 4, dv = p.dv, ds = d + 4;
   float* sK = sm;                  // [C][ds]
   float* sQ = sK + kChunk * ds;    // [C][ds]
   float* sL = sQ + kChunk * ds;    // [C][ds]
@@ -335,19 +422,23 @@ __global__ void __launch_bounds__(kPrepThreads)
   float* oUv = p.Uv + ch * kChunk * dv;
   const int nb = (n + 15) >> 4;
 
-  for (int e = tid; e < n * d; e += kPrepThreads) {
-    const int i = e / d, c = e - i * d;
+  const bool vec = p.vec_in != 0;
+#pragma unroll 2
+  for (int e = tid; e < n * d4; e += kWkvThreads) {
+    const int i = e / d4, c = 4 * (e - i * d4);
     const long long t = t0 + i;
-    sQ[i * ds + c] = ldf(static_cast<const S*>(p.q) + t * p.ld_q + h * d + c);
-    sK[i * ds + c] = ldf(static_cast<const S*>(p.k) + t * p.ld_k + h * d + c);
-    sL[i * ds + c] = fmaxf(-expf(static_cast<const float*>(p.a)[t * p.ld_a + h * d + c] + p.dt_bias[h * d + c]), kLogDecayFloor);
+    const float4 q = load4(static_cast<const S*>(p.q) + t * p.ld_q + h * d + c, vec);
+    const float4 k = load4(static_cast<const S*>(p.k) + t * p.ld_k + h * d + c, vec);
+    const float4 a = load4(static_cast<const float*>(p.a) + t * p.ld_a + h * d + c, vec);
+    const float4 b = load4(p.dt_bias + h * d + c, vec);
+    auto decay = [](float z) { return fmaxf(-expf(z), kLogDecayFloor) * kLog2E; };
+    *reinterpret_cast<float4*>(sQ + i * ds + c) = q;
+    *reinterpret_cast<float4*>(sK + i * ds + c) = k;
+    *reinterpret_cast<float4*>(sL + i * ds + c) = make_float4(decay(a.x + b.x), decay(a.y + b.y), decay(a.z + b.z), decay(a.w + b.w));
   }
-  for (int e = tid; e < n * dv; e += kPrepThreads) {
-    const int i = e / dv, c = e - i * dv;
-    oUv[e] = ldf(static_cast<const S*>(p.v) + static_cast<long long>(t0 + i) * p.ld_v + h * dv + c);
-  }
+  widen_values<S, false>(p, oUv, h, t0, n, tid, kWkvThreads);
   __syncthreads();
-  for (int e = tid; e < nb * d; e += kPrepThreads) {
+  for (int e = tid; e < nb * d; e += kWkvThreads) {
     const int blk = e / d, c = e - blk * d;
     float run = 0.f;
     for (int i = 16 * blk; i < min(16 * blk + 16, n); ++i) {
@@ -359,7 +450,7 @@ __global__ void __launch_bounds__(kPrepThreads)
   __syncthreads();
 
   // ---- pairs within a sub-block: a warp takes two rows, 16 lanes each, a lane one column of the row's sub-block
-  for (int i2 = 2 * warp; i2 < n; i2 += 2 * (kPrepThreads / 32)) {
+  for (int i2 = 2 * warp; i2 < n; i2 += 2 * (kWkvThreads / 32)) {
     const int i = i2 + (lane >> 4), j = (i & ~15) + (lane & 15);
     if (i < n && j <= i) {
       const float *qi = sQ + i * ds, *kj = sK + j * ds, *lj = sL + j * ds, *li = sL + (i > 0 ? i - 1 : 0) * ds;  // (i > j: row i - 1 is in the sub-block)
@@ -371,30 +462,35 @@ __global__ void __launch_bounds__(kPrepThreads)
           acc += q4.x * u[c] * k4.x + q4.y * u[c + 1] * k4.y + q4.z * u[c + 2] * k4.z + q4.w * u[c + 3] * k4.w;
         } else {
           const float4 a4 = *reinterpret_cast<const float4*>(li + c), b4 = *reinterpret_cast<const float4*>(lj + c);
-          acc += q4.x * k4.x * expf(a4.x - b4.x) + q4.y * k4.y * expf(a4.y - b4.y) + q4.z * k4.z * expf(a4.z - b4.z) +
-                 q4.w * k4.w * expf(a4.w - b4.w);
+          acc += q4.x * k4.x * exp2f(a4.x - b4.x) + q4.y * k4.y * exp2f(a4.y - b4.y) + q4.z * k4.z * exp2f(a4.z - b4.z) +
+                 q4.w * k4.w * exp2f(a4.w - b4.w);
         }
       }
       oB[i * kChunk + j] = acc;
     }
   }
   __syncthreads();
-  for (int e = tid; e < n * d; e += kPrepThreads) {
-    const int i = e / d, c = e - i * d;
-    if (i & 15) sQ[i * ds + c] *= expf(sL[(i - 1) * ds + c]);
-    sK[i * ds + c] *= expf(sT[(i >> 4) * d + c] - sL[i * ds + c]);
+  auto weaken = [](float* row, float4 l) {
+    float4 v = *reinterpret_cast<float4*>(row);
+    *reinterpret_cast<float4*>(row) = make_float4(v.x * exp2f(l.x), v.y * exp2f(l.y), v.z * exp2f(l.z), v.w * exp2f(l.w));
+  };
+  for (int e = tid; e < n * d4; e += kWkvThreads) {
+    const int i = e / d4, c = 4 * (e - i * d4);
+    if (i & 15) weaken(sQ + i * ds + c, *reinterpret_cast<const float4*>(sL + (i - 1) * ds + c));
+    const float4 t = *reinterpret_cast<const float4*>(sT + (i >> 4) * d + c), l = *reinterpret_cast<const float4*>(sL + i * ds + c);
+    weaken(sK + i * ds + c, make_float4(t.x - l.x, t.y - l.y, t.z - l.z, t.w - l.w));
   }
   // ---- pairs across: four rows of the sub-block and 32 columns a warp
   for (int blk = 1; blk < nb; ++blk) {
     __syncthreads();
     if (blk > 1) {  // rows before the last sub-block reach this one through its total
-      for (int e = tid; e < 16 * (blk - 1) * d; e += kPrepThreads) {
-        const int j = e / d, c = e - j * d;
-        sK[j * ds + c] *= expf(sT[(blk - 1) * d + c]);
+      for (int e = tid; e < 16 * (blk - 1) * d4; e += kWkvThreads) {
+        const int j = e / d4, c = 4 * (e - j * d4);
+        weaken(sK + j * ds + c, *reinterpret_cast<const float4*>(sT + (blk - 1) * d + c));
       }
       __syncthreads();
     }
-    const int rg = warp & 3, j = (warp >> 2) * 32 + lane;  // warps 8.. have no columns (at most 48 are before a sub-block)
+    const int rg = warp & 3, j = (warp >> 2) * 32 + lane;
     const int i0 = 16 * blk + 4 * rg;
     if (j < 16 * blk && i0 < n) {
       const float* kj = sK + j * ds;
@@ -415,18 +511,23 @@ __global__ void __launch_bounds__(kPrepThreads)
   }
   __syncthreads();
   // ---- what the other launches read: q weakened from the chunk's start, k to its end, the whole chunk's decay
-  for (int e = tid; e < n * d; e += kPrepThreads) {
-    const int i = e / d, c = e - i * d, blk = i >> 4;
-    float before = 0.f;
-    for (int b = 0; b < blk; ++b) before += sT[b * d + c];
-    oQg[e] = sQ[i * ds + c] * expf(before);
-    oKe[e] = sK[i * ds + c] * (blk < nb - 1 ? expf(sT[(nb - 1) * d + c]) : 1.f);
+  for (int e = tid; e < n * d4; e += kWkvThreads) {
+    const int i = e / d4, c = 4 * (e - i * d4), blk = i >> 4;
+    float4 l = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int b = 0; b < blk; ++b) {
+      const float4 t = *reinterpret_cast<const float4*>(sT + b * d + c);
+      l = make_float4(l.x + t.x, l.y + t.y, l.z + t.z, l.w + t.w);
+    }
+    const float4 q = *reinterpret_cast<const float4*>(sQ + i * ds + c);
+    *reinterpret_cast<float4*>(oQg + i * d + c) = make_float4(q.x * exp2f(l.x), q.y * exp2f(l.y), q.z * exp2f(l.z), q.w * exp2f(l.w));
+    if (blk < nb - 1) weaken(sK + i * ds + c, *reinterpret_cast<const float4*>(sT + (nb - 1) * d + c));
+    *reinterpret_cast<float4*>(oKe + i * d + c) = *reinterpret_cast<const float4*>(sK + i * ds + c);
   }
   float* oEg = p.Eg + ch * d;
-  for (int c = tid; c < d; c += kPrepThreads) {
+  for (int c = tid; c < d; c += kWkvThreads) {
     float all = 0.f;
     for (int b = 0; b < nb; ++b) all += sT[b * d + c];
-    oEg[c] = expf(all);
+    oEg[c] = exp2f(all);
   }
 }
 
@@ -650,6 +751,28 @@ __device__ __forceinline__ void product_nn(float (&acc)[4][4], const float* __re
   }
 }
 
+// `count` floats (a multiple of 4, 16-byte aligned at both ends) by asynchronous copies
+__device__ __forceinline__ void copy_rows(float* __restrict__ dst, const float* __restrict__ src, int count, int tid) {
+  for (int e = 4 * tid; e < count; e += 4 * kDecayThreads) cp_async16(dst + e, src + e);
+}
+
+// Columns c0 .. c0 + 63 of `rows` rows of a [rows, dv] matrix, zeros beyond dv
+__device__ __forceinline__ void copy_tile(float* __restrict__ dst, const float* __restrict__ src, int rows, int dv, int c0, int tid) {
+  if (dv % 4 == 0 && reinterpret_cast<uintptr_t>(src) % 16 == 0) {
+    for (int e = tid; e < rows * (kDecayTile / 4); e += kDecayThreads) {
+      const int j = e / (kDecayTile / 4), c = 4 * (e % (kDecayTile / 4));
+      float* to = dst + j * kDecayTile + c;
+      if (c0 + c < dv) cp_async16(to, src + static_cast<size_t>(j) * dv + c0 + c);
+      else *reinterpret_cast<float4*>(to) = make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    return;
+  }
+  for (int e = tid; e < rows * kDecayTile; e += kDecayThreads) {
+    const int j = e / kDecayTile, c = e % kDecayTile;
+    dst[e] = (c0 + c < dv) ? src[static_cast<size_t>(j) * dv + c0 + c] : 0.f;
+  }
+}
+
 // N [d, dv] per (chunk, head), chunk-major
 __global__ void __launch_bounds__(kDecayThreads)
     decay_chunk_state_kernel(ChunkArgs p) {
@@ -666,11 +789,10 @@ __global__ void __launch_bounds__(kDecayThreads)
   const size_t ch = static_cast<size_t>(chunk) * p.H + h;
   const float* gKe = p.Ke + ch * kChunk * d;
   const float* gV = p.Uv + ch * kChunk * dv;
-  for (int e = tid; e < n * d; e += kDecayThreads) sKe[e] = gKe[e];
-  for (int e = tid; e < n * kDecayTile; e += kDecayThreads) {
-    const int j = e / kDecayTile, c = e % kDecayTile;
-    sV[e] = (c0 + c < dv) ? gV[static_cast<size_t>(j) * dv + c0 + c] : 0.f;
-  }
+  copy_rows(sKe, gKe, n * d, tid);
+  copy_tile(sV, gV, n, dv, c0, tid);
+  cp_async_commit();
+  cp_async_wait<0>();
   __syncthreads();
   float* gN = p.N + ch * static_cast<size_t>(d) * dv;
   const int cc = 4 * (tid % 16);
@@ -730,8 +852,7 @@ __global__ void __launch_bounds__(kDecayThreads)
   extern __shared__ __align__(16) float sm[];
   const int d = p.d, dv = p.dv;
   float* sQg = sm;                          // [C][d]
-  float* sB = sQg + kChunk * d;             // [C][C]
-  float* sS = sB + kChunk * kChunk;         // [d][tile]
+  float* sS = sQg + kChunk * d;             // [d][tile]
   float* sV = sS + d * kDecayTile;          // [C][tile]
   pdl_launch_dependents();
   pdl_wait();
@@ -744,16 +865,11 @@ __global__ void __launch_bounds__(kDecayThreads)
   const float* gB = p.B + ch * kChunk * kChunk;
   const float* gS = p.N + ch * static_cast<size_t>(d) * dv;
   const float* gV = p.Uv + ch * kChunk * dv;
-  for (int e = tid; e < n * d; e += kDecayThreads) sQg[e] = gQg[e];
-  for (int e = tid; e < n * kChunk; e += kDecayThreads) sB[e] = gB[e];
-  for (int e = tid; e < d * kDecayTile; e += kDecayThreads) {
-    const int k = e / kDecayTile, c = e % kDecayTile;
-    sS[e] = (c0 + c < dv) ? gS[static_cast<size_t>(k) * dv + c0 + c] : 0.f;
-  }
-  for (int e = tid; e < n * kDecayTile; e += kDecayThreads) {
-    const int j = e / kDecayTile, c = e % kDecayTile;
-    sV[e] = (c0 + c < dv) ? gV[static_cast<size_t>(j) * dv + c0 + c] : 0.f;
-  }
+  copy_rows(sQg, gQg, n * d, tid);
+  copy_tile(sS, gS, d, dv, c0, tid);
+  copy_tile(sV, gV, n, dv, c0, tid);
+  cp_async_commit();
+  cp_async_wait<0>();
   __syncthreads();
   // thread: rows i0 .. i0 + 3, columns cc .. cc + 3 (rows at and beyond n hold stale values that are not stored)
   const int cc = 4 * (tid % 16), i0 = 4 * (tid / 16);
@@ -764,7 +880,7 @@ __global__ void __launch_bounds__(kDecayThreads)
 #pragma unroll
       for (int c = 0; c < 4; ++c) acc[r][c] = 0.f;
     product_nn(acc, sQg, d, i0, sS, cc, d, false);
-    product_nn(acc, sB, kChunk, i0, sV, cc, i0 + 4, true);
+    product_nn(acc, gB, kChunk, i0, sV, cc, i0 + 4, true);  // (B from the L1 cache: one more block fits an SM)
 #pragma unroll
     for (int r = 0; r < 4; ++r)
 #pragma unroll
@@ -971,8 +1087,8 @@ __global__ void __launch_bounds__(kDecayThreads)
 
 inline size_t prepare_smem(int d, int rule, bool sub_blocks = false) {
   if (rule == kRuleWkv) return wkv_prepare_smem(d);
-  const bool delta = rule == kRuleDelta;
-  return sizeof(float) * (static_cast<size_t>(kChunk) * (d + 1) * (delta ? 3 : 2) + (delta ? kChunk * (kChunk + 1) : 0) +
+  if (rule != kRuleDelta) return decay_prepare_smem(d);
+  return sizeof(float) * (static_cast<size_t>(kChunk) * (d + 1) * 3 + kChunk * (kChunk + 1) +
                           (sub_blocks ? static_cast<size_t>(48 + 32) * (d + 1) : 0));
 }
 inline size_t apply_smem(int d, bool delta, int nc = 16) {
@@ -987,12 +1103,17 @@ int launch_chunked(ChunkArgs a, int n_chunks, cudaStream_t stream) {
   const size_t sp = prepare_smem(a.d, RULE, a.sub_blocks != 0);
   void (*prep)(ChunkArgs) = nullptr;
   if constexpr (RULE == kRuleWkv) prep = wkv_prepare_kernel<S>;
-  else prep = chunk_prepare_kernel<S, RULE>;
+  else if constexpr (DELTA) prep = chunk_prepare_kernel<S>;
+  else prep = decay_prepare_kernel<S, RULE>;
+  const size_t unit = 4 * sizeof(S);
+  auto whole = [&](const void* ptr, long long ld) { return reinterpret_cast<uintptr_t>(ptr) % unit == 0 && ld % 4 == 0; };
+  a.vec_in = whole(a.q, a.ld_q) && whole(a.k, a.ld_k) && whole(a.v, a.ld_v) &&
+             (RULE != kRuleWkv || (reinterpret_cast<uintptr_t>(a.a) % 16 == 0 && a.ld_a % 4 == 0 && reinterpret_cast<uintptr_t>(a.dt_bias) % 16 == 0));
   if (sp > 48 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(prep, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(sp));
     if (e != cudaSuccess) return static_cast<int>(e);
   }
-  launch_pdl(prep, dim3(n_chunks, a.H), dim3(kPrepThreads), sp, stream, a);
+  launch_pdl(prep, dim3(n_chunks, a.H), dim3(DELTA ? kPrepThreads : RULE == kRuleWkv ? kWkvThreads : kDecayPrepThreads), sp, stream, a);
   if (DELTA) {
     const int d = a.d;
     const int tiles_c = (d + a.dv + kDecayTile - 1) / kDecayTile, tiles_o = (a.dv + kDecayTile - 1) / kDecayTile;
@@ -1019,8 +1140,7 @@ int launch_chunked(ChunkArgs a, int n_chunks, cudaStream_t stream) {
   if (!DELTA) {
     const int tiles = (a.dv + kDecayTile - 1) / kDecayTile;
     const size_t s1 = sizeof(float) * kChunk * (static_cast<size_t>(a.d) + kDecayTile);
-    const size_t s3 = sizeof(float) * (static_cast<size_t>(kChunk) * a.d + kChunk * kChunk +
-                                       static_cast<size_t>(a.d) * kDecayTile + kChunk * kDecayTile);
+    const size_t s3 = sizeof(float) * (static_cast<size_t>(kChunk) * a.d + static_cast<size_t>(a.d) * kDecayTile + kChunk * kDecayTile);
     if (s3 <= 200 * 1024 && tiles <= 65535) {
       for (auto pair : {std::make_pair(decay_chunk_state_kernel, s1), std::make_pair(decay_chunk_output_kernel, s3)}) {
         if (pair.second > 48 * 1024) {

@@ -233,6 +233,125 @@ __global__ void __launch_bounds__(kHeadRopeWarps * 32)
   }
 }
 
+// The same for heads of an even size whose turning pairs are neighbours (or that do not turn): a lane holds the pairs
+// lane, lane + 32, ... of a head, so the partner is its own and the sines and cosines, made once, serve every row of the
+// token that the warp takes (rows warp, warp + WARPS, ..., all of them loaded before the first is used).
+template <typename S, int NP, int ROWS>  // NP pairs per lane: heads of up to 64 NP entries
+__global__ void __launch_bounds__(kHeadRopeWarps * 32)
+    head_norm_rope_pairs_kernel(const HeadRopeArgs p) {
+  pdl_launch_dependents();
+  const int t = blockIdx.x;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int n_rows = p.H + 2 * p.G, half = p.rot_dims >> 1;
+  const int first = (blockIdx.y * kHeadRopeWarps + warp) * ROWS;
+  pdl_wait();
+  if (first >= n_rows) return;
+  const int pos = p.positions[t];
+  float2 x[ROWS][NP];
+#pragma unroll
+  for (int r = 0; r < ROWS; ++r) {
+    const int row = first + r;
+    const bool is_q = row < p.H, is_v = row >= p.H + p.G;
+    const int h = is_q ? row : is_v ? row - p.H - p.G : row - p.H;
+    const int width = is_v ? p.dv : p.d;
+    const S* src = (is_q ? static_cast<const S*>(p.q) + static_cast<long long>(t) * p.ld_q
+                         : is_v ? static_cast<const S*>(p.v) + static_cast<long long>(t) * p.ld_v
+                                : static_cast<const S*>(p.k) + static_cast<long long>(t) * p.ld_k) + h * width;
+    const float* bias = is_q ? p.q_bias : is_v ? p.v_bias : p.k_bias;
+#pragma unroll
+    for (int j = 0; j < NP; ++j) {
+      const int i = 2 * (lane + 32 * j);
+      x[r][j] = make_float2(0.f, 0.f);
+      if (row < n_rows && i < width) {
+        x[r][j] = ldf2(src + i);
+        if (bias) {
+          const float2 b = ldf2(bias + h * width + i);
+          x[r][j].x += b.x;
+          x[r][j].y += b.y;
+        }
+      }
+    }
+  }
+  float2 turn[NP];  // cosine, sine
+  if (first < p.H + p.G) {
+#pragma unroll
+    for (int j = 0; j < NP; ++j) {
+      const int f = lane + 32 * j;
+      turn[j] = make_float2(1.f, 0.f);
+      if (f < half) {
+        float s, c;
+        sincosf(static_cast<float>(pos) * p.inv_freq[f], &s, &c);
+        turn[j] = make_float2(c * p.amplitude, s * p.amplitude);
+      }
+    }
+  }
+  S* page_row = nullptr;
+  if (first + ROWS > p.H) {
+    const int page = p.block_table[static_cast<size_t>(p.seq_of[t]) * p.max_blocks + pos / p.page_size];
+    page_row = static_cast<S*>(p.pool) + (static_cast<size_t>(page) * 2 * p.page_size + pos % p.page_size) * (p.G * p.Dp);
+  }
+#pragma unroll
+  for (int r = 0; r < ROWS; ++r) {
+    const int row = first + r;
+    if (row >= n_rows) return;
+    if (row >= p.H + p.G) {
+      const int g = row - p.H - p.G;
+      S* vals = p.values ? static_cast<S*>(p.values) + (static_cast<size_t>(t) * p.G + g) * p.dv : nullptr;
+      S* dst = page_row + static_cast<size_t>(p.page_size) * (p.G * p.Dp) + g * p.Dp;
+      const float l = p.mix ? *p.mix : 0.f;
+#pragma unroll
+      for (int j = 0; j < NP; ++j) {
+        const int i = 2 * (lane + 32 * j);
+        if (i < p.dv) {
+          if (p.mix) {
+            const float2 y = ldf2(vals + i);
+            x[r][j] = make_float2((1.f - l) * x[r][j].x + l * y.x, (1.f - l) * x[r][j].y + l * y.y);
+          } else if (vals) {
+            stf2(vals + i, x[r][j]);
+          }
+        }
+        if (i < p.Dp) stf2(dst + i, x[r][j]);
+      }
+      continue;
+    }
+    const bool is_q = row < p.H;
+    const int h = is_q ? row : row - p.H;
+    if (p.norm_eps >= 0.f) {
+      const float* w = is_q ? p.q_w : p.k_w;
+      float ss = 0.f;
+#pragma unroll
+      for (int j = 0; j < NP; ++j) ss += x[r][j].x * x[r][j].x + x[r][j].y * x[r][j].y;
+      const float inv = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(p.d) + p.norm_eps);
+#pragma unroll
+      for (int j = 0; j < NP; ++j) {
+        const int i = 2 * (lane + 32 * j);
+        float2 g = make_float2(1.f, 1.f);
+        if (w && i < p.d) g = ldf2(w + i);
+        x[r][j] = make_float2(x[r][j].x * inv * g.x, x[r][j].y * inv * g.y);
+      }
+    }
+    S* dst = is_q ? static_cast<S*>(p.q_out) + (static_cast<size_t>(t) * p.H + h) * p.Dp : page_row + h * p.Dp;
+#pragma unroll
+    for (int j = 0; j < NP; ++j) {
+      const int i = 2 * (lane + 32 * j);
+      const float2 y = make_float2(x[r][j].x * turn[j].x - x[r][j].y * turn[j].y, x[r][j].y * turn[j].x + x[r][j].x * turn[j].y);
+      if (i < p.Dp) stf2(dst + i, y);  // (entries from d on are zero; what does not turn has cosine one, sine zero)
+    }
+  }
+}
+
+template <typename S, int NP>
+void launch_head_rope_pairs(const HeadRopeArgs& a, int T, cudaStream_t stream) {
+  const int n_rows = a.H + 2 * a.G;
+  const int warps1 = n_rows, warps2 = (n_rows + 1) / 2;
+  if (T >= 128)  // enough tokens to fill the GPU: two rows a warp
+    launch_pdl(head_norm_rope_pairs_kernel<S, NP, 2>, dim3(T, (warps2 + kHeadRopeWarps - 1) / kHeadRopeWarps),
+               dim3(kHeadRopeWarps * 32), 0, stream, a);
+  else
+    launch_pdl(head_norm_rope_pairs_kernel<S, NP, 1>, dim3(T, (warps1 + kHeadRopeWarps - 1) / kHeadRopeWarps),
+               dim3(kHeadRopeWarps * 32), 0, stream, a);
+}
+
 }  // namespace pmm
 
 // q [T, H*d], k [T, G*d], v [T, G*dv] rows of stride ld; inv_freq [rot_dims/2] floats (may be nullptr when
@@ -277,6 +396,18 @@ PMM_EXPORT int pmm_head_norm_rope_store(const void* q, long long ld_q, const voi
   const pmm::HeadRopeArgs a{q, k, v, ld_q, ld_k, ld_v, inv_freq, positions, seq_of, block_table, max_blocks, page_size,
                             pool, q_out, H, G, d, dv, Dp, rot_dims, half_layout, amplitude, q_bias, k_bias, v_bias,
                             norm_eps, q_w, k_w, values, mix};
+  const size_t unit = dtype == PMM_DTYPE_BF16 ? 4 : 8;
+  auto even = [](const void* ptr, size_t bytes) { return reinterpret_cast<uintptr_t>(ptr) % bytes == 0; };
+  if ((rot_dims == 0 || !half_layout) && d % 2 == 0 && dv % 2 == 0 && Dp % 2 == 0 && ld_q % 2 == 0 && ld_k % 2 == 0 && ld_v % 2 == 0 &&
+      even(q, unit) && even(k, unit) && even(v, unit) && even(pool, unit) && even(q_out, unit) && even(values, unit) &&
+      even(q_bias, 8) && even(k_bias, 8) && even(v_bias, 8) && even(q_w, 8) && even(k_w, 8)) {
+    PMM_DISPATCH_DTYPE(dtype, S, {
+      if (Dp <= 64) pmm::launch_head_rope_pairs<S, 1>(a, T, stream);
+      else if (Dp <= 128) pmm::launch_head_rope_pairs<S, 2>(a, T, stream);
+      else pmm::launch_head_rope_pairs<S, 4>(a, T, stream);
+    });
+    return pmm::launch_status();
+  }
   const dim3 grid(T, (H + 2 * G + pmm::kHeadRopeWarps - 1) / pmm::kHeadRopeWarps);
   PMM_DISPATCH_DTYPE(dtype, S, pmm::launch_pdl(pmm::head_norm_rope_store_kernel<S>, grid, dim3(pmm::kHeadRopeWarps * 32), 0, stream, a));
   return pmm::launch_status();

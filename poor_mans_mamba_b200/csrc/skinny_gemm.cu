@@ -411,7 +411,7 @@ __device__ void SkinnyBlock<MT, MODE>::finish_tile(float (&acc)[MT][4], int n0) 
           if (MODE == kSgMulti) {
             pr.y[static_cast<size_t>(m) * pr.ldy + n] = __float2bfloat16_rn(acc[nt][e]);
           } else if (MODE == kSgGelu) {
-            args.y[static_cast<size_t>(m) * args.ldy + n] = __float2bfloat16_rn(gelu_erf_f(acc[nt][e]));
+            args.y[static_cast<size_t>(m) * args.ldy + n] = __float2bfloat16_rn(gelu_erf_fast(acc[nt][e]));
           } else if (MODE == kSgStore) {
             const float inv = pr.h_in ? sInv[m] : 1.f;  // the row's norm factor (norm prologue)
             args.y[static_cast<size_t>(m) * args.ldy + n] = __float2bfloat16_rn(acc[nt][e] * inv);

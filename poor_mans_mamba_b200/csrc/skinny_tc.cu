@@ -263,7 +263,7 @@ __global__ void __launch_bounds__(kStThreads)
       } else if (MODE == kStStore || MODE == kStGelu) {
         if (MODE == kStGelu) {
 #pragma unroll
-          for (int e = 0; e < 32; ++e) v[e] = __float_as_uint(gelu_erf_f(__uint_as_float(v[e])));
+          for (int e = 0; e < 32; ++e) v[e] = __float_as_uint(gelu_erf_fast(__uint_as_float(v[e])));
         }
         bf16* dst = args.y + static_cast<long long>(m) * args.ldy + n0;
         if (whole) {

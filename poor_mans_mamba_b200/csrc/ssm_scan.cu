@@ -287,6 +287,67 @@ __global__ void __launch_bounds__(kGroupWarps * 32)
   }
 }
 
+// The same for widths that are a multiple of 4: LANES lanes share a (token, group), four neighbouring entries a lane and
+// piece, P pieces.
+template <typename S, typename Y, int LANES, int P>
+__global__ void __launch_bounds__(256)
+    gated_norm_narrow_vec_kernel(const Y* __restrict__ y, const S* __restrict__ z_raw, long long ld_z, float z_scale,
+                                 const float* __restrict__ z_bias, const float* __restrict__ w, float eps, S* __restrict__ out,
+                                 long long ld_out, int T, int I, int group_width, int gate_sigmoid) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int groups = I / group_width;
+  const long long item = (static_cast<long long>(blockIdx.x) * 256 + threadIdx.x) / LANES;
+  const bool ok = item < static_cast<long long>(T) * groups;   // (whole warps take part in the sums)
+  const int t = ok ? static_cast<int>(item / groups) : 0, c0 = ok ? static_cast<int>(item % groups) * group_width : 0;
+  const int lane = threadIdx.x % LANES;
+  float4 v[P], z[P];
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < P; ++j) {
+    const int i = 4 * (lane + LANES * j);
+    v[j] = z[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (ok && i < group_width) {
+      v[j] = ldf4(y + static_cast<size_t>(t) * I + c0 + i);
+      z[j] = ldf4(z_raw + static_cast<long long>(t) * ld_z + c0 + i);
+    }
+    ss += v[j].x * v[j].x + v[j].y * v[j].y + v[j].z * v[j].z + v[j].w * v[j].w;
+  }
+#pragma unroll
+  for (int o = LANES / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  const float inv = 1.0f / sqrtf(ss / static_cast<float>(group_width) + eps);
+  auto gate = [&](float zz, float b) {
+    const float x = zz * z_scale + b;
+    return gate_sigmoid ? 1.f / (1.f + expf(-x)) : silu_f(x);
+  };
+#pragma unroll
+  for (int j = 0; j < P; ++j) {
+    const int i = 4 * (lane + LANES * j);
+    if (ok && i < group_width) {
+      const int c = c0 + i;
+      const float4 g = ldf4(w + c), b = z_bias ? ldf4(z_bias + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      stf4(out + static_cast<long long>(t) * ld_out + c,
+           make_float4(v[j].x * inv * g.x * gate(z[j].x, b.x), v[j].y * inv * g.y * gate(z[j].y, b.y),
+                       v[j].z * inv * g.z * gate(z[j].z, b.z), v[j].w * inv * g.w * gate(z[j].w, b.w)));
+    }
+  }
+}
+
+template <typename S, typename Y>
+void launch_gated_norm_narrow(const Y* y, const S* z, long long ld_z, float z_scale, const float* z_bias, const float* w, float eps,
+                              S* out, long long ld_out, int T, int I, int gw, int gate_sigmoid, cudaStream_t stream) {
+  auto aligned = [](const void* p, size_t bytes) { return reinterpret_cast<uintptr_t>(p) % bytes == 0; };
+  const long long items = static_cast<long long>(T) * (I / gw);
+  const bool vec = gw % 4 == 0 && ld_z % 4 == 0 && ld_out % 4 == 0 && aligned(y, 4 * sizeof(Y)) && aligned(z, 4 * sizeof(S)) &&
+                   aligned(out, 4 * sizeof(S)) && aligned(w, 16) && aligned(z_bias, 16);
+  const int lanes = !vec ? 32 : gw <= 32 ? 8 : gw <= 64 ? 16 : 32;
+  auto kern = !vec ? gated_norm_narrow_kernel<S, Y>
+            : gw <= 32 ? gated_norm_narrow_vec_kernel<S, Y, 8, 1> : gw <= 64 ? gated_norm_narrow_vec_kernel<S, Y, 16, 1>
+            : gw <= 128 ? gated_norm_narrow_vec_kernel<S, Y, 32, 1> : gated_norm_narrow_vec_kernel<S, Y, 32, 2>;
+  launch_pdl(kern, dim3(static_cast<unsigned>((items * lanes + 255) / 256)), dim3(256), 0, stream, y, z, ld_z, z_scale, z_bias, w,
+             eps, out, ld_out, T, I, gw, gate_sigmoid);
+}
+
 template <typename S>
 int launch_scan(const void* xbc, int ld_xbc, const void* dt_raw, long long ld_dt, float dt_scale,
                 const float* dt_shift, const float* a_log, const float* d_skip, float* state,
@@ -357,17 +418,14 @@ PMM_EXPORT int pmm_gated_norm(const void* y, const void* z_raw, long long ld_z, 
   if (n_groups <= 0 || I % n_groups || n_groups > 65535) return PMM_ERR_BAD_ARGUMENT;
   const int gw = I / n_groups;
   if (w && norm_before_gate && n_groups > 1 && gw <= 256) {
-    const long long items = static_cast<long long>(T) * n_groups;
-    const dim3 narrow(static_cast<unsigned>((items + pmm::kGroupWarps - 1) / pmm::kGroupWarps));
-#define PMM_NARROW_CASE(Y)                                                                                             \
-  pmm::launch_pdl(pmm::gated_norm_narrow_kernel<S, Y>, narrow, dim3(pmm::kGroupWarps * 32), 0, stream,                 \
-                  static_cast<const Y*>(y), static_cast<const S*>(z_raw), ld_z, z_scale, z_bias, w, eps,               \
-                  static_cast<S*>(out), ld_out, T, I, gw, gate_sigmoid)
     PMM_DISPATCH_DTYPE(dtype, S, {
-      if (y_f32) PMM_NARROW_CASE(float);
-      else PMM_NARROW_CASE(S);
+      if (y_f32)
+        pmm::launch_gated_norm_narrow<S, float>(static_cast<const float*>(y), static_cast<const S*>(z_raw), ld_z, z_scale, z_bias, w,
+                                                eps, static_cast<S*>(out), ld_out, T, I, gw, gate_sigmoid, stream);
+      else
+        pmm::launch_gated_norm_narrow<S, S>(static_cast<const S*>(y), static_cast<const S*>(z_raw), ld_z, z_scale, z_bias, w, eps,
+                                            static_cast<S*>(out), ld_out, T, I, gw, gate_sigmoid, stream);
     });
-#undef PMM_NARROW_CASE
     return pmm::launch_status();
   }
   const size_t smem = w ? static_cast<size_t>(gw) * sizeof(float) * (norm_before_gate ? 2 : 1) : 0;

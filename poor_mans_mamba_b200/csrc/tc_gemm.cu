@@ -1,6 +1,6 @@
 // Blackwell tensor-core matrix product with a fused SwiGLU epilogue for prompt portions:
 //   act[t, f] = silu((x W_gate^T)[t, f] * gate_mult) * (x W_up^T)[t, f]         (bfloat16 out)
-// or, in plain mode, y = x W^T (optionally with the exact form of GELU on it).  x [T, K] and W [rows, K] are bfloat16, K-major.
+// or, in plain mode, y = x W^T.  x [T, K] and W [rows, K] are bfloat16, K-major.
 //
 // One block computes a 256-token x 128-feature tile of act (two 128 x 256 accumulators, one per
 // half of the tokens: the 128 gate columns next to their 128 up columns) with the
@@ -45,9 +45,7 @@ constexpr size_t kTcSmem = static_cast<size_t>(kTcStages) * (kTcABytes + kTcBByt
 // (limit rides in gate_mult's place).
 // kTcGeluGlu: the same layout with act = gelu_tanh(gate * gate_mult) * up, the tanh form of GELU,
 //   gelu_tanh(z) = 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))) = z / (1 + exp(-2 sqrt(2/pi) (z + 0.044715 z^3))).
-// kTcGelu: plain layout, y = gelu(x W^T) in the erf form.
-enum { kTcPlain = 0, kTcSwiglu = 1, kTcClampedGlu = 2, kTcGeluGlu = 3, kTcGelu = 4 };
-__host__ __device__ constexpr bool tc_gated(int mode) { return mode != kTcPlain && mode != kTcGelu; }
+enum { kTcPlain = 0, kTcSwiglu = 1, kTcClampedGlu = 2, kTcGeluGlu = 3 };
 
 __device__ __forceinline__ float gelu_tanh_fast(float z) {
   return __fdividef(z, 1.f + __expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
@@ -75,7 +73,7 @@ __global__ void __launch_bounds__(kTcThreads)
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int m0 = blockIdx.x * kTcM;
-  const int n0 = blockIdx.y * (tc_gated(MODE) ? kTcN / 2 : kTcN);  // first output column
+  const int n0 = blockIdx.y * (MODE != kTcPlain ? kTcN / 2 : kTcN);  // first output column
   const int k_blocks = K / kTcK;
 
   if (threadIdx.x == 0) {
@@ -112,7 +110,7 @@ __global__ void __launch_bounds__(kTcThreads)
         mbar_expect_tx(&bar_full[s], kTcABytes + kTcBBytes);
         tma_load_2d(sA + s * kTcABytes, &map_x, kb * kTcK, m0, &bar_full[s]);                               // tokens 0..127
         tma_load_2d(sA + s * kTcABytes + kTcABytes / 2, &map_x, kb * kTcK, m0 + kTcMH, &bar_full[s]);      // tokens 128..255
-        if (tc_gated(MODE)) {
+        if (MODE != kTcPlain) {
           tma_load_2d(sB + s * kTcBBytes, &map_w, kb * kTcK, n0, &bar_full[s]);                      // gate rows
           tma_load_2d(sB + s * kTcBBytes + kTcBBytes / 2, &map_w, kb * kTcK, F + n0, &bar_full[s]);  // up rows
         } else {
@@ -170,7 +168,7 @@ __global__ void __launch_bounds__(kTcThreads)
       asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
       const int m = m0 + mhalf * kTcMH + quad * 32 + lane;  // this thread's token row
       const unsigned lane_base = tmem_base + (static_cast<unsigned>(quad * 32) << 16) + mhalf * kTcN;
-      if (tc_gated(MODE)) {
+      if (MODE != kTcPlain) {
 #pragma unroll 1
         for (int c = 0; c < kTcN / 64; ++c) {
           unsigned g[32], u[32];
@@ -218,10 +216,8 @@ __global__ void __launch_bounds__(kTcThreads)
               uint4 pack;
               __nv_bfloat162* p2 = reinterpret_cast<__nv_bfloat162*>(&pack);
 #pragma unroll
-              for (int e = 0; e < 4; ++e) {
-                const float y0 = __uint_as_float(v[j + 2 * e]), y1 = __uint_as_float(v[j + 2 * e + 1]);
-                p2[e] = MODE == kTcGelu ? __floats2bfloat162_rn(gelu_erf_f(y0), gelu_erf_f(y1)) : __floats2bfloat162_rn(y0, y1);
-              }
+              for (int e = 0; e < 4; ++e)
+                p2[e] = __floats2bfloat162_rn(__uint_as_float(v[j + 2 * e]), __uint_as_float(v[j + 2 * e + 1]));
               *reinterpret_cast<uint4*>(dst + j) = pack;
             }
           }
@@ -257,13 +253,13 @@ inline bool make_map(CUtensorMap* map, const void* base, long long rows, long lo
 // multiple of 128 (SwiGLU: F) or 256 (plain), 16-byte aligned rows.
 PMM_EXPORT int pmm_tc_gemm_supported(int mode, int K, int n_out, long long ldx, long long ld_out) {
   if (K <= 0 || K % pmm::kTcK || ldx % 8 || ld_out % 8) return 0;
-  return pmm::tc_gated(mode) ? (n_out % 128 == 0) : (n_out % 256 == 0);
+  return mode != pmm::kTcPlain ? (n_out % 128 == 0) : (n_out % 256 == 0);
 }
 
 // mode 1: out[T, F] = silu((x Wg^T) * gate_mult) * (x Wu^T) with w = [Wg; Wu] ([2F, K]).
 // mode 2: the same layout with the clamped gated activation (limit = gate_mult, act_alpha, act_shift).
 // mode 3: the same layout with gelu_tanh on the gate (gate_mult as in mode 1).
-// mode 0: out[T, N] = x w^T with w [N, K]; mode 4: gelu of that.  status: one int, stays 0 unless a bounded wait gave up.
+// mode 0: out[T, N] = x w^T with w [N, K].  status: one int, stays 0 unless a bounded wait gave up.
 namespace pmm {
 template <int MODE>
 int launch_tc_gemm(const CUtensorMap& map_x, const CUtensorMap& map_w, dim3 grid, void* out, long long ld_out, int T, int K,
@@ -281,14 +277,14 @@ PMM_EXPORT int pmm_tc_gemm_act(int mode, const void* x, long long ldx, const voi
                                int K, int n_out, float gate_mult, float act_alpha, float act_shift, int* status,
                                cudaStream_t stream) {
   if (T <= 0) return 0;
-  if (mode < 0 || mode > 4 || !pmm_tc_gemm_supported(mode, K, n_out, ldx, ld_out) || !status) return PMM_ERR_BAD_ARGUMENT;
+  if (mode < 0 || mode > 3 || !pmm_tc_gemm_supported(mode, K, n_out, ldx, ld_out) || !status) return PMM_ERR_BAD_ARGUMENT;
   if (reinterpret_cast<uintptr_t>(x) % 16 || reinterpret_cast<uintptr_t>(w) % 16 || reinterpret_cast<uintptr_t>(out) % 16)
     return PMM_ERR_BAD_ARGUMENT;
   CUtensorMap map_x, map_w;
-  const long long w_rows = pmm::tc_gated(mode) ? 2LL * n_out : n_out;
+  const long long w_rows = mode != pmm::kTcPlain ? 2LL * n_out : n_out;
   if (!pmm::make_map(&map_x, x, T, K, ldx, pmm::kTcMH) || !pmm::make_map(&map_w, w, w_rows, K, K, pmm::kTcN / 2))
     return PMM_ERR_BAD_ARGUMENT;
-  const int cols_per_block = pmm::tc_gated(mode) ? pmm::kTcN / 2 : pmm::kTcN;
+  const int cols_per_block = mode != pmm::kTcPlain ? pmm::kTcN / 2 : pmm::kTcN;
   dim3 grid((T + pmm::kTcM - 1) / pmm::kTcM, n_out / cols_per_block);
   if (mode == pmm::kTcSwiglu)
     return pmm::launch_tc_gemm<pmm::kTcSwiglu>(map_x, map_w, grid, out, ld_out, T, K, n_out, gate_mult, act_alpha, act_shift,
@@ -299,9 +295,6 @@ PMM_EXPORT int pmm_tc_gemm_act(int mode, const void* x, long long ldx, const voi
   if (mode == pmm::kTcClampedGlu)
     return pmm::launch_tc_gemm<pmm::kTcClampedGlu>(map_x, map_w, grid, out, ld_out, T, K, n_out, gate_mult, act_alpha,
                                                    act_shift, status, stream);
-  if (mode == pmm::kTcGelu)
-    return pmm::launch_tc_gemm<pmm::kTcGelu>(map_x, map_w, grid, out, ld_out, T, K, n_out, gate_mult, act_alpha, act_shift,
-                                             status, stream);
   return pmm::launch_tc_gemm<pmm::kTcPlain>(map_x, map_w, grid, out, ld_out, T, K, n_out, gate_mult, act_alpha, act_shift,
                                             status, stream);
 }

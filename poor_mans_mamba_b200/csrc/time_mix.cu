@@ -20,30 +20,13 @@ struct RowPiece<S, 1> {
   static __device__ __forceinline__ void load(const S* p, float (&v)[1]) { v[0] = ldf(p); }
   static __device__ __forceinline__ void store(S* p, const float (&v)[1]) { stf(p, v[0]); }
 };
-template <>
-struct RowPiece<float, 4> {
-  static __device__ __forceinline__ void load(const float* p, float (&v)[4]) {
-    const float4 x = *reinterpret_cast<const float4*>(p);
+template <typename S>
+struct RowPiece<S, 4> {
+  static __device__ __forceinline__ void load(const S* p, float (&v)[4]) {
+    const float4 x = ldf4(p);
     v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w;
   }
-  static __device__ __forceinline__ void store(float* p, const float (&v)[4]) {
-    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
-  }
-};
-template <>
-struct RowPiece<__nv_bfloat16, 4> {
-  static __device__ __forceinline__ void load(const __nv_bfloat16* p, float (&v)[4]) {
-    const uint2 raw = *reinterpret_cast<const uint2*>(p);
-    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
-    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
-    v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
-  }
-  static __device__ __forceinline__ void store(__nv_bfloat16* p, const float (&v)[4]) {
-    uint2 raw;
-    *reinterpret_cast<__nv_bfloat162*>(&raw.x) = __floats2bfloat162_rn(v[0], v[1]);
-    *reinterpret_cast<__nv_bfloat162*>(&raw.y) = __floats2bfloat162_rn(v[2], v[3]);
-    *reinterpret_cast<uint2*>(p) = raw;
-  }
+  static __device__ __forceinline__ void store(S* p, const float (&v)[4]) { stf4(p, make_float4(v[0], v[1], v[2], v[3])); }
 };
 
 // A block takes the columns blockIdx.y * kMixThreads * VEC .. of `tokens` consecutive rows from blockIdx.x * tokens on.
@@ -94,7 +77,7 @@ __global__ void __launch_bounds__(kMixThreads)
   }
 }
 
-// ---- a = tanh(z) w^T: a block takes 64 channels and 8 tokens at a time; z [T, R], w [C, R]
+// ---- a = tanh(z) w^T: a block takes 32 channels and up to 16 tokens, 8 at a time; z [T, R], w [C, R]
 constexpr int kLrThreads = 256;
 constexpr int kLrChannels = 32;  // channels per block, 8 lanes each
 
@@ -164,7 +147,7 @@ PMM_EXPORT int pmm_low_rank_tanh(const void* z, long long ld_z, const void* w, f
                                  cudaStream_t stream) {
   if (T <= 0) return 0;
   if (C <= 0 || R <= 0 || R > 2048) return PMM_ERR_BAD_ARGUMENT;
-  int tokens = 64;
+  int tokens = 16;  // (more of them a block: less of w read twice, but fewer blocks)
   while (tokens > 8 && sizeof(float) * static_cast<size_t>(tokens) * R > 40 * 1024) tokens /= 2;
   const size_t smem = sizeof(float) * static_cast<size_t>(tokens) * R;
   const dim3 grid((C + pmm::kLrChannels - 1) / pmm::kLrChannels, (T + tokens - 1) / tokens);

@@ -1718,9 +1718,8 @@ def tc_gemm_clamped_glu(x: Tensor, gate_up: Tensor, limit: float, alpha: float, 
           float(limit), float(alpha), float(shift), _tc_status(x.device).data_ptr(), _stream())
 
 
-def tc_gemm(x: Tensor, weight: Tensor, out: Tensor, gelu: bool = False) -> None:
-    """out[T, N] = x @ weight^T on tcgen05 (bfloat16 in and out, float accumulation); ``gelu``: the exact form of GELU in
-    the epilogue."""
+def tc_gemm(x: Tensor, weight: Tensor, out: Tensor) -> None:
+    """out[T, N] = x @ weight^T on tcgen05 (bfloat16 in and out, float accumulation)."""
     _cuda(x, weight, out)
     T, K = x.shape
     N = weight.shape[0]
@@ -1729,10 +1728,6 @@ def tc_gemm(x: Tensor, weight: Tensor, out: Tensor, gelu: bool = False) -> None:
         raise KernelError("tc_gemm: out must be bfloat16 [T, N], rows 16-byte aligned")
     if not (tc_gemm_supported(x, weight, N, False)):
         raise KernelError("tc_gemm: sizes or alignment outside what the kernel takes")
-    if gelu:
-        _call("pmm_tc_gemm_act", 4, x.data_ptr(), x.stride(0), weight.data_ptr(), out.data_ptr(), out.stride(0), T, K, N,
-              1.0, 0.0, 0.0, _tc_status(x.device).data_ptr(), _stream())
-        return
     _call("pmm_tc_gemm", 0, x.data_ptr(), x.stride(0), weight.data_ptr(), out.data_ptr(), out.stride(0), T, K, N,
           1.0, _tc_status(x.device).data_ptr(), _stream())
 

@@ -550,8 +550,8 @@ def test_the_two_sides_are_normed_and_halved(dtype):
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("T,D,F", [(1, 64, 96), (5, 50, 33), (16, 256, 512), (40, 1024, 320), (64, 2048, 64), (63, 96, 40), (300, 64, 88), (6000, 128, 1024)])
 def test_plain_feed_forward_in_all_its_forms(dtype, T, D, F):
-    """Weight-streaming products of up to 64 tokens in both tensor-core forms, the tcgen05 product of many tokens, and the
-    library product with a launch for the activation; GELU's exact form (the tanh form differs by up to 5e-4)."""
+    """Weight-streaming products of up to 64 tokens in both tensor-core forms, and the library product with a launch for the
+    activation; GELU's exact form (the tanh form differs by up to 5e-4)."""
     part = build_part("feed_forward", PartSpec("mlp", "mlp", {"intermediate_size": F, "activation": "gelu", "tensors": ("up", "down")}), hidden_size=D)
     up, down = rnd(F, D, seed=1, scale=1.5 * D ** -0.5), rnd(D, F, seed=2, scale=F ** -0.5)
     part.bind({"up": up.to(DEV, dtype), "down": down.to(DEV, dtype)})
@@ -571,6 +571,12 @@ def test_gelu_is_exact_where_the_tanh_form_is_not():
     close(x[0], P.gelu_erf(z.double()), torch.float32, "gelu", f32=1e-6)
     tanh_form = torch.nn.functional.gelu(z.double(), approximate="tanh")
     assert float((P.gelu_erf(z.double()) - tanh_form).abs().max()) > 1e-4
+    zb = z.to(torch.bfloat16)     # the short form for bfloat16 results: within half a step of bfloat16 and 1e-6 of the exact one
+    for width in (4000, 4001):    # eight elements a thread, and one by one
+        y = zb[:width].to(DEV).view(1, -1).clone()
+        K.gelu_(y)
+        want = P.gelu_erf(zb[:width].double())
+        assert bool(((y[0].double().cpu() - want).abs() <= want.abs() * 2.0 ** -8 + 1e-6).all())
     t = z.to(DEV).view(1, -1).clone()
     K.tanh_(t)
     close(t[0], torch.tanh(z.double()), torch.float32, "tanh", f32=1e-6)
