@@ -1146,7 +1146,9 @@ def paged_attention(q: Tensor, pool: Tensor, block_table: Tensor, positions: Ten
                     new_lens: Optional[Sequence[int]] = None, use_tensor_cores: bool = True,
                     split_counter: Optional[Tensor] = None, tile_rows: Optional[int] = None,
                     sink: Optional[Tensor] = None, keep_first: int = 0, lse: Optional[Tensor] = None) -> None:
-    """Causal attention of every token over keys lo..pos of its request in the paged cache.
+    """Causal attention of every token over keys lo..pos of its request in the paged cache.  ``window`` > 0: the last
+    ``window`` keys; below zero: the keys of the token's own chunk of -window positions, counted from position 0 (in
+    `flash_decode_attention` and `attention_tc` likewise).
     ``keep_first``: the request's first keep_first keys stay visible behind a window (at their true positions).
     The float kernel walks both key ranges itself; the tensor-core kernel takes them with one key split and
     ``lse`` (float32 [T, Hq, 2] scratch): it leaves every row's maximum and sum there and `kept_first_merge` adds

@@ -387,7 +387,7 @@ def _random_config(seed):
             mixer = C.attention(G * rng.randint(1, 6), G, dim, dv, dim ** -0.5, rot=rot, yarn=yarn if rot else None, v_mix=v_mix)
         elif kind == "parallel":
             G, dim, rd = rng.choice([1, 2, 3]), rng.choice([8, 16, 48, 64, 96]), rng.choice([8, 16, 32, 64, 96])
-            decays = [rng.choice([0.5, 0.9, 0.96875, 0.99, 0.998]) for _ in range(rng.randint(1, 6))]
+            decays = [rng.choice([0.5, 0.9, 0.97, 0.99, 0.998]) for _ in range(rng.randint(1, 6))]
             mixer = C.parallel((G * rng.randint(1, 4), G, dim, rng.choice([dim, 16, 40]), dim ** -0.5, rng.choice([1, 7, 16, 40, 64, 100])),
                                (rd, rng.choice([rd, 16, 48]), decays, (rng.choice([rd, rd // 2]), rng.choice([100.0, 1e6]))))
         else:
